@@ -88,3 +88,6 @@ class ModelSpec:
     # Entries of the run order before which the rows are mixed with the embedded rows (``PassInput``).
     pass_inputs: tuple = ()
     pass_input_name: str = "loop."
+    # Residual streams (0: one plain residual row): every row starts as so many copies of the embedded row, the layers'
+    # blocks mix them (block ``streams``), and their sum is what the final norm reads.
+    streams: int = 0

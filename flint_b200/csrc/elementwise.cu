@@ -13,10 +13,11 @@ using namespace flint;
 // --------------------------------------------------------------------------- embed
 // fed_rows (may be null): for each row -1, or the place in `fed_from` (the sampler's last output, still on the
 // device) that holds the row's token: a decoded token can be fed to the next step before the host has read it.
+// out [T, copies, H]: every row is written `copies` times.
 template <typename TT>
 __global__ void embed_kernel(const int* __restrict__ ids, const int* __restrict__ fed_rows,
                              const int* __restrict__ fed_from, const TT* __restrict__ table,
-                             float* __restrict__ out, int T, int H, int V, float scale) {
+                             float* __restrict__ out, int T, int H, int V, float scale, int copies) {
   pdl_launch();
   pdl_wait();
   const int r = blockIdx.x;
@@ -24,19 +25,22 @@ __global__ void embed_kernel(const int* __restrict__ ids, const int* __restrict_
   int id = fed >= 0 ? fed_from[fed] : ids[r];
   id = id < 0 ? 0 : (id >= V ? V - 1 : id);  // ids are validated on the host; never read outside
   const TT* src = table + (size_t)id * H;
-  float* dst = out + (size_t)r * H;
-  for (int d = threadIdx.x; d < H; d += blockDim.x) dst[d] = to_f32(src[d]) * scale;
+  float* dst = out + (size_t)r * copies * H;
+  for (int d = threadIdx.x; d < H; d += blockDim.x) {
+    const float v = to_f32(src[d]) * scale;
+    for (int k = 0; k < copies; ++k) dst[(size_t)k * H + d] = v;
+  }
 }
 
 extern "C" int flint_embed(const int* ids, const int* fed_rows, const int* fed_from, const void* table, int table_dtype,
-                           float* out, int T, int H, int V, float scale, cudaStream_t stream) {
+                           float* out, int T, int H, int V, float scale, int copies, cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (H <= 0 || V <= 0) return fail("embed: bad sizes H=%d V=%d", H, V);
+  if (H <= 0 || V <= 0 || copies < 1) return fail("embed: bad sizes H=%d V=%d copies=%d", H, V, copies);
   if ((fed_rows == nullptr) != (fed_from == nullptr)) return fail("embed: fed rows and their source come together");
   const int threads = H >= 1024 ? 256 : (H >= 256 ? 128 : 64);
   FLINT_DISPATCH_DTYPE(table_dtype, TT,
       launch_pdl(embed_kernel<TT>, dim3(T), dim3(threads), 0, stream, ids, fed_rows, fed_from, (const TT*)table, out, T,
-                 H, V, scale));
+                 H, V, scale, copies));
   return check_launch("embed");
 }
 
@@ -436,7 +440,7 @@ extern "C" int flint_add_partials(float* x, const float* partials, int n_partial
 // rows that made them).
 template <typename TO>
 __global__ void gated_act_kernel(const float* __restrict__ p, int S, long long stride, TO* __restrict__ out,
-                                 int rows, int I, int act, float p0, float p1) {
+                                 int rows, int I, int act, float p0, float p1, const float* __restrict__ bias) {
   pdl_launch();
   pdl_wait();
   const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -447,6 +451,10 @@ __global__ void gated_act_kernel(const float* __restrict__ p, int S, long long s
     const float* row = p + (size_t)z * stride + (size_t)r * paired_rows(I) + paired_gate_row(c);
     g += row[0];
     u += row[GATE_BLOCK];
+  }
+  if (bias) {              // paired like the columns
+    g += bias[paired_gate_row(c)];
+    u += bias[paired_gate_row(c) + GATE_BLOCK];
   }
   float y;
   if (act == 2) {          // clamped: g = min(g, c), u = clamp(u, -c, c); g sigmoid(slope g) (u + 1); p0 = slope, p1 = c
@@ -462,14 +470,14 @@ __global__ void gated_act_kernel(const float* __restrict__ p, int S, long long s
 }
 
 extern "C" int flint_gated_act(const float* partials, int S, long long stride, void* out, int out_dtype, int rows,
-                               int I, int act, float p0, float p1, cudaStream_t stream) {
+                               int I, int act, float p0, float p1, const float* bias, cudaStream_t stream) {
   const long long n = (long long)rows * I;
   if (n <= 0) return 0;
   if (S < 1) return fail("gated_act: needs at least one partial");
   if (act < 0 || act > 2) return fail("gated_act: unknown activation %d", act);
   FLINT_DISPATCH_DTYPE(out_dtype, TO,
       launch_pdl(gated_act_kernel<TO>, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream, partials, S, stride,
-                 (TO*)out, rows, I, act, p0, p1));
+                 (TO*)out, rows, I, act, p0, p1, bias));
   return check_launch("gated_act");
 }
 

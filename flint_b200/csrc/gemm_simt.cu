@@ -29,7 +29,7 @@ gemm_simt_kernel(const TX* __restrict__ x, int ldx, const TW* __restrict__ w, co
                  TO* __restrict__ out, int ldo, int accumulate, int act,
                  const int* __restrict__ tile_expert, const int* __restrict__ tile_row0,
                  const int* __restrict__ n_tiles, const int* __restrict__ offsets, int tile_rows,
-                 long long expert_stride, int M, int N, int K) {
+                 long long expert_stride, int M, int N, int K, float act_slope, float act_limit) {
   __shared__ float xs[BK][BM + 4];
   __shared__ float ws[BK][BN + 4];
   __shared__ float us[GATED ? BK : 1][BN + 4];
@@ -90,8 +90,22 @@ gemm_simt_kernel(const TX* __restrict__ x, int ldx, const TW* __restrict__ w, co
       const int gc = col0 + tx * 4 + j;
       if (gc >= N) continue;
       float v = acc[i][j];
-      if (GATED) v = act_fn(v, act) * acc_u[i][j];
-      if (bias) v += bias[gc];
+      if (GATED) {          // a gated product's bias is paired like its weight rows and comes before the activation
+        float up = acc_u[i][j];
+        if (bias) {
+          v += bias[paired_gate_row(gc)];
+          up += bias[paired_gate_row(gc) + GATE_BLOCK];
+        }
+        if (act == 2) {     // clamped: gate sigmoid(slope gate) (up + 1)
+          v = fminf(v, act_limit);
+          up = fminf(fmaxf(up, -act_limit), act_limit);
+          v = v / (1.0f + expf(-act_slope * v)) * (up + 1.0f);
+        } else {
+          v = act_fn(v, act) * up;
+        }
+      } else if (bias) {
+        v += bias[gc];
+      }
       const size_t o = (size_t)gr * ldo + gc;
       if (accumulate) v += to_f32(out[o]);
       out[o] = from_f32<TO>(v);
@@ -105,11 +119,14 @@ gemm_simt_kernel(const TX* __restrict__ x, int ldx, const TW* __restrict__ w, co
 // Dense: tile_expert == NULL, rows = M, one "expert".  Grouped: rows of expert e are
 // offsets[e] .. offsets[e+1]-1, and tile i covers up to tile_rows (<= 64) rows from tile_row0[i] of
 // expert tile_expert[i]; only the first *n_tiles tiles exist (max_tiles bounds the grid).
+// A gated product's bias has paired_rows(N) entries and is added before the activation; act 2 is the clamped form with
+// act_slope and act_limit.
 extern "C" int flint_gemm_simt(const void* x, int x_dtype, int ldx, const void* w, int gated,
                                int w_dtype, const float* bias, void* out, int out_dtype, int ldo,
                                int accumulate, int act, const int* tile_expert,
                                const int* tile_row0, const int* n_tiles, const int* offsets,
-                               int max_tiles, int tile_rows, int M, int N, int K, cudaStream_t stream) {
+                               int max_tiles, int tile_rows, int M, int N, int K, float act_slope, float act_limit,
+                               cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (K <= 0) return fail("gemm_simt: K=%d", K);
   const long long expert_stride = (long long)(gated ? paired_rows(N) : N) * K;
@@ -124,11 +141,11 @@ extern "C" int flint_gemm_simt(const void* x, int x_dtype, int ldx, const void* 
     if (gated)                                                                                    \
       gemm_simt_kernel<TX, TW, TO, true><<<grid, THREADS, 0, stream>>>(                           \
           (const TX*)x, ldx, (const TW*)w, bias, (TO*)out, ldo, accumulate, act,                  \
-          tile_expert, tile_row0, n_tiles, offsets, tile_rows, expert_stride, M, N, K);                                     \
+          tile_expert, tile_row0, n_tiles, offsets, tile_rows, expert_stride, M, N, K, act_slope, act_limit);                                     \
     else                                                                                          \
       gemm_simt_kernel<TX, TW, TO, false><<<grid, THREADS, 0, stream>>>(                          \
           (const TX*)x, ldx, (const TW*)w, bias, (TO*)out, ldo, accumulate, act,                  \
-          tile_expert, tile_row0, n_tiles, offsets, tile_rows, expert_stride, M, N, K);                                     \
+          tile_expert, tile_row0, n_tiles, offsets, tile_rows, expert_stride, M, N, K, act_slope, act_limit);                                     \
   } while (0)
   FLINT_DISPATCH_DTYPE(x_dtype, TX, FLINT_DISPATCH_DTYPE(w_dtype, TW,
       FLINT_DISPATCH_DTYPE(out_dtype, TO, LAUNCH(TX, TW, TO))));

@@ -75,6 +75,13 @@ struct Params {
 // parameters go into a second kernel argument.
 static_assert(sizeof(Params) <= 128, "keep the parameter struct within 128 bytes");
 
+// What only gated products take: the constants of the clamped activation, and biases of the gate and up values (paired
+// like the weight rows that make them; null: none).
+struct GateParams {
+  const float* bias;
+  float slope, limit;
+};
+
 // Instruction descriptor, kind::f16: fp32 accumulator, bf16 A and B, both K-major, M = 128, N = bn.
 __device__ __forceinline__ uint32_t instr_desc(int bn) {
   return (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(bn >> 3) << 17) | ((uint32_t)(BM >> 4) << 24);
@@ -85,12 +92,23 @@ __device__ __forceinline__ float act_fn(float g, int act) {
   return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
 }
 
+// act 0, 1: act(gate) * up; act 2: gate and up clamped, gate sigmoid(slope gate) (up + 1)
+__device__ __forceinline__ float gated_fn(float gate, float up, int act, const GateParams& gp) {
+  if (act == 2) {
+    gate = fminf(gate, gp.limit);
+    up = fminf(fmaxf(up, -gp.limit), gp.limit);
+    return gate / (1.0f + __expf(-gp.slope * gate)) * (up + 1.0f);
+  }
+  return act_fn(gate, act) * up;
+}
+
 // Persistent: a block walks over work items (feature tile, row tile, piece of K) with a stride of the
 // grid.  The TMA ring runs on across items, and the accumulator is double-buffered in tensor memory, so
 // the epilogue of one item overlaps the main loop of the next.
 template <int BN, bool GATED>
 __global__ void __launch_bounds__(THREADS)
-gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x, const Params p) {
+gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x, const Params p,
+               const GateParams gp) {
   extern __shared__ uint8_t smem_raw[];
   __shared__ __align__(8) uint64_t bars[2 * 16 + 4];   // full[stages], empty[stages], acc_full[2], acc_empty[2]
   __shared__ uint32_t tmem_holder;
@@ -287,7 +305,9 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
       // features (lanes 0-15 hold its gate values, lanes 16-31 its up values)
       const int f = GATED ? w.f0 + q * GATE_BLOCK + (lane & 15) : w.f0 + q * 32 + lane;
       const bool f_ok = f < p.N;
-      const float bias = (p.bias && f_ok && !raw) ? p.bias[f] : 0.f;
+      const float bias = (!GATED && p.bias && f_ok && !raw) ? p.bias[f] : 0.f;
+      const float gate_bias = (GATED && gp.bias && f_ok) ? gp.bias[paired_gate_row(f)] : 0.f;
+      const float up_bias = (GATED && gp.bias && f_ok) ? gp.bias[paired_gate_row(f) + GATE_BLOCK] : 0.f;
       const uint32_t lane_addr = tmem + buf * ACC_COLS + ((uint32_t)(q * 32) << 16);
       constexpr int CH = BN < 32 ? 16 : 32;         // columns fetched from tensor memory at a time
 #pragma unroll 1
@@ -306,8 +326,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
 #pragma unroll
             for (int c = 0; c < 4; ++c) {
               const float got = __shfl_xor_sync(0xffffffffu, low ? v[4 + c] : v[c], 16);
-              const float gate = low ? v[c] : got, up = low ? got : v[4 + c];
-              v[c] = act_fn(gate, p.act) * up;
+              const float gate = (low ? v[c] : got) + gate_bias, up = (low ? got : v[4 + c]) + up_bias;
+              v[c] = gated_fn(gate, up, p.act, gp);
             }
           }
 #pragma unroll
@@ -413,7 +433,7 @@ int weight_map(CUtensorMap* m, const void* ptr, long long rows, int K, int box_r
 }
 
 template <int BN, bool GATED>
-int launch(const CUtensorMap& mw, const CUtensorMap& mx, const Params& p, dim3 grid, cudaStream_t stream) {
+int launch(const CUtensorMap& mw, const CUtensorMap& mx, const Params& p, const GateParams& gp, dim3 grid, cudaStream_t stream) {
   constexpr int stage_bytes = BM * BK * 2 + BN * BK * 2;
   const size_t smem = (size_t)p.stages * stage_bytes + 1024;
   static bool configured = false;   // per instantiation
@@ -438,7 +458,7 @@ int launch(const CUtensorMap& mw, const CUtensorMap& mx, const Params& p, dim3 g
   const long long items = p.stream_k ? (long long)grid.x * grid.y * ((p.K + BK - 1) / BK)
                                      : (long long)grid.x * grid.y * grid.z;
   const unsigned blocks = (unsigned)(items < (long long)sm_count * per_sm ? items : (long long)sm_count * per_sm);
-  launch_pdl(gemm_tc_kernel<BN, GATED>, dim3(blocks), dim3(THREADS), smem, stream, mw, mx, p);
+  launch_pdl(gemm_tc_kernel<BN, GATED>, dim3(blocks), dim3(THREADS), smem, stream, mw, mx, p, gp);
   return check_launch("gemm_tc");
 }
 
@@ -479,11 +499,14 @@ extern "C" long long flint_gemm_tc_partial_floats(int rows, int N, int splits) {
 // starts, because a product over the same map ran between the two (it lets its dependents start only after its
 // own wait for the map's kernel); the first weight tiles are then fetched before the wait for the kernel before.
 // error_flag: device int, set to 1 if a bounded wait ran out.
+// A gated product's bias has paired_rows(N) entries, paired like the rows of w, and is added before the activation;
+// act 2 is the clamped form, g = min(gate, act_limit), u = clamp(up, -act_limit, act_limit), g sigmoid(act_slope g) (u + 1).
 extern "C" int flint_gemm_tc(const void* x, int ldx, const void* w, int gated, const float* bias, void* out,
                              int out_dtype, int ldo, int accumulate, int act, const int* tile_expert,
                              const int* tile_row0, const int* n_tiles, const int* offsets, int max_tiles,
                              int n_experts, int rows, int N, int K, int bn, int splits, float* partial,
-                             int defer, int stream_k, int plan_ready, int* error_flag, cudaStream_t stream) {
+                             int defer, int stream_k, int plan_ready, int* error_flag, float act_slope,
+                             float act_limit, cudaStream_t stream) {
   if (rows <= 0 || N <= 0) return 0;
   if (K <= 0 || (K & 7)) return fail("gemm_tc: K=%d must be a positive multiple of 8 (16-byte rows for TMA)", K);
   if (ldx < K || (ldx & 7)) return fail("gemm_tc: row stride %d must be a multiple of 8 and at least K", ldx);
@@ -516,6 +539,10 @@ extern "C" int flint_gemm_tc(const void* x, int ldx, const void* w, int gated, c
   p.w_expert_rows = w_expert_rows;
   p.plan_ready = (tile_expert && plan_ready) ? 1 : 0;
   p.wait_cycles = wait_limit();
+  GateParams gp;
+  gp.bias = w_up ? bias : nullptr;
+  gp.slope = act_slope;
+  gp.limit = act_limit;
   p.stages = flint_gemm_tc_stages(bn, w_up ? 1 : 0);
   // few rows: the product streams its weights and is bound by how many bytes an SM keeps in flight and by how
   // evenly the tiles spread; four stages of 18 KB let three blocks share an SM (444 resident blocks)
@@ -525,7 +552,7 @@ extern "C" int flint_gemm_tc(const void* x, int ldx, const void* w, int gated, c
   int rc;
 #define CASE(B)                                                                             \
   case B:                                                                                   \
-    rc = w_up ? launch<B, true>(mw, mx, p, grid, stream) : launch<B, false>(mw, mx, p, grid, stream); \
+    rc = w_up ? launch<B, true>(mw, mx, p, gp, grid, stream) : launch<B, false>(mw, mx, p, gp, grid, stream); \
     break;
   switch (bn) {
     CASE(16) CASE(32) CASE(64) CASE(128) CASE(256)

@@ -7,13 +7,18 @@
 // against key j is qa[t, h] . row_j, and its output in latent space is sum_j p_j c_j: every head
 // attends over the same rows, and the values are the first C numbers of the keys.
 //
+//   flint_latent_down       for queries that go through a latent of their own: sums the partial sums of the down
+//                           projections [q latent | latent and rotated key part | ...], norms the q latent (out in the
+//                           activation type) and writes the cache row
 //   flint_latent_prepare    sums the partial sums of the q (and latent) projection, rotates the
 //                           rotated parts (neighbouring dims 2i, 2i+1 or halves i, i+n/2), norms the
 //                           latent and writes the cache row; q_plain and the rotated q part go out
 //                           in the activation type
 //   flint_latent_attention  one warp per (row, chunk of 4 heads, split of the key range): a lane owns
 //                           a key in the score phase and output dims lane, lane+32, ... in the value
-//                           phase; online softmax in float32; splits are merged in a fixed order
+//                           phase; online softmax in float32; splits are merged in a fixed order.  A sink (a logit
+//                           per head that joins the denominator and has no key) is what the first split's maximum
+//                           and sum start from
 //
 // The reference has no such mixer (its attention is grouped-query over cached keys and values:
 // crates/thuban_kernel/wgsl/attn.wgsl); these kernels have no counterpart there.
@@ -26,6 +31,54 @@ namespace {
 constexpr int GC = 4;           // heads per warp
 constexpr int WARPS = 4;
 constexpr int MAX_DPL = 16;     // output dims per lane: latent size <= 512
+
+// One column's partial sums, added in order with up to eight loads in flight.
+__device__ __forceinline__ float sum_partials(const float* col, int n_partials, long long stride) {
+  float s = 0.f;
+  for (int z0 = 0; z0 < n_partials; z0 += 8) {
+    float v[8];
+#pragma unroll
+    for (int u = 0; u < 8; ++u) v[u] = z0 + u < n_partials ? col[(size_t)(z0 + u) * stride] : 0.f;
+#pragma unroll
+    for (int u = 0; u < 8; ++u) s += v[u];
+  }
+  return s;
+}
+
+// A token's cache row from the sums total(base ..): the latent divided by its root mean square and scaled, the rotated
+// key part, zeros to the row's end.  The whole block calls; sm holds C floats of the block's own (each thread reads
+// back what it wrote).
+template <typename Total, typename TC>
+__device__ __forceinline__ void write_latent_row(Total total, int base, const float* __restrict__ norm_w, float eps,
+                                                 const float* __restrict__ cos_t, const float* __restrict__ sin_t,
+                                                 int rot_dims, int interleaved, int p, long long cache_row,
+                                                 TC* __restrict__ k_cache, int R, int C, int row_w, float* sm, float* red) {
+  const int half = rot_dims / 2, units = half + (R - rot_dims);
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < C; i += blockDim.x) {
+    const float v = total(base + i);
+    sm[i] = v;
+    ss += v * v;
+  }
+  ss = block_sum(ss, red);
+  const float inv = 1.0f / sqrtf(ss / (float)C + eps);
+  if (cache_row < 0) return;
+  TC* dst = k_cache + cache_row * row_w;
+  for (int i = threadIdx.x; i < C; i += blockDim.x) dst[i] = from_f32<TC>(sm[i] * inv * norm_w[i]);
+  for (int u = threadIdx.x; u < units; u += blockDim.x) {
+    if (u < half) {
+      const int d0 = interleaved ? 2 * u : u, d1 = interleaved ? 2 * u + 1 : u + half;
+      const float a = total(base + C + d0), b = total(base + C + d1);
+      const float c = cos_t[(size_t)p * half + u], s = sin_t[(size_t)p * half + u];
+      dst[C + d0] = from_f32<TC>(a * c - b * s);
+      dst[C + d1] = from_f32<TC>(b * c + a * s);
+    } else {
+      const int d = rot_dims + (u - half);
+      dst[C + d] = from_f32<TC>(total(base + C + d));
+    }
+  }
+  for (int i = C + R + threadIdx.x; i < row_w; i += blockDim.x) dst[i] = from_f32<TC>(0.f);
+}
 
 template <typename TQ, typename TC>
 __global__ void __launch_bounds__(256)
@@ -50,11 +103,7 @@ latent_prepare_kernel(const float* __restrict__ proj, int n_partials, long long 
   pdl_wait();
   if (missing && threadIdx.x == 0) atomicExch(status, 1);
   const float* row = proj + (size_t)t * W;
-  auto total = [&](int col) {
-    float s = 0.f;
-    for (int z = 0; z < n_partials; ++z) s += row[(size_t)z * partial_stride + col];
-    return s;
-  };
+  auto total = [&](int col) { return sum_partials(row + col, n_partials, partial_stride); };
   const int half = rot_dims / 2, DR = D + R, Dk = C + R;
   const int units = half + (R - rot_dims);        // rotating pairs, then the dims that pass unchanged
   // the pair of unit u (< half) and the rotation of (a, b) by the angle of pair u at position p
@@ -83,32 +132,45 @@ latent_prepare_kernel(const float* __restrict__ proj, int n_partials, long long 
     }
   }
   if (!write_kv) return;
-  const int base = H * DR;
+  write_latent_row(total, H * DR, norm_w, eps, cos_t, sin_t, rot_dims, interleaved, p, cache_row, k_cache, R, C, row_w, sm, red);
+}
+
+// proj [S][T, W], columns [q latent (Q) | latent (C) | rotated key part (R) | ...]: c_q = rmsnorm(q latent) out, and, with
+// write_kv, the token's cache row.  One block per row.
+template <typename TQ, typename TC>
+__global__ void __launch_bounds__(256)
+latent_down_kernel(const float* __restrict__ proj, int n_partials, long long partial_stride, int W, int Q,
+                   const float* __restrict__ q_norm, const int* __restrict__ pos, const int* __restrict__ slot,
+                   const float* __restrict__ cos_t, const float* __restrict__ sin_t, int rot_dims, int interleaved,
+                   const float* __restrict__ norm_w, float eps, TQ* __restrict__ c_q, TC* __restrict__ k_cache,
+                   const int* __restrict__ block_table, int max_pages, int page_size, int R, int C, int row_w,
+                   int write_kv, int* __restrict__ status) {
+  extern __shared__ float sm[];         // Q floats of the q latent, then C of the latent, before their norms
+  __shared__ float red[32];
+  pdl_launch();
+  const int t = blockIdx.x, p = pos[t];
+  long long cache_row = -1;
+  bool missing = false;
+  if (write_kv) {
+    const int page = block_table[(size_t)slot[t] * max_pages + p / page_size];
+    if (page >= 0) cache_row = (long long)page * page_size + p % page_size;
+    else missing = true;
+  }
+  pdl_wait();
+  if (missing && threadIdx.x == 0) atomicExch(status, 1);
+  const float* row = proj + (size_t)t * W;
+  auto total = [&](int col) { return sum_partials(row + col, n_partials, partial_stride); };
   float ss = 0.f;
-  for (int i = threadIdx.x; i < C; i += blockDim.x) {
-    const float v = total(base + i);
+  for (int i = threadIdx.x; i < Q; i += blockDim.x) {
+    const float v = total(i);
     sm[i] = v;
     ss += v * v;
   }
   ss = block_sum(ss, red);
-  const float inv = 1.0f / sqrtf(ss / (float)C + eps);
-  if (cache_row < 0) return;
-  TC* dst = k_cache + cache_row * row_w;
-  for (int i = threadIdx.x; i < C; i += blockDim.x) dst[i] = from_f32<TC>(sm[i] * inv * norm_w[i]);
-  for (int u = threadIdx.x; u < units; u += blockDim.x) {
-    if (u < half) {
-      int d0, d1;
-      dims_of(u, d0, d1);
-      const float a = total(base + C + d0), b = total(base + C + d1);
-      const float c = cos_t[(size_t)p * half + u], s = sin_t[(size_t)p * half + u];
-      dst[C + d0] = from_f32<TC>(a * c - b * s);
-      dst[C + d1] = from_f32<TC>(b * c + a * s);
-    } else {
-      const int d = rot_dims + (u - half);
-      dst[C + d] = from_f32<TC>(total(base + C + d));
-    }
-  }
-  for (int i = Dk + threadIdx.x; i < row_w; i += blockDim.x) dst[i] = from_f32<TC>(0.f);
+  const float inv = 1.0f / sqrtf(ss / (float)Q + eps);
+  for (int i = threadIdx.x; i < Q; i += blockDim.x) c_q[(size_t)t * Q + i] = from_f32<TQ>(sm[i] * inv * q_norm[i]);
+  if (!write_kv) return;
+  write_latent_row(total, Q, norm_w, eps, cos_t, sin_t, rot_dims, interleaved, p, cache_row, k_cache, R, C, row_w, sm + Q, red);
 }
 
 template <typename TQ, typename TC, typename TO>
@@ -117,7 +179,7 @@ latent_attention_kernel(const TQ* __restrict__ qa, const TC* __restrict__ k_cach
                         int max_pages, int page_size, const int* __restrict__ pos, const int* __restrict__ slot,
                         TO* __restrict__ out, float* __restrict__ scratch, int T, int H, int C, int Dk, int row_w,
                         int window, float scale, int split_keys, int n_splits, int g_chunks,
-                        const int* __restrict__ row_list) {
+                        const int* __restrict__ row_list, const float* __restrict__ sinks) {
   extern __shared__ float smem[];   // per warp: GC * row_w floats of q
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const long long item = (long long)blockIdx.x * WARPS + warp;
@@ -147,8 +209,9 @@ latent_attention_kernel(const TQ* __restrict__ qa, const TC* __restrict__ k_cach
   float m[GC], l[GC], acc[GC][MAX_DPL];
 #pragma unroll
   for (int g = 0; g < GC; ++g) {
-    m[g] = -INFINITY;
-    l[g] = 0.f;
+    const bool sink = sinks && split == 0 && g < ng;      // e^(sink - m) = 1
+    m[g] = sink ? sinks[h0 + g] : -INFINITY;
+    l[g] = sink ? 1.f : 0.f;
 #pragma unroll
     for (int i = 0; i < MAX_DPL; ++i) acc[g][i] = 0.f;
   }
@@ -267,7 +330,7 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ qa, const __nv_bfl
                             const int* __restrict__ block_table, int max_pages, int page_size,
                             const int* __restrict__ pos, const int* __restrict__ slot, __nv_bfloat16* __restrict__ out,
                             float* __restrict__ scratch, int T, int H, int C, int Dk, int row_w, int Dkp, int window,
-                            float scale, int nt, int nh, int split_keys, int n_splits) {
+                            float scale, int nt, int nh, int split_keys, int n_splits, const float* __restrict__ sinks) {
   using flint_attn::ldsm4;
   using flint_attn::ldsm4t;
   using flint_attn::mma16816;
@@ -353,6 +416,11 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ qa, const __nv_bfl
     };
     const int p_lo = p_a + r_lo / nhh, p_hi = p_a + r_hi / nhh;   // positions of this lane's rows (if they are in the run)
     float m_lo = -INFINITY, m_hi = -INFINITY, l_lo = 0.f, l_hi = 0.f;
+    if (sinks && split == 0) {                                    // the sink joins the denominator once: 2^(sink - m) = 1
+      m_lo = sinks[h0 + r_lo % nhh] * 1.4426950408889634f;
+      m_hi = sinks[h0 + r_hi % nhh] * 1.4426950408889634f;
+      l_lo = l_hi = 1.f;
+    }
     float o[NTW][4];
 #pragma unroll
     for (int i = 0; i < NTW; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
@@ -516,15 +584,24 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ qa, const __nv_bfl
 }
 // ---------------------------------------------------------------------------------------------
 // A small product per head, all heads in one launch: out[t, h, :] = W[h] x[t, h, :] (bfloat16 in and out,
-// float32 sums).  x and out may be views into wider rows (strides in elements).  Block (64 tokens, 64 outputs,
+// float32 sums), optionally times sigmoid(gate[t, h, :]), the gate given as float32 partial sums.  x and out may be views into wider rows (strides in elements).  Block (64 tokens, 64 outputs,
 // head): four warps of 16 tokens each, operands staged in shared memory 64 columns at a time, the next stage on
 // its way while this one is multiplied.
 constexpr int HP_M = 64, HP_N = 64, HP_K = 64, HP_S = HP_K + 8;
 
+struct HeadGate {              // column h N + n of row t: sum of n_partials numbers `stride` apart; z null: no gate
+  const float* z;
+  int n_partials;
+  long long stride, row;
+  __device__ __forceinline__ float at(int t, int col) const {
+    return 1.0f / (1.0f + expf(-sum_partials(z + (size_t)t * row + col, n_partials, stride)));
+  }
+};
+
 __global__ void __launch_bounds__(128)
 head_products_kernel(const __nv_bfloat16* __restrict__ x, long long sx_t, long long sx_h,
                      const __nv_bfloat16* __restrict__ w, __nv_bfloat16* __restrict__ out, long long so_t,
-                     long long so_h, int T, int N, int K) {
+                     long long so_h, int T, int N, int K, const HeadGate gate) {
   using flint_attn::ldsm4;
   using flint_attn::mma16816;
   __shared__ __align__(16) __nv_bfloat16 As[2][HP_M * HP_S];      // two stages, filled by asynchronous copies
@@ -590,8 +667,13 @@ head_products_kernel(const __nv_bfloat16* __restrict__ x, long long sx_t, long l
 #pragma unroll
     for (int nb = 0; nb < HP_N / 8; ++nb) {
       const int n = n0 + nb * 8 + 2 * (lane & 3);
-      if (n < N) dst[n] = __float2bfloat16_rn(acc[nb][2 * half]);
-      if (n + 1 < N) dst[n + 1] = __float2bfloat16_rn(acc[nb][2 * half + 1]);
+      float v0 = acc[nb][2 * half], v1 = acc[nb][2 * half + 1];
+      if (gate.z) {
+        if (n < N) v0 *= gate.at(t, h * N + n);
+        if (n + 1 < N) v1 *= gate.at(t, h * N + n + 1);
+      }
+      if (n < N) dst[n] = __float2bfloat16_rn(v0);
+      if (n + 1 < N) dst[n + 1] = __float2bfloat16_rn(v1);
     }
   }
 }
@@ -602,7 +684,7 @@ constexpr int HPS_T = 16;        // tokens at most
 __global__ void __launch_bounds__(256)
 head_products_small_kernel(const __nv_bfloat16* __restrict__ x, long long sx_t, long long sx_h,
                            const __nv_bfloat16* __restrict__ w, __nv_bfloat16* __restrict__ out, long long so_t,
-                           long long so_h, int T, int N, int K) {
+                           long long so_h, int T, int N, int K, const HeadGate gate) {
   extern __shared__ float xs[];                  // [T][K]
   pdl_launch();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -640,12 +722,27 @@ head_products_small_kernel(const __nv_bfloat16* __restrict__ x, long long sx_t, 
         acc[t] += wf[0] * x0.x + wf[1] * x0.y + wf[2] * x0.z + wf[3] * x0.w + wf[4] * x1.x + wf[5] * x1.y + wf[6] * x1.z + wf[7] * x1.w;
       }
   }
+  float mine = 0.f;                              // lane t keeps token t's sum
 #pragma unroll
   for (int t = 0; t < HPS_T; ++t)
     if (t < T) {
       const float v = warp_sum(acc[t]);
-      if (lane == 0) out[(size_t)t * so_t + (size_t)h * so_h + n] = __float2bfloat16_rn(v);
+      if (lane == t) mine = v;
     }
+  if (lane < T) {
+    if (gate.z) mine *= gate.at(lane, h * N + n);
+    out[(size_t)lane * so_t + (size_t)h * so_h + n] = __float2bfloat16_rn(mine);
+  }
+}
+
+// x[t, c] <- x[t, c] sigmoid(gate[t, c]) in place: for products that do not take the gate along.
+template <typename TX>
+__global__ void gate_rows_kernel(TX* __restrict__ x, const HeadGate gate, int T, int N) {
+  pdl_launch();
+  pdl_wait();
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= (long long)T * N) return;
+  x[i] = from_f32<TX>(to_f32(x[i]) * gate.at((int)(i / N), (int)(i % N)));
 }
 }  // namespace
 
@@ -674,12 +771,13 @@ extern "C" int flint_latent_prepare(const float* proj, int n_partials, long long
   return check_launch("latent_prepare");
 }
 
-// qa [T, H, Dk] -> out [T, H, C] (both q_dtype); scratch holds T*H*n_splits*(C+2) floats when n_splits > 1.
+// qa [T, H, Dk] -> out [T, H, C] (both q_dtype); scratch holds T*H*n_splits*(C+2) floats when n_splits > 1; sinks [H] or
+// null.
 extern "C" int flint_latent_attention(const void* qa, int q_dtype, const void* k_cache, int cache_dtype,
                                       const int* block_table, int max_pages, int page_size, const int* pos,
                                       const int* slot, void* out, int T, int H, int C, int Dk, int row_w, int window,
                                       float scale, int split_keys, int n_splits, float* scratch,
-                                      const int* row_list, cudaStream_t stream) {
+                                      const int* row_list, const float* sinks, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (C < 1 || C > 32 * MAX_DPL) return fail("latent_attention: latent size %d (supported: 1..%d)", C, 32 * MAX_DPL);
   if (Dk < C || row_w < Dk || (row_w & 7)) return fail("latent_attention: bad row sizes C=%d Dk=%d row=%d", C, Dk, row_w);
@@ -698,7 +796,7 @@ extern "C" int flint_latent_attention(const void* qa, int q_dtype, const void* k
                            200 * 1024);                                                                         \
     latent_attention_kernel<TQ, TC, TQ><<<(unsigned)blocks, WARPS * 32, smem, stream>>>(                        \
         (const TQ*)qa, (const TC*)k_cache, block_table, max_pages, page_size, pos, slot, (TQ*)out, scratch, T,  \
-        H, C, Dk, row_w, window, scale, split_keys, n_splits, g_chunks, row_list);                              \
+        H, C, Dk, row_w, window, scale, split_keys, n_splits, g_chunks, row_list, sinks);                       \
   } while (0)
   FLINT_DISPATCH_DTYPE(q_dtype, TQ, FLINT_DISPATCH_DTYPE(cache_dtype, TC, LAUNCH(TQ, TC)));
 #undef LAUNCH
@@ -716,7 +814,7 @@ extern "C" int flint_latent_attention(const void* qa, int q_dtype, const void* k
 extern "C" int flint_latent_attention_mma(const void* qa, const void* k_cache, const int* block_table, int max_pages,
                                           int page_size, const int* pos, const int* slot, void* out, int T, int H, int C,
                                           int Dk, int row_w, int window, float scale, int nt, int nh, int split_keys,
-                                          int n_splits, float* scratch, cudaStream_t stream) {
+                                          int n_splits, float* scratch, const float* sinks, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (C < 1 || C > 512) return fail("latent_attention: latent size %d (supported: 1..512)", C);
   if (Dk < C || row_w < Dk || (row_w & 7)) return fail("latent_attention: bad row sizes C=%d Dk=%d row=%d", C, Dk, row_w);
@@ -737,7 +835,8 @@ extern "C" int flint_latent_attention_mma(const void* qa, const void* k_cache, c
       cudaFuncSetAttribute(latent_attention_mma_kernel<N>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);  \
     launch_pdl(latent_attention_mma_kernel<N>, grid, dim3(TC_THREADS), smem, stream,                                  \
                (const __nv_bfloat16*)qa, (const __nv_bfloat16*)k_cache, block_table, max_pages, page_size, pos, slot, \
-               (__nv_bfloat16*)out, scratch, T, H, C, Dk, row_w, Dkp, window, scale, nt, nh, split_keys, n_splits);   \
+               (__nv_bfloat16*)out, scratch, T, H, C, Dk, row_w, Dkp, window, scale, nt, nh, split_keys, n_splits, \
+               sinks);                                                                                                 \
   } while (0)
   if (C <= 64) LAUNCH(2);
   else if (C <= 128) LAUNCH(4);
@@ -754,21 +853,61 @@ extern "C" int flint_latent_attention_mma(const void* qa, const void* k_cache, c
 
 // out[t, h, :] = W[h] x[t, h, :] for all heads: x [T, H, K] and out [T, H, N] bfloat16 with strides (elements) per
 // token and per head, w [H, N, K] bfloat16.  K and the strides of x must be multiples of 8, x and w 16-byte aligned.
+// gate (or null): out is multiplied by sigmoid of the sum of gate_partials float32 numbers gate_stride apart, at row t and
+// column h N + n of rows gate_row numbers apart.
 extern "C" int flint_head_products(const void* x, long long sx_t, long long sx_h, const void* w, void* out,
-                                   long long so_t, long long so_h, int T, int H, int N, int K, cudaStream_t stream) {
+                                   long long so_t, long long so_h, int T, int H, int N, int K, const float* gate,
+                                   int gate_partials, long long gate_stride, long long gate_row, cudaStream_t stream) {
   if (T <= 0 || H <= 0 || N <= 0) return 0;
   if (K <= 0 || (K & 7) || (sx_t & 7) || (sx_h & 7) || ((uintptr_t)x & 15) || ((uintptr_t)w & 15))
     return fail("head_products: K=%d and the strides of x must be multiples of 8, x and w 16-byte aligned", K);
   if (H > 65535 || (N + HP_N - 1) / HP_N > 65535) return fail("head_products: too many heads or outputs");
+  if (gate && gate_partials < 1) return fail("head_products: a gate needs at least one partial");
+  const HeadGate hg = {gate, gate_partials, gate_stride, gate_row};
   if (T <= HPS_T && (size_t)T * K * sizeof(float) <= 48 * 1024) {
     launch_pdl(head_products_small_kernel, dim3((N + 7) / 8, H), dim3(256), (size_t)T * K * sizeof(float), stream,
-               (const __nv_bfloat16*)x, sx_t, sx_h, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, so_t, so_h, T, N, K);
+               (const __nv_bfloat16*)x, sx_t, sx_h, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, so_t, so_h, T, N, K,
+               hg);
     return check_launch("head_products (few tokens)");
   }
   dim3 grid((T + HP_M - 1) / HP_M, (N + HP_N - 1) / HP_N, H);
   launch_pdl(head_products_kernel, grid, dim3(128), 0, stream, (const __nv_bfloat16*)x, sx_t, sx_h,
-             (const __nv_bfloat16*)w, (__nv_bfloat16*)out, so_t, so_h, T, N, K);
+             (const __nv_bfloat16*)w, (__nv_bfloat16*)out, so_t, so_h, T, N, K, hg);
   return check_launch("head_products");
+}
+
+// x [T, N] <- x sigmoid(gate) in place; the gate as in flint_head_products.
+extern "C" int flint_gate_rows(void* x, int dtype, const float* gate, int gate_partials, long long gate_stride,
+                               long long gate_row, int T, int N, cudaStream_t stream) {
+  if (T <= 0 || N <= 0) return 0;
+  if (!gate || gate_partials < 1) return fail("gate_rows: needs a gate");
+  const HeadGate hg = {gate, gate_partials, gate_stride, gate_row};
+  FLINT_DISPATCH_DTYPE(dtype, TX,
+      launch_pdl(gate_rows_kernel<TX>, dim3((unsigned)(((long long)T * N + 255) / 256)), dim3(256), 0, stream, (TX*)x, hg, T, N));
+  return check_launch("gate_rows");
+}
+
+// proj [S, T, W] float32 partial sums, columns [q latent (Q) | latent (C) | rotated key part (R) | ...]; c_q [T, Q] in
+// q_dtype; with write_kv the cache row of each token as in flint_latent_prepare (else the columns are [q latent | ...]).
+extern "C" int flint_latent_down(const float* proj, int n_partials, long long partial_stride, int W, int Q,
+                                 const float* q_norm, const int* pos, const int* slot, const float* cos_t,
+                                 const float* sin_t, int rot_dims, int interleaved, const float* norm_w, float eps,
+                                 void* c_q, int q_dtype, void* k_cache, int cache_dtype, const int* block_table,
+                                 int max_pages, int page_size, int T, int R, int C, int row_w, int write_kv, int* status,
+                                 cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (n_partials < 1) return fail("latent_down: needs at least one partial");
+  if (Q < 1 || R < 0 || C < 1 || W < Q + (write_kv ? C + R : 0)) return fail("latent_down: bad sizes Q=%d R=%d C=%d W=%d", Q, R, C, W);
+  if (rot_dims < 0 || rot_dims > R || (rot_dims & 1)) return fail("latent_down: %d rotating dims do not fit %d", rot_dims, R);
+  if (write_kv && (row_w < C + R || (row_w & 7))) return fail("latent_down: cache rows of %d numbers do not hold %d", row_w, C + R);
+  if (write_kv && (!k_cache || !norm_w || page_size <= 0)) return fail("latent_down: no cache to write to");
+  const size_t smem = (size_t)(Q + C) * sizeof(float);
+  if (smem > 48 * 1024) return fail("latent_down: latents of %d and %d numbers are too large", Q, C);
+  FLINT_DISPATCH_DTYPE(q_dtype, TQ, FLINT_DISPATCH_DTYPE(cache_dtype, TC,
+      (launch_pdl(latent_down_kernel<TQ, TC>, dim3(T), dim3(256), smem, stream, proj, n_partials, partial_stride, W, Q,
+                  q_norm, pos, slot, cos_t, sin_t, rot_dims, interleaved, norm_w, eps, (TQ*)c_q, (TC*)k_cache, block_table,
+                  max_pages, page_size, R, C, row_w, write_kv, status))));
+  return check_launch("latent_down");
 }
 
 extern "C" const char* flint_latent_last_error() { return g_error; }

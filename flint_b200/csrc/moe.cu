@@ -178,7 +178,9 @@ router_topk_kernel(const float* __restrict__ x, const TW* __restrict__ wr, int t
 }
 
 // One block.  expert_ids [T*top] -> per-expert counts, offsets (exclusive scan), the sorted row
-// of every (token, choice) and the tile map for the grouped products.
+// of every (token, choice) and the tile map for the grouped products.  Numbers from E on name experts that have no
+// weights and hand a token's own row on: their choices take no sorted row and get row_of = n_assign + token instead, and
+// the sorted rows that are left over at the end get token_of = -1.
 __global__ void moe_plan_kernel(const int* __restrict__ expert_ids, int n_assign, int E,
                                 int tile_rows, int* __restrict__ counts, int* __restrict__ offsets,
                                 int* __restrict__ row_of, int* __restrict__ token_of,
@@ -192,7 +194,8 @@ __global__ void moe_plan_kernel(const int* __restrict__ expert_ids, int n_assign
   __syncthreads();
   // rank of each assignment inside its expert (the order inside an expert has no effect on
   // any result: rows are independent in the products and are added back per token)
-  for (int a = threadIdx.x; a < n_assign; a += blockDim.x) row_of[a] = atomicAdd(&cnt[expert_ids[a]], 1);
+  for (int a = threadIdx.x; a < n_assign; a += blockDim.x)
+    if (expert_ids[a] < E) row_of[a] = atomicAdd(&cnt[expert_ids[a]], 1);
   __syncthreads();
   if (threadIdx.x == 0) {
     int run = 0, tiles = 0;
@@ -214,7 +217,12 @@ __global__ void moe_plan_kernel(const int* __restrict__ expert_ids, int n_assign
     *n_tiles = tiles < max_tiles ? tiles : max_tiles;
   }
   __syncthreads();
+  for (int r = off[E] + threadIdx.x; r < n_assign; r += blockDim.x) token_of[r] = -1;
   for (int a = threadIdx.x; a < n_assign; a += blockDim.x) {
+    if (expert_ids[a] >= E) {
+      row_of[a] = n_assign + a / top;
+      continue;
+    }
     const int row = off[expert_ids[a]] + row_of[a];
     row_of[a] = row;
     token_of[row] = a / top;
@@ -239,6 +247,7 @@ moe_dispatch_kernel(const int* __restrict__ expert_ids, int n_assign, int E, int
   pdl_wait();
   const int tid = threadIdx.x;
   if (tid < n_assign) ids[tid] = expert_ids[tid];
+  if (tid == 0) my_token = -1;
   __syncthreads();
   if (tid < E) {
     int c = 0;
@@ -274,7 +283,9 @@ moe_dispatch_kernel(const int* __restrict__ expert_ids, int n_assign, int E, int
     }
   }
   __syncthreads();
-  if (tid < n_assign) {
+  if (tid < n_assign && ids[tid] >= E) {
+    if (blockIdx.x == 0) row_of[tid] = n_assign + tid / top;
+  } else if (tid < n_assign) {
     const int row = off[ids[tid]] + rank;
     if (blockIdx.x == 0) {
       row_of[tid] = row;
@@ -282,7 +293,10 @@ moe_dispatch_kernel(const int* __restrict__ expert_ids, int n_assign, int E, int
     }
     if (row == (int)blockIdx.x) my_token = tid / top;
   }
+  if (blockIdx.x == 0)
+    for (int r = off[E] + tid; r < n_assign; r += blockDim.x) token_of[r] = -1;
   __syncthreads();
+  if (my_token < 0) return;                     // a sorted row that no choice takes
   const uint4* src = x + (size_t)my_token * row_vecs;
   uint4* dst = xs + (size_t)blockIdx.x * row_vecs;
   for (int i = tid; i < row_vecs; i += blockDim.x) dst[i] = src[i];
@@ -405,13 +419,13 @@ extern "C" int flint_router_sigmoid(const float* x, const void* wr, int w_dtype,
   return check_launch("router_sigmoid");
 }
 
-// The grouped sigmoid router (select_sigmoid_grouped_by_warp) as a kernel of its own: a warp takes RT tokens, walks
+// The router with corrected choice scores (select_corrected_by_warp) as a kernel of its own: a warp takes RT tokens, walks
 // the experts' weight rows once for all of them, then selects token by token.
 template <typename TW>
 __global__ void __launch_bounds__(128)
 router_sigmoid_grouped_kernel(const float* __restrict__ x, const TW* __restrict__ wr, const float* __restrict__ correction,
-                              int T, int H, int E, int top, int n_groups, int keep, int normalize, float out_scale,
-                              int* __restrict__ expert_ids, float* __restrict__ gates, float* __restrict__ logits_out) {
+                              int softmax, int T, int H, int E, int top, int n_groups, int keep, int normalize,
+                              float out_scale, int* __restrict__ expert_ids, float* __restrict__ gates, float* __restrict__ logits_out) {
   extern __shared__ float smem[];            // per warp: RT * E logits, then E choice scores
   pdl_launch();
   pdl_wait();
@@ -445,14 +459,15 @@ router_sigmoid_grouped_kernel(const float* __restrict__ x, const TW* __restrict_
     if (logits_out)
       for (int e = lane; e < E; e += 32) logits_out[(size_t)t * E + e] = zr[e];
     __syncwarp();
-    select_sigmoid_grouped_by_warp(zr, c, correction, lane, E, top, n_groups, keep, normalize, out_scale,
-                                   expert_ids + (size_t)t * top, gates + (size_t)t * top);
+    select_corrected_by_warp(zr, c, correction, softmax != 0, lane, E, top, n_groups, keep, normalize, out_scale,
+                             expert_ids + (size_t)t * top, gates + (size_t)t * top);
     __syncwarp();
   }
 }
 
-extern "C" int flint_router_sigmoid_grouped(const float* x, const void* wr, int w_dtype, const float* correction, int E,
-                                            int top, int n_groups, int keep, int normalize, float out_scale,
+// softmax != 0: the scores are the softmax of the logits instead of their sigmoids.
+extern "C" int flint_router_sigmoid_grouped(const float* x, const void* wr, int w_dtype, const float* correction,
+                                            int softmax, int E, int top, int n_groups, int keep, int normalize, float out_scale,
                                             int* expert_ids, float* gates, float* logits_out, int T, int H,
                                             cudaStream_t stream) {
   if (T <= 0) return 0;
@@ -463,8 +478,8 @@ extern "C" int flint_router_sigmoid_grouped(const float* x, const void* wr, int 
   if (smem > 48 * 1024) return fail("router_sigmoid_grouped: too many experts (%d)", E);
   const unsigned blocks = (unsigned)((T + 4 * RT - 1) / (4 * RT));
   FLINT_DISPATCH_DTYPE(w_dtype, TW,
-      launch_pdl(router_sigmoid_grouped_kernel<TW>, dim3(blocks), dim3(128), smem, stream, x, (const TW*)wr, correction, T, H,
-                 E, top, n_groups, keep, normalize, out_scale, expert_ids, gates, logits_out));
+      launch_pdl(router_sigmoid_grouped_kernel<TW>, dim3(blocks), dim3(128), smem, stream, x, (const TW*)wr, correction, softmax, T,
+                 H, E, top, n_groups, keep, normalize, out_scale, expert_ids, gates, logits_out));
   return check_launch("router_sigmoid_grouped");
 }
 

@@ -170,16 +170,16 @@ class CudaOps:
                 self._fn(m, f"flint_{m}_last_error")
 
     # ------------------------------------------------------------------ row-wise
-    def embed(self, ids, table, out, scale=1.0, fed_rows=None, fed_from=None):
-        """Rows of the table by token id.  ``fed_rows`` [T] with ``fed_from``: where a row's entry is not
+    def embed(self, ids, table, out, scale=1.0, fed_rows=None, fed_from=None, copies=1):
+        """Rows of the table by token id (``out`` [T, H]; with ``copies`` each written so many times, [T, copies, H]).  ``fed_rows`` [T] with ``fed_from``: where a row's entry is not
         negative, its token is read from that place of ``fed_from`` (tokens sampled on the device that the
         host has not read yet) instead of ``ids``."""
         _check(ids, "ids", torch.int32, 1)
         _check(table, "table", dims=2)
-        _check(out, "out", torch.float32, 2)
+        _check(out, "out", torch.float32)
         T, (V, H) = ids.numel(), table.shape
-        if tuple(out.shape) != (T, H):
-            raise KernelError(f"embed: out must be [{T}, {H}]")
+        if tuple(out.shape) not in ((T, copies, H),) + (((T, H),) if copies == 1 else ()):
+            raise KernelError(f"embed: out must be [{T}, {H}] or [{T}, copies, {H}]")
         if (fed_rows is None) != (fed_from is None):
             raise KernelError("embed: fed rows and their source come together")
         if fed_rows is not None:
@@ -188,7 +188,7 @@ class CudaOps:
             if fed_rows.numel() != T:
                 raise KernelError(f"embed: fed_rows must have {T} entries")
         self._run("elementwise", "flint_embed", _ptr(ids), _ptr(fed_rows), _ptr(fed_from), _ptr(table),
-                  c_int(_code(table.dtype)), _ptr(out), c_int(T), c_int(H), c_int(V), c_float(scale))
+                  c_int(_code(table.dtype)), _ptr(out), c_int(T), c_int(H), c_int(V), c_float(scale), c_int(copies))
 
     def norm(self, x, gamma, beta, eps, mode, out_f32=None, out_bf16=None, row_index=None):
         """mode 'layer' or 'rms'; writes float32 and/or bfloat16 copies of the result."""
@@ -208,17 +208,42 @@ class CudaOps:
         self._run("elementwise", "flint_norm", _ptr(x), _ptr(row_index), _ptr(gamma), _ptr(beta), c_float(eps),
                   c_int({"layer": 0, "rms": 1}[mode]), _ptr(out_f32), _ptr(out_bf16), c_int(rows), c_int(H))
 
+    FUSED_STREAMS = 4      # streams of a residual row that the row kernel takes
+
     def row_norm(self, x, gamma, beta, eps, mode, out_f32=None, out_bf16=None, row_index=None, pending=None,
-                 router=None):
+                 router=None, gather=None):
         """Norm of the residual rows with what is pending applied first (x is updated in place) and,
         on request, the routing of every row.  Falls back to separate kernels for widths that the
-        fused kernel does not take."""
-        _check(x, "x", torch.float32, 2)
-        T, H = x.shape
-        if H % 4 or H > 16384 or (router is not None and (row_index is not None or H * 4 > 160000
-                                                          or router.weight.shape[0] > H
-                                                          or (getattr(router, "rule", "") == "sigmoid_grouped"
-                                                              and 2 * router.weight.shape[0] > H))):
+        fused kernel does not take.  x [T, H], or several streams of it [T, S, H]: then what is pending goes into the
+        streams by its ``mix`` and ``spread`` (x is updated in place unless ``row_index`` is given), and the norm reads
+        their sum weighted by ``gather`` [S]."""
+        _check(x, "x", torch.float32)
+        streams = x.shape[1] if x.dim() == 3 else 0
+        T, H = x.shape[0], x.shape[-1]
+        mix = spread = None
+        if streams:
+            if gamma is not None and (gather is None or gather.dtype != torch.float32 or gather.numel() != streams):
+                raise KernelError(f"row_norm: the norm of {streams} streams needs as many float32 weights")
+            if pending is not None:
+                mix, spread = pending.mix, pending.spread
+                if mix is None or spread is None or tuple(mix.shape) != (streams, streams) or spread.numel() != streams \
+                        or mix.dtype != torch.float32 or spread.dtype != torch.float32:
+                    raise KernelError("row_norm: what is pending needs the streams' float32 mixing weights")
+            if H % 4 or H > 16384 or streams > self.FUSED_STREAMS:
+                # the streams by a kernel of their own, then the norm of what it leaves
+                rows = row_index.numel() if row_index is not None else T
+                u = torch.empty((rows, H), dtype=torch.float32, device=x.device) if gamma is not None else None
+                self._stream_update(x, row_index, rows, pending, mix, spread, gather, u)
+                if u is not None:
+                    self.row_norm(u, gamma, beta, eps, mode, out_f32, out_bf16, None, None, router)
+                return
+            if router is not None and (row_index is not None or not self._router_rides(router, H)):
+                tmp = out_f32 if out_f32 is not None else torch.empty((T, H), dtype=torch.float32, device=x.device)
+                self.row_norm(x, gamma, beta, eps, mode, tmp, out_bf16, row_index, pending, None, gather)
+                return self.route(tmp, router)
+        elif x.dim() != 2:
+            raise KernelError(f"x must have 2 or 3 dims, got shape {tuple(x.shape)}")
+        if H % 4 or H > 16384 or (router is not None and (row_index is not None or not self._router_rides(router, H))):
             if pending is not None:
                 self.apply_pending(x, pending)
             tmp = out_f32
@@ -273,8 +298,9 @@ class CudaOps:
                 _check(r_aux, "router weights out", torch.float32, 2)
                 if tuple(r_aux.shape) != (T, r_top + r_extra) or r_top < 1:
                     raise KernelError(f"row_norm: the sigmoid router's weights must be [{T}, {r_top + r_extra}]")
-            elif getattr(router, "rule", "") == "sigmoid_grouped":
-                r_rule, r_corr, r_norm = 2, router.correction, 1 if router.normalize else 0
+            elif getattr(router, "rule", "") in ("sigmoid_grouped", "softmax_corrected"):
+                r_rule = 2 if router.rule == "sigmoid_grouped" else 3
+                r_corr, r_norm = router.correction, 1 if router.normalize else 0
                 if r_corr is not None and (r_corr.dtype != torch.float32 or r_corr.numel() != E):
                     raise KernelError("row_norm: the router's correction must be float32, one per expert")
         self._run("row_fused", "flint_row_norm", _ptr(x), _ptr(row_index), c_int(rows), c_int(H), _ptr(partials),
@@ -282,11 +308,40 @@ class CudaOps:
                   c_float(eps), c_int({"layer": 0, "rms": 1}[mode]), _ptr(out_f32), _ptr(out_bf16), _ptr(wr),
                   c_int(_code(wr.dtype) if wr is not None else 0), c_int(E), c_float(jit), _ptr(ids), _ptr(gates),
                   _ptr(logits), c_int(r_top), c_int(r_groups), c_int(r_keep), c_float(r_scale), c_int(r_rule), c_int(r_extra),
-                  _ptr(r_aux), _ptr(r_corr), c_int(r_norm))
+                  _ptr(r_aux), _ptr(r_corr), c_int(r_norm), c_int(streams), _ptr(mix), _ptr(spread), _ptr(gather))
+
+    @staticmethod
+    def _router_rides(router, H):
+        """Whether the row kernel can route rows of H numbers while it has them."""
+        E = router.weight.shape[0]
+        return H * 4 <= 160000 and (2 if getattr(router, "rule", "") in ("sigmoid_grouped", "softmax_corrected") else 1) * E <= H
+
+    def _stream_update(self, x, row_index, rows, pending, mix, spread, gather, u):
+        T, S, H = x.shape
+        partials = bias = y = row_of = gates = None
+        n = stride = top = 0
+        if pending is not None:
+            if pending.partials is not None:
+                partials, bias = pending.partials, pending.bias
+                _check(partials, "pending partials", torch.float32, 3)
+                if tuple(partials.shape[1:]) != (T, H):
+                    raise KernelError("stream_update: pending partial sums do not match the streams")
+                n, stride = partials.shape[0], partials.stride(0)
+            if pending.y is not None:
+                y, row_of, gates = pending.y, pending.row_of, pending.gates
+                _check(y, "pending expert rows", torch.float32, 2)
+                top = row_of.numel() // max(T, 1)
+                if y.shape[1] != H or row_of.numel() != top * T or gates.numel() != top * T:
+                    raise KernelError("stream_update: pending expert rows do not match the streams")
+        self._run("row_fused", "flint_stream_update", _ptr(x), _ptr(row_index), c_int(rows), c_int(H), _ptr(partials), c_int(n),
+                  c_longlong(stride), _ptr(bias), _ptr(y), _ptr(row_of), _ptr(gates), c_int(top), c_int(S), _ptr(mix),
+                  _ptr(spread), _ptr(gather), _ptr(u))
 
     def apply_pending(self, x, pending):
-        """x += what a part left pending (for a norm that cannot take it along)."""
-        _check(x, "x", torch.float32, 2)
+        """x += what a part left pending (for a norm that cannot take it along); x [T, S, H]: into its streams."""
+        _check(x, "x", torch.float32)
+        if x.dim() == 3:
+            return self.row_norm(x, None, None, 0.0, "layer", pending=pending)
         T, H = x.shape
         if H % 4 == 0 and H <= 16384:
             return self.row_norm(x, None, None, 0.0, "layer", pending=pending)
@@ -383,23 +438,18 @@ class CudaOps:
             flat[..., half, :, :] = w.reshape(*lead, blocks, b, k)
         return out.view(*lead, 2 * blocks * b, k)
 
-    def gated_gemm(self, x, w13, out, act="silu", plan: MoePlan | None = None, act_params=None):
-        """out = act(x @ Wg.T) * (x @ Wu.T); w13 = pair_gate_up(Wg, Wu): [paired_rows(N), K], or with a
-        plan (rows grouped by expert) [E, paired_rows(N), K].  act "swish_clamped" with act_params (slope, limit):
-        g = min(gate, limit), u = clamp(up, -limit, limit), out = g sigmoid(slope g) (u + 1); it runs as a plain
-        product over the paired rows and an activation kernel over its float32 sums."""
-        if act == "swish_clamped":
-            if act_params is None or plan is not None:
-                raise KernelError("gated_gemm: swish_clamped takes (slope, limit) and no plan")
-            _check(out, "out", dims=2)
-            M, N = out.shape
-            if w13.dim() != 2 or w13.shape[0] != self.paired_rows(N) or w13.shape[1] != x.shape[1] or x.shape[0] != M:
-                raise KernelError("gated_gemm: shapes do not match")
-            parts = self.gemm_partials(x, w13)
-            return self._run("elementwise", "flint_gated_act", _ptr(parts), c_int(parts.shape[0]), c_longlong(parts.stride(0)),
-                             _ptr(out), c_int(_code(out.dtype)), c_int(M), c_int(N), c_int(2), c_float(act_params[0]),
-                             c_float(act_params[1]))
-        self._gemm(x, w13, True, out, None, False, act, plan)
+    GATED_ACTS = {"silu": 0, "gelu_pytorch_tanh": 1, "swish_clamped": 2}
+
+    def gated_gemm(self, x, w13, out, act="silu", plan: MoePlan | None = None, act_params=None, bias=None):
+        """out = act(x @ Wg.T + bg) * (x @ Wu.T + bu); w13 = pair_gate_up(Wg, Wu): [paired_rows(N), K], or with a
+        plan (rows grouped by expert) [E, paired_rows(N), K]; ``bias`` = pair_gate_up(bg, bu) as one float32 vector
+        (dense products only).  act "swish_clamped" with act_params (slope, limit): g = min(gate, limit),
+        u = clamp(up, -limit, limit), out = g sigmoid(slope g) (u + 1)."""
+        if act not in self.GATED_ACTS or (act == "swish_clamped") != (act_params is not None):
+            raise KernelError(f"gated_gemm: activation {act!r} with constants {act_params!r}")
+        if bias is not None and (plan is not None or bias.dtype != torch.float32 or bias.numel() != self.paired_rows(out.shape[1])):
+            raise KernelError("gated_gemm: a bias is float32, paired like the weight rows, and goes with a dense product")
+        self._gemm(x, w13, True, out, bias, False, act, plan, act_params=act_params or (0.0, 0.0))
 
     ROW_ACTS = {"none": 0, "gelu": 1, "gelu_pytorch_tanh": 2, "silu": 3, "relu2": 4}
 
@@ -468,7 +518,7 @@ class CudaOps:
                   _ptr(plan.tile_row0 if plan else None), _ptr(plan.n_tiles if plan else None),
                   _ptr(plan.offsets if plan else None), c_int(plan.max_tiles if plan else 0), c_int(E), c_int(M),
                   c_int(N), c_int(K), c_int(bn), c_int(splits), _ptr(out), c_int(1), c_int(stream_k),
-                  c_int(1 if plan_ready and plan is not None else 0), _ptr(self.tc_error))
+                  c_int(1 if plan_ready and plan is not None else 0), _ptr(self.tc_error), c_float(0.0), c_float(0.0))
         return out
 
     def _k_splits(self, M, N, K, bn):
@@ -482,7 +532,7 @@ class CudaOps:
         # 32-row tile counted at three, 17 to 32 rows ran 432 items on 296 places and a decode step took 1.5 % longer)
         return max(1, min(((3 if bn < 32 else 2) * self.sm_count) // tiles, kb // 4, 16))
 
-    def _gemm(self, x, w, gated, out, bias, accumulate, act, plan, plan_ready=False):
+    def _gemm(self, x, w, gated, out, bias, accumulate, act, plan, plan_ready=False, act_params=(0.0, 0.0)):
         _check(x, "x", dims=2, contiguous=False)
         _check(out, "out", dims=2, contiguous=False)
         if x.stride(1) != 1 or out.stride(1) != 1:
@@ -502,9 +552,9 @@ class CudaOps:
             raise KernelError(f"gemm: shapes x{tuple(x.shape)} w{tuple(w.shape)} out{tuple(out.shape)} do not match")
         if bias is not None:
             _check(bias, "bias", torch.float32, 1)
-            if bias.numel() != N:
+            if bias.numel() != (self.paired_rows(N) if gated else N):
                 raise KernelError("gemm: bias length does not match")
-        act_code = {"silu": 0, "gelu_pytorch_tanh": 1}[act]
+        act_code = self.GATED_ACTS[act]
         if self.tensor_core_ok(x, w, plan):
             if gated and M <= 128:
                 # few rows: the product is bound by streaming the weights, and a gated tile cannot split
@@ -513,11 +563,11 @@ class CudaOps:
                 parts = self.gemm_partials(x, w, plan=plan)
                 self._run("elementwise", "flint_gated_act", _ptr(parts), c_int(parts.shape[0]),
                           c_longlong(parts.stride(0)), _ptr(out), c_int(_code(out.dtype)), c_int(M), c_int(N),
-                          c_int(act_code), c_float(0.0), c_float(0.0))
+                          c_int(act_code), c_float(act_params[0]), c_float(act_params[1]), _ptr(bias))
                 return
-            self._gemm_tc(x, w, gated, out, bias, accumulate, act_code, plan, M, N, K, plan_ready)
+            self._gemm_tc(x, w, gated, out, bias, accumulate, act_code, plan, M, N, K, plan_ready, act_params)
         else:
-            self._gemm_simt(x, w, gated, out, bias, accumulate, act_code, plan, M, N, K)
+            self._gemm_simt(x, w, gated, out, bias, accumulate, act_code, plan, M, N, K, act_params)
 
     # bfloat16 x bfloat16 with 16-byte aligned rows goes to the tensor cores; everything else
     # (float32 operands: the true 32-bit path; odd K) to the float32 pipes
@@ -539,7 +589,7 @@ class CudaOps:
             return 64
         return self.token_tile(-(-top * n_tokens // n_experts))
 
-    def _gemm_tc(self, x, w, gated, out, bias, accumulate, act_code, plan, M, N, K, plan_ready=False):
+    def _gemm_tc(self, x, w, gated, out, bias, accumulate, act_code, plan, M, N, K, plan_ready=False, act_params=(0.0, 0.0)):
         if plan is not None:
             bn, splits, E = plan.tile_rows, 1, plan.n_experts
         else:
@@ -556,14 +606,14 @@ class CudaOps:
                   _ptr(plan.n_tiles if plan else None), _ptr(plan.offsets if plan else None),
                   c_int(plan.max_tiles if plan else 0), c_int(E), c_int(M), c_int(N), c_int(K), c_int(bn),
                   c_int(splits), _ptr(partial), c_int(0), c_int(0), c_int(1 if plan_ready and plan is not None else 0),
-                  _ptr(self.tc_error))
+                  _ptr(self.tc_error), c_float(act_params[0]), c_float(act_params[1]))
 
     @staticmethod
     def _product_label(N, K, plan, gated):
         """How a profile lists a product: its weight shape, and whether it is gated or over experts."""
         return f"{N}x{K}" + (" gated" if gated else "") + (" experts" if plan is not None else "")
 
-    def _gemm_simt(self, x, w, gated, out, bias, accumulate, act_code, plan, M, N, K):
+    def _gemm_simt(self, x, w, gated, out, bias, accumulate, act_code, plan, M, N, K, act_params=(0.0, 0.0)):
         if plan is not None and plan.tile_rows > 64:
             raise KernelError("gemm_simt: the plan's row tiles must not exceed 64 rows")
         self._label = self._product_label(N, K, plan, gated)
@@ -572,7 +622,8 @@ class CudaOps:
                   c_int(out.stride(0)), c_int(1 if accumulate else 0), c_int(act_code),
                   _ptr(plan.tile_expert if plan else None), _ptr(plan.tile_row0 if plan else None),
                   _ptr(plan.n_tiles if plan else None), _ptr(plan.offsets if plan else None),
-                  c_int(plan.max_tiles if plan else 0), c_int(plan.tile_rows if plan else 0), c_int(M), c_int(N), c_int(K))
+                  c_int(plan.max_tiles if plan else 0), c_int(plan.tile_rows if plan else 0), c_int(M), c_int(N), c_int(K),
+                  c_float(act_params[0]), c_float(act_params[1]))
 
     # ------------------------------------------------------------------ attention
     def attention_plan(self, T, nq, nkv, span, hd=128, bf16=True, ragged=True):
@@ -938,11 +989,12 @@ class CudaOps:
                   _ptr(out), c_int(_code(out.dtype)), c_int(T), c_int(H), c_int(V))
 
     # ------------------------------------------------------------------ state carried from token to token
-    def short_conv(self, u, col0, w, bias, act, pos, slot, state, y):
+    def short_conv(self, u, col0, w, bias, act, pos, slot, state, y, ring_rows=None):
         """y[t, c] = act(bias[c] + sum_j w[c, j] u[t - taps + 1 + j, col0 + c]) over the rows of each request, zeros
         before its start: u [T, >= col0 + C] float32 rows (a view; rows may be strided), w [C, taps], y [T, C] float32.
         ``state`` [slots, >= (taps - 1) C] float32 (a view of the slab's rows) holds each request's last taps - 1
-        inputs and is brought up to date.  act: "none" or "silu"."""
+        inputs and is brought up to date (``ring_rows``, default taps - 1: the rows of C inputs it has; the input at
+        position p lies in row p mod ring_rows).  act: "none" or "silu"."""
         _check(u, "u", torch.float32, 2, contiguous=False)
         _check(w, "w", torch.float32, 2)
         _check(y, "y", torch.float32, 2)
@@ -958,11 +1010,12 @@ class CudaOps:
             if state is None:
                 raise KernelError("short_conv: a convolution over time needs the requests' state")
             _check(state, "state", torch.float32, 2, contiguous=False)
-            if state.stride(1) != 1 or state.shape[1] < (taps - 1) * C:
+            if state.stride(1) != 1 or state.shape[1] < (ring_rows or taps - 1) * C:
                 raise KernelError("short_conv: the state's rows are too short")
         self._run("recurrent", "flint_short_conv", _ptr(u), c_longlong(u.stride(0)), c_int(col0), _ptr(w), _ptr(bias),
                   c_int(1 if act == "silu" else 0), _ptr(pos), _ptr(slot), _ptr(state),
-                  c_longlong(state.stride(0) if state is not None else 0), _ptr(y), c_int(T), c_int(C), c_int(taps))
+                  c_longlong(state.stride(0) if state is not None else 0), _ptr(y), c_int(T), c_int(C), c_int(taps),
+                  c_int(ring_rows or taps - 1))
         self.launches += 1 if taps > 1 else 0
 
     def delta_prepare(self, y, b, a, dt_bias, a_log, qk, decay, beta, H, G, D, unit_eps):
@@ -1232,9 +1285,10 @@ class CudaOps:
                   _ptr(decay), _ptr(dt), c_int(T), c_int(H), c_int(D))
 
     # ------------------------------------------------------------------ attention over a cached latent
-    def head_products(self, x, w, out):
+    def head_products(self, x, w, out, gate=None):
         """A small product per head: out[t, h, :] = w[h] @ x[t, h, :].  x [T, H, K], w [H, N, K], out [T, H, N]; x and
-        out may be views into wider rows (their last axis contiguous)."""
+        out may be views into wider rows (their last axis contiguous).  ``gate`` [S, T, H N] float32 (a view of partial
+        sums; out then is dense): out[t, h, n] is multiplied by sigmoid(sum of gate[:, t, h N + n])."""
         _check(x, "x", dims=3, contiguous=False)
         _check(out, "out", dims=3, contiguous=False)
         _check(w, "w", dims=3)
@@ -1244,14 +1298,22 @@ class CudaOps:
             raise KernelError(f"head_products: shapes x{tuple(x.shape)} w{tuple(w.shape)} out{tuple(out.shape)} do not match")
         if x.stride(2) != 1 or out.stride(2) != 1:
             raise KernelError("head_products: the last axis must be contiguous")
+        gate_args = (_ptr(None), c_int(0), c_longlong(0), c_longlong(0))
+        if gate is not None:
+            _check(gate, "gate", torch.float32, 3, contiguous=False)
+            if tuple(gate.shape[1:]) != (T, H * N) or gate.stride(2) != 1 or not out.is_contiguous():
+                raise KernelError("head_products: a gate needs partial sums [S, T, heads x outputs] and a dense output")
+            gate_args = (_ptr(gate), c_int(gate.shape[0]), c_longlong(gate.stride(0)), c_longlong(gate.stride(1)))
         if (x.dtype == w.dtype == out.dtype == torch.bfloat16 and K % 8 == 0 and x.stride(0) % 8 == 0 and x.stride(1) % 8 == 0
                 and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0):
             # all heads in one launch on the tensor cores
             return self._run("latent", "flint_head_products", _ptr(x), c_longlong(x.stride(0)), c_longlong(x.stride(1)),
                              _ptr(w), _ptr(out), c_longlong(out.stride(0)), c_longlong(out.stride(1)), c_int(T), c_int(H),
-                             c_int(N), c_int(K))
+                             c_int(N), c_int(K), *gate_args)
         for h in range(H):
             self.gemm(x[:, h, :], w[h], out[:, h, :])
+        if gate is not None:
+            self._run("latent", "flint_gate_rows", _ptr(out), c_int(_code(out.dtype)), *gate_args, c_int(T), c_int(H * N))
 
     def latent_prepare(self, proj, pos, slot, cos, sin, rot_dims, style, norm_w, eps, q_plain, qa, cache, H, D, R, C,
                        write_kv, status):
@@ -1291,6 +1353,37 @@ class CudaOps:
                   c_int(max_pages), c_int(P), c_int(T), c_int(H), c_int(D), c_int(R), c_int(C), c_int(row_w),
                   c_int(1 if write_kv else 0), _ptr(status))
 
+    def latent_down(self, proj, q_rank, q_norm, pos, slot, cos, sin, rot_dims, style, norm_w, eps, c_q, cache, R, C, write_kv,
+                    status):
+        """proj [S, T, W] float32 (partial sums, columns [q latent (q_rank) | latent (C) | rotated key part (R) | ...], or
+        [q latent | ...] without ``write_kv``): c_q [T, q_rank] = the q latent divided by its root mean square and
+        scaled by q_norm, and, with ``write_kv``, the token's cache row as in ``latent_prepare``."""
+        if style not in ("half", "interleaved"):
+            raise KernelError(f"latent_down: unknown rotation style {style!r}")
+        _check(proj, "proj", torch.float32, 3)
+        S, T, W = proj.shape
+        _check(c_q, "c_q", dims=2)
+        if tuple(c_q.shape) != (T, q_rank) or q_norm.dtype != torch.float32 or q_norm.numel() != q_rank:
+            raise KernelError("latent_down: the q latent's buffers do not match its size")
+        _check(cos, "cos", torch.float32, 2)
+        _check(sin, "sin", torch.float32, 2)
+        if rot_dims and cos.shape[1] * 2 != rot_dims:
+            raise KernelError("latent_down: table width must be rot_dims/2")
+        k = bt = None
+        cdt, P, max_pages, row_w = F32, 16, 0, 0
+        if write_kv:
+            k, bt, P = cache.k, cache.block_table, cache.page_size
+            cdt, max_pages, row_w = _code(k.dtype), bt.shape[1], k.shape[-1]
+            if tuple(k.shape[1:]) != (1, P, row_w) or row_w < C + R or row_w % 8:
+                raise KernelError(f"latent_down: cache pages are {tuple(k.shape[1:])}, expected (1, {P}, >= {C + R})")
+            if norm_w is None or norm_w.dtype != torch.float32 or norm_w.numel() != C:
+                raise KernelError("latent_down: the latent's norm scale must be float32 of the latent size")
+        self._run("latent", "flint_latent_down", _ptr(proj), c_int(S), c_longlong(proj.stride(0)), c_int(W), c_int(q_rank),
+                  _ptr(q_norm), _ptr(pos), _ptr(slot), _ptr(cos), _ptr(sin), c_int(rot_dims),
+                  c_int(1 if style == "interleaved" else 0), _ptr(norm_w), c_float(eps), _ptr(c_q), c_int(_code(c_q.dtype)),
+                  _ptr(k), c_int(cdt), _ptr(bt), c_int(max_pages), c_int(P), c_int(T), c_int(R), c_int(C), c_int(row_w),
+                  c_int(1 if write_kv else 0), _ptr(status))
+
     def latent_attention_plan(self, T, H, span):
         """(keys per split, splits) for the float32-pipe kernel: enough warps to fill the device, at least 64
         keys each."""
@@ -1299,11 +1392,11 @@ class CudaOps:
         keys = -(-(-(-max(span, 1) // n)) // 32) * 32
         return keys, -(-max(span, 1) // keys)
 
-    def latent_attention(self, qa, cache, step, out, H, C, window, scale, splits=None, rows=None, kernel=None):
+    def latent_attention(self, qa, cache, step, out, H, C, window, scale, splits=None, rows=None, kernel=None, sinks=None):
         """Every row's heads over its request's cached latent rows: qa [T, H, Dk] (key up-projection folded in)
         -> out [T, H, C], the probability-weighted sum of the latents (causal, ``window`` 0 = all keys).
         bfloat16 rows run on the tensor cores (``kernel`` "mma"), everything else, and a list of ``rows``, on the
-        float32 pipes ("simt")."""
+        float32 pipes ("simt").  ``sinks`` [H] float32: a logit per head that joins the softmax's denominator once."""
         _check(qa, "qa", dims=3)
         _check(out, "out", qa.dtype, 3)
         T, Dk = qa.shape[0], qa.shape[2]
@@ -1311,6 +1404,8 @@ class CudaOps:
         row_w = k.shape[-1]
         if qa.shape[1] != H or tuple(out.shape) != (T, H, C) or tuple(k.shape[1:]) != (1, P, row_w) or row_w < Dk:
             raise KernelError("latent_attention: shapes do not match")
+        if sinks is not None and (sinks.dtype != torch.float32 or sinks.numel() != H):
+            raise KernelError(f"latent_attention: sinks must be float32 [{H}]")
         span = min(step.max_kv_len, window) if window else step.max_kv_len
         mma_ok = qa.dtype == torch.bfloat16 and k.dtype == torch.bfloat16 and rows is None and C <= 512 and row_w <= 640
         if kernel is None:
@@ -1321,6 +1416,8 @@ class CudaOps:
             nh = min(H, 32)
             decode = T == len(getattr(step, "entries", ()))          # one token a request: a block per token
             nt = 1 if decode else max(1, 32 // nh)
+            if window:          # a block's tokens see a window each: between them nt - 1 keys more than one token
+                span = min(step.max_kv_len, window + nt - 1)
             if splits is None:
                 blocks = -(-T // nt) * -(-H // nh)
                 n = max(1, min(-(-max(span, 1) // 128), (2 * self.sm_count) // blocks))
@@ -1333,7 +1430,7 @@ class CudaOps:
             return self._run("latent", "flint_latent_attention_mma", _ptr(qa), _ptr(k), _ptr(cache.block_table),
                              c_int(cache.block_table.shape[1]), c_int(P), _ptr(step.pos), _ptr(step.slot), _ptr(out),
                              c_int(T), c_int(H), c_int(C), c_int(Dk), c_int(row_w), c_int(window), c_float(scale),
-                             c_int(nt), c_int(nh), c_int(keys), c_int(n), _ptr(scratch))
+                             c_int(nt), c_int(nh), c_int(keys), c_int(n), _ptr(scratch), _ptr(sinks))
         if kernel != "simt":
             raise KernelError(f"latent_attention: unknown kernel {kernel!r}")
         if rows is not None:
@@ -1346,7 +1443,81 @@ class CudaOps:
         self._run("latent", "flint_latent_attention", _ptr(qa), c_int(_code(qa.dtype)), _ptr(k), c_int(_code(k.dtype)),
                   _ptr(cache.block_table), c_int(cache.block_table.shape[1]), c_int(P), _ptr(step.pos), _ptr(step.slot),
                   _ptr(out), c_int(T), c_int(H), c_int(C), c_int(Dk), c_int(row_w), c_int(window), c_float(scale),
-                  c_int(keys), c_int(n), _ptr(scratch), _ptr(rows))
+                  c_int(keys), c_int(n), _ptr(scratch), _ptr(rows), _ptr(sinks))
+
+    # ------------------------------------------------------------------ real-gated linear recurrent unit
+    def rglru_gates(self, u, w_r, b_r, w_i, b_i, rate, a, b, kernel=None):
+        """u [T, W] float32; w_r, w_i [B, n, n] (out, in; W = B n); b_r, b_i, rate [W] float32: a = exp(rate r) and
+        b = sqrt(1 - a^2) i u with r, i = sigmoid(block-diagonal products of u + bias), a and b [T, W] float32.
+        bfloat16 blocks run on the tensor cores with u in three bfloat16 parts (``kernel`` "mma"), else on the
+        float32 pipes ("simt")."""
+        for name, t in (("u", u), ("a", a), ("b", b)):
+            _check(t, name, torch.float32, 2)
+        T, W = u.shape
+        _check(w_r, "w_r", dims=3)
+        _check(w_i, "w_i", w_r.dtype, 3)
+        B, n = w_r.shape[0], w_r.shape[1]
+        if tuple(w_r.shape) != (B, n, n) or w_i.shape != w_r.shape or B * n != W or a.shape != u.shape or b.shape != u.shape \
+                or any(t.dtype != torch.float32 or t.numel() != W for t in (b_r, b_i, rate)):
+            raise KernelError("rglru_gates: shapes do not match")
+        mma_ok = w_r.dtype == torch.bfloat16 and n % 8 == 0
+        kernel = kernel or ("mma" if mma_ok else "simt")
+        if kernel == "mma" and not mma_ok:
+            raise KernelError("rglru_gates: the tensor-core form takes bfloat16 blocks of a multiple of 8 channels")
+        self._run("rglru", "flint_rglru_gates", _ptr(u), _ptr(w_r), _ptr(b_r), _ptr(w_i), _ptr(b_i), c_int(_code(w_r.dtype)),
+                  _ptr(rate), _ptr(a), _ptr(b), c_int(T), c_int(W), c_int(B), c_int(1 if kernel == "mma" else 0))
+
+    def rglru_scan(self, a, b, y, slot, seq_start, n_seq, longest, state, out):
+        """Per channel S <- a S + b over every request's rows (request e owns rows seq_start[e] .. seq_start[e + 1] - 1;
+        ``seq_start`` None: row e alone; none owns more than ``longest``), from and into the first W numbers of
+        ``state``'s rows; out [T, W] = S gelu_tanh(y), y a [T, W] float32 view."""
+        _check(a, "a", torch.float32, 2)
+        _check(b, "b", torch.float32, 2)
+        _check(y, "y", torch.float32, 2, contiguous=False)
+        _check(state, "state", torch.float32, 2, contiguous=False)
+        _check(out, "out", dims=2)
+        T, W = a.shape
+        if b.shape != a.shape or tuple(y.shape) != (T, W) or y.stride(1) != 1 or state.shape[1] < W or state.stride(1) != 1 \
+                or out.shape != a.shape:
+            raise KernelError("rglru_scan: shapes do not match")
+        if seq_start is not None:
+            _check(seq_start, "seq_start", torch.int32, 1)
+            if seq_start.numel() != n_seq + 1:
+                raise KernelError("rglru_scan: seq_start must have one entry more than there are requests")
+        elif n_seq != T:
+            raise KernelError("rglru_scan: without seq_start every request brings one row")
+        chunk = self._fn("rglru", "flint_rglru_chunk")()
+        n = -(-int(longest) // chunk)
+        totals = torch.empty((n_seq, n + 1, 2, W), dtype=torch.float32, device=a.device) if n > 1 else None
+        self._run("rglru", "flint_rglru_scan", _ptr(a), _ptr(b), _ptr(y), c_longlong(y.stride(0)), _ptr(slot), _ptr(seq_start),
+                  c_int(n_seq), c_int(int(longest)), _ptr(state), c_longlong(state.stride(0)), _ptr(totals), _ptr(out),
+                  c_int(_code(out.dtype)), c_int(W))
+        self.launches += 1 if n > 1 else 0
+
+    RGLRU_STEP_BLOCK = 4096     # channels a diagonal block may have at most in the single-token kernel
+
+    def rglru_step(self, proj, bias, conv_w, conv_b, w_r, b_r, w_i, b_i, rate, pos, slot, state, out):
+        """The mixer from its projection to its output for a batch of single tokens (row e is request e): proj
+        [S, T, 2 W] float32 (partial sums of [y | x], ``bias`` [2 W] apart), conv_w [W, taps], conv_b [W], blocks as in
+        ``rglru_gates``; state's rows [S (W) | taps rows of the last inputs (the input at p in row p mod taps)] are
+        brought up to date; out [T, W]."""
+        _check(proj, "proj", torch.float32, 3)
+        S, T, W2 = proj.shape
+        W = W2 // 2
+        taps = conv_w.shape[1]
+        B, n = w_r.shape[0], w_r.shape[1]
+        _check(w_r, "w_r", dims=3)
+        _check(w_i, "w_i", w_r.dtype, 3)
+        _check(state, "state", torch.float32, 2, contiguous=False)
+        _check(out, "out", dims=2)
+        if B * n != W or w_i.shape != w_r.shape or tuple(conv_w.shape) != (W, taps) or bias.numel() != W2 \
+                or state.shape[1] < W * (1 + taps) or state.stride(1) != 1 or tuple(out.shape) != (T, W) \
+                or any(t.dtype != torch.float32 or t.numel() != W for t in (conv_b, b_r, b_i, rate)):
+            raise KernelError("rglru_step: shapes do not match")
+        self._run("rglru", "flint_rglru_step", _ptr(proj), c_int(S), c_longlong(proj.stride(0)), _ptr(bias), _ptr(conv_w),
+                  _ptr(conv_b), c_int(taps), _ptr(w_r), _ptr(b_r), _ptr(w_i), _ptr(b_i), c_int(_code(w_r.dtype)), _ptr(rate),
+                  _ptr(pos), _ptr(slot), _ptr(state), c_longlong(state.stride(0)), _ptr(out), c_int(_code(out.dtype)), c_int(T),
+                  c_int(W), c_int(B))
 
     # ------------------------------------------------------------------ additions to the embedded rows
     def pair_embed_add(self, ids, pos, slot, last, table, out, mul_prev, mul_cur, fed_rows=None, fed_from=None):
@@ -1385,10 +1556,10 @@ class CudaOps:
         if getattr(router, "rule", "") == "sigmoid":
             return self.router_sigmoid(x, router.weight, router.weight.shape[0] - router.extra, router.top, router.expert_ids,
                                        router.gates, router.weights, getattr(router, "logits", None))
-        if getattr(router, "rule", "") == "sigmoid_grouped":
+        if getattr(router, "rule", "") in ("sigmoid_grouped", "softmax_corrected"):
             return self.router_sigmoid_grouped(x, router.weight, router.correction, router.top, router.groups, router.keep,
                                                router.normalize, router.scale, router.expert_ids, router.gates,
-                                               getattr(router, "logits", None))
+                                               getattr(router, "logits", None), softmax=router.rule == "softmax_corrected")
         if int(getattr(router, "top", 0)) > 0:
             return self.router_topk(x, router.weight, router.top, router.groups, router.keep, router.scale,
                                     router.expert_ids, router.gates, getattr(router, "logits", None))
@@ -1438,8 +1609,8 @@ class CudaOps:
                   _ptr(expert_ids), _ptr(scores), _ptr(weights), _ptr(logits_out), c_int(T), c_int(H))
 
     def router_sigmoid_grouped(self, x, wr, correction, top, n_groups, keep, normalize, scale, expert_ids, gates,
-                               logits_out=None):
-        """Scores sigmoid(x wr^T) in float32; choice scores add ``correction`` [E] (or None); a group of neighbouring
+                               logits_out=None, softmax=False):
+        """Scores sigmoid(x wr^T), or with ``softmax`` softmax(x wr^T), in float32; choice scores add ``correction`` [E] (or None); a group of neighbouring
         experts scores as the sum of its two largest choice scores, only the ``keep`` best of ``n_groups`` groups may be
         chosen from, the ``top`` largest choice scores are (the lower index among equals); gates [T, top]: the chosen
         experts' scores, over their sum (+ 1e-20) if ``normalize``, times ``scale``."""
@@ -1455,8 +1626,8 @@ class CudaOps:
             raise KernelError("router_sigmoid_grouped: the correction must be float32, one per expert")
         if logits_out is not None:
             _check(logits_out, "logits_out", torch.float32, 2)
-        self._run("moe", "flint_router_sigmoid_grouped", _ptr(x), _ptr(wr), c_int(_code(wr.dtype)), _ptr(correction), c_int(E),
-                  c_int(top), c_int(n_groups), c_int(keep), c_int(1 if normalize else 0), c_float(scale), _ptr(expert_ids),
+        self._run("moe", "flint_router_sigmoid_grouped", _ptr(x), _ptr(wr), c_int(_code(wr.dtype)), _ptr(correction),
+                  c_int(1 if softmax else 0), c_int(E), c_int(top), c_int(n_groups), c_int(keep), c_int(1 if normalize else 0), c_float(scale), _ptr(expert_ids),
                   _ptr(gates), _ptr(logits_out), c_int(T), c_int(H))
 
     def _plan_buffers(self, expert_ids, n_experts, tile_rows):
@@ -1483,7 +1654,9 @@ class CudaOps:
 
     def moe_dispatch(self, expert_ids, n_experts, tile_rows, x):
         """The plan for these choices and the rows of x in its order: (plan, xs) with
-        xs[r] = x[plan.token_of[r]].  Few rows take one fused launch."""
+        xs[r] = x[plan.token_of[r]].  Few rows take one fused launch.  Choices from ``n_experts`` on name experts without
+        weights (identity): they take no row, plan.row_of gives them choices + token, and as many rows at the end of
+        xs belong to nobody."""
         _check(x, "x", dims=2)
         n = expert_ids.numel()
         xs = torch.empty((n, x.shape[1]), dtype=x.dtype, device=x.device)

@@ -2,8 +2,8 @@
 // the gated delta rule and of a state-space model with a scalar decay per head, and what surrounds them.
 //
 // Short convolution.  y[t, c] = act(b[c] + sum_j w[c, j] u[t - taps + 1 + j, c]) over the rows of one request, zeros
-// before its first position.  The inputs of earlier steps come from the request's state, taps - 1 rows: the input at
-// position p lives in state row p mod (taps - 1).  The convolution's kernel only reads the state; a second kernel,
+// before its first position.  The inputs of earlier steps come from the request's state, R >= taps - 1 rows: the input at
+// position p lives in state row p mod R.  The convolution's kernel only reads the state; a second kernel,
 // launched behind it, stores the inputs of every request's last taps - 1 rows of the step.  So every row of the batch
 // is worked independently, and no row of the state is read and written in one launch.
 //
@@ -41,11 +41,11 @@ __device__ __forceinline__ bool same_request(const int* pos, const int* slot, in
 __global__ void short_conv_kernel(const float* __restrict__ u, long long in_stride, int col0, const float* __restrict__ w,
                                   const float* __restrict__ bias, int act, const int* __restrict__ pos,
                                   const int* __restrict__ slot, const float* __restrict__ ring, long long ring_stride,
-                                  float* __restrict__ y, int T, int C, int taps) {
+                                  float* __restrict__ y, int T, int C, int taps, int R) {
   pdl_launch();
   pdl_wait();
   const int t = blockIdx.x;
-  const int p = pos[t], R = taps - 1;
+  const int p = pos[t];
   // how many of the taps - 1 earlier inputs are rows of this batch
   int have = 0;
   while (have < taps - 1 && same_request(pos, slot, t, have + 1, T)) ++have;
@@ -67,12 +67,12 @@ __global__ void short_conv_kernel(const float* __restrict__ u, long long in_stri
 // The inputs that outlive the step: a row that is among the last taps - 1 of its request's rows stores its input.
 __global__ void short_conv_keep_kernel(const float* __restrict__ u, long long in_stride, int col0,
                                        const int* __restrict__ pos, const int* __restrict__ slot, float* __restrict__ ring,
-                                       long long ring_stride, int T, int C, int taps) {
+                                       long long ring_stride, int T, int C, int taps, int R) {
   pdl_launch();
   pdl_wait();
   const int t = blockIdx.x;
   if (same_request(pos, slot, t, -(taps - 1), T)) return;
-  float* mine = ring + (size_t)slot[t] * ring_stride + (size_t)(pos[t] % (taps - 1)) * C;
+  float* mine = ring + (size_t)slot[t] * ring_stride + (size_t)(pos[t] % R) * C;
   const float* row = u + (size_t)t * in_stride + col0;
   for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < C; c += gridDim.y * blockDim.x) mine[c] = row[c];
 }
@@ -692,18 +692,19 @@ static int row_threads(int W) { return W >= 2048 ? 1024 : W >= 1024 ? 512 : W >=
 
 extern "C" int flint_short_conv(const float* u, long long in_stride, int col0, const float* w, const float* bias, int act,
                                 const int* pos, const int* slot, float* ring, long long ring_stride, float* y, int T,
-                                int C, int taps, cudaStream_t stream) {
+                                int C, int taps, int ring_rows, cudaStream_t stream) {
   if (T <= 0 || C <= 0) return 0;
+  if (ring_rows < taps - 1) return fail("short_conv: %d rows of state do not hold the last %d inputs", ring_rows, taps - 1);
   if (taps < 1 || taps > 64) return fail("short_conv: %d taps are not supported (1 to 64)", taps);
   if (taps > 1 && !ring) return fail("short_conv: a convolution over time needs the requests' state");
   // few rows (decoded tokens): a thread a channel, so that the rows spread over the chip; many rows: four channels a thread
   const int threads = C >= 1024 ? 256 : 128, per = T >= 256 ? 4 : 1;
   const dim3 grid((unsigned)T, (unsigned)min((C + threads * per - 1) / (threads * per), 65535));
   launch_pdl(short_conv_kernel, grid, dim3(threads), 0, stream, u, in_stride, col0, w, bias, act, pos, slot,
-             (const float*)ring, ring_stride, y, T, C, taps);
+             (const float*)ring, ring_stride, y, T, C, taps, ring_rows);
   if (taps > 1)
     launch_pdl(short_conv_keep_kernel, grid, dim3(threads), 0, stream, u, in_stride, col0, pos, slot, ring, ring_stride, T, C,
-               taps);
+               taps, ring_rows);
   return check_launch("short_conv");
 }
 

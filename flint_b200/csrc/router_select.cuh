@@ -129,18 +129,27 @@ __device__ __forceinline__ void select_sigmoid_by_warp(float* s, int lane, int E
   for (int e = lane; e < extra; e += 32) weights[top + e] = s[E + e];
 }
 
-// The choice of a sigmoid router limited to groups, by one warp, from float32 logits in shared memory: scores
-// s = sigmoid(logit); choice scores c = s + correction (a learned offset per expert, or none); the E experts form
+// The choice of a router with corrected choice scores, limited to groups, by one warp, from float32 logits in shared
+// memory: scores s = sigmoid(logit), or with `softmax` the softmax of the logits; choice scores c = s + correction (a learned offset per expert, or none); the E experts form
 // n_groups equal groups of neighbours and a group scores as the sum of its two largest choice scores (of its one,
 // if it has one member); only members of the `keep` best groups may be chosen (the others count as minus infinity:
 // choice scores may be negative); the `top` largest choice scores of those are chosen (the lower index among equals).
 // gates: the chosen experts' s, divided by their sum (+ 1e-20) if `normalize`, times out_scale.  `s` holds the logits
 // on entry and the scores afterwards; `c` is scratch for E floats in shared memory.
-__device__ __forceinline__ void select_sigmoid_grouped_by_warp(float* s, float* c, const float* __restrict__ correction,
-                                                               int lane, int E, int top, int n_groups, int keep,
-                                                               int normalize, float out_scale, int* ids, float* gates) {
+__device__ __forceinline__ void select_corrected_by_warp(float* s, float* c, const float* __restrict__ correction,
+                                                         bool softmax, int lane, int E, int top, int n_groups, int keep,
+                                                         int normalize, float out_scale, int* ids, float* gates) {
+  float m = 0.f, denom = 1.f;
+  if (softmax) {
+    m = -INFINITY;
+    for (int e = lane; e < E; e += 32) m = fmaxf(m, s[e]);
+    m = warp_max(m);
+    denom = 0.f;
+    for (int e = lane; e < E; e += 32) denom += expf(s[e] - m);
+    denom = warp_sum(denom);
+  }
   for (int e = lane; e < E; e += 32) {
-    const float v = 1.0f / (1.0f + expf(-s[e]));
+    const float v = softmax ? expf(s[e] - m) / denom : 1.0f / (1.0f + expf(-s[e]));
     s[e] = v;
     c[e] = correction ? v + correction[e] : v;
   }

@@ -6,6 +6,12 @@
 //   x[row] += g0 * y[r0] + g1 * y[r1]                 (the two selected experts' outputs)
 //   y = LayerNorm(x[row]) or RMSNorm(x[row])          float32 statistics, two passes over registers
 //   out_f32 / out_bf16 <- y
+//
+// With several streams a row [S, H] is kept instead of x[row] [H]: with r what is pending (the two additions above),
+//
+//   x_t[row] <- sum_s mix[s, t] x_s[row] + out[t] r       (all t from the old streams; only with something pending)
+//   y = norm(sum_s gather[s] x_s[row])
+//
 //   logits_e = <y, Wr[e]>, sparsemixer top-2          (float32; same selection as moe.cu)
 //
 // Fusing these saves, per layer of a decode step, the kernels that would only add to the
@@ -22,6 +28,8 @@ using namespace flint;
 namespace {
 constexpr int MAX_VPT = 4;
 constexpr int MAX_E = 256;
+constexpr int FUSED_STREAMS = 4;         // streams the row kernel takes (their columns are held in registers)
+constexpr int MAX_STREAMS = 16;          // streams the update kernel takes
 
 struct RowArgs {
   float* x;
@@ -33,8 +41,11 @@ struct RowArgs {
   const void* wr; int E; float jitter_eps; int* expert_ids; float* gates;
   int top, n_groups, keep; float out_scale;      // top > 0: the softmax router limited to groups instead of sparsemixer
   int rule, extra; float* aux;  // rule 1: the sigmoid router (scores into gates, the last `extra` rows of wr are gates: aux)
-  const float* correction; int normalize;   // rule 2: the sigmoid router limited to groups (select_sigmoid_grouped_by_warp)
+  const float* correction; int normalize;   // rule 2: the sigmoid router limited to groups (select_corrected_by_warp); rule 3: the same over a softmax
   float* router_logits;        // optional [rows, E]: the logits the selection was made from (for tests)
+  int n_streams;               // > 0: x is [rows, n_streams, H]; the mixing weights of what is pending, of the norm's input
+  const float* mix; const float* spread; const float* gather;
+  int store;                   // streams: whether the new streams are written back
   int H;
 };
 
@@ -56,6 +67,46 @@ __device__ __forceinline__ void load_w8(const __nv_bfloat16* p, float* f) {
     f[2 * i] = __uint_as_float(w[i] << 16);
     f[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
   }
+}
+
+// The mixing weights of a kernel's streams, staged in shared memory (they are weights: no kernel writes them).
+template <int ST>
+struct StreamWeights { float mix[ST > 0 ? ST * ST : 1], spread[ST > 0 ? ST : 1], gather[ST > 0 ? ST : 1]; };
+
+template <int ST>
+__device__ __forceinline__ void load_stream_weights(StreamWeights<ST>& w, const RowArgs& a) {
+  for (int i = threadIdx.x; i < a.n_streams * a.n_streams; i += blockDim.x) w.mix[i] = a.mix ? a.mix[i] : 0.f;
+  for (int i = threadIdx.x; i < a.n_streams; i += blockDim.x) {
+    w.spread[i] = a.spread ? a.spread[i] : 0.f;
+    w.gather[i] = a.gather ? a.gather[i] : 0.f;
+  }
+}
+
+// Four neighbouring columns of one row's streams: bring them up to date with what is pending (r), store them, and
+// return the norm's input.  xr: the row's first stream, at the columns.
+template <int ST>
+__device__ __forceinline__ float4 stream_columns(float* xr, const float4 r, const StreamWeights<ST>& w, const RowArgs& a,
+                                                 bool pending) {
+  float4 x[ST > 0 ? ST : 1];
+  const int n = a.n_streams;
+#pragma unroll
+  for (int s = 0; s < ST; ++s) x[s] = s < n ? ld4(xr + (size_t)s * a.H) : make_float4(0.f, 0.f, 0.f, 0.f);
+  float4 u = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int t = 0; t < ST; ++t) {
+    if (t >= n) break;
+    float4 v = x[t];
+    if (pending) {
+      v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+      for (int s = 0; s < ST; ++s)
+        if (s < n) fma4(v, w.mix[s * n + t], x[s]);
+      fma4(v, w.spread[t], r);
+      if (a.store) *reinterpret_cast<float4*>(xr + (size_t)t * a.H) = v;
+    }
+    fma4(u, w.gather[t], v);
+  }
+  return u;
 }
 
 // sparsemixer top-2 of one row (float32; same selection as moe.cu).  Up to 32 experts sit one per lane of a
@@ -108,23 +159,29 @@ __device__ __forceinline__ void select_two_serial(const float* s, int E, float j
 }
 
 // One block per row; a thread holds VPT vectors of four values of its row.
-template <int VPT, typename TW>
+// ST: 0 for a plain residual row, else the most streams this form takes.
+template <int VPT, typename TW, int ST>
 __global__ void __launch_bounds__(1024)
 row_norm_kernel(const __grid_constant__ RowArgs a) {
   extern __shared__ float smem[];          // router only: H floats of the normalised row, then partial logits
   __shared__ float red[32];
+  __shared__ StreamWeights<ST> hw;
   pdl_launch();
+  if constexpr (ST > 0) {
+    load_stream_weights<ST>(hw, a);
+    __syncthreads();
+  }
   pdl_wait();
   const int H = a.H, n4 = H >> 2;
   {
     const int r = blockIdx.x;
     const int src = a.row_index ? a.row_index[r] : r;
-    float* xr = a.x + (size_t)src * H;
+    float* xr = a.x + (size_t)src * (ST > 0 ? a.n_streams : 1) * H;
     float4 v[VPT];
 #pragma unroll
     for (int i = 0; i < VPT; ++i) {
       const int c = threadIdx.x + i * blockDim.x;
-      v[i] = c < n4 ? ld4(xr + 4 * c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      v[i] = ST == 0 && c < n4 ? ld4(xr + 4 * c) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
     const bool pending = a.partials || a.comb_y;
     if (a.partials) {
@@ -170,7 +227,13 @@ row_norm_kernel(const __grid_constant__ RowArgs a) {
 #pragma unroll
       for (int i = 0; i < VPT; ++i) add4(v[i], t[i]);
     }
-    if (pending) {
+    if constexpr (ST > 0) {
+#pragma unroll
+      for (int i = 0; i < VPT; ++i) {
+        const int c = threadIdx.x + i * blockDim.x;
+        if (c < n4) v[i] = stream_columns<ST>(xr + 4 * c, v[i], hw, a, pending);
+      }
+    } else if (pending) {
 #pragma unroll
       for (int i = 0; i < VPT; ++i) {
         const int c = threadIdx.x + i * blockDim.x;
@@ -281,8 +344,8 @@ row_norm_kernel(const __grid_constant__ RowArgs a) {
       if (a.router_logits) a.router_logits[(size_t)r * E + e] = t;
     }
     __syncwarp();
-    if (a.rule == 2)
-      select_sigmoid_grouped_by_warp(s, s + E, a.correction, lane, E, a.top, a.n_groups, a.keep, a.normalize, a.out_scale,
+    if (a.rule >= 2)
+      select_corrected_by_warp(s, s + E, a.correction, a.rule == 3, lane, E, a.top, a.n_groups, a.keep, a.normalize, a.out_scale,
                                      a.expert_ids + (size_t)a.top * r, a.gates + (size_t)a.top * r);
     else if (a.rule == 1)
       select_sigmoid_by_warp(s, lane, E - a.extra, a.extra, a.top, a.expert_ids + (size_t)a.top * r,
@@ -352,11 +415,12 @@ __device__ __forceinline__ float cluster_sum(float block_value, float* slots, ui
   return t;
 }
 
-template <int VPT, typename TW>
+template <int VPT, typename TW, int ST>
 __global__ void __launch_bounds__(256)
 row_norm_cluster_kernel(const __grid_constant__ RowArgs a, const int vec_per_block) {
   extern __shared__ float smem[];          // router only: this block's columns of the normalised row, partial logits
   __shared__ float red[32];
+  __shared__ StreamWeights<ST> hw;
   __shared__ float sum_slots[MAX_CL], sq_slots[MAX_CL];
   const uint32_t rank = cluster_rank(), CL = cluster_blocks();
   const int H = a.H, n4 = H >> 2;
@@ -378,13 +442,14 @@ row_norm_cluster_kernel(const __grid_constant__ RowArgs a, const int vec_per_blo
     b[i] = (a.gamma && a.beta && ok[i]) ? ld4(a.beta + 4 * col[i]) : make_float4(0.f, 0.f, 0.f, 0.f);
   }
   pdl_launch();
+  if constexpr (ST > 0) load_stream_weights<ST>(hw, a);
   cluster_barrier();        // every block of the cluster runs before any of them writes into another's memory
   pdl_wait();
   const int src = a.row_index ? a.row_index[r] : r;
-  float* xr = a.x + (size_t)src * H;
+  float* xr = a.x + (size_t)src * (ST > 0 ? a.n_streams : 1) * H;
   float4 v[VPT];
 #pragma unroll
-  for (int i = 0; i < VPT; ++i) v[i] = ok[i] ? ld4(xr + 4 * col[i]) : make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int i = 0; i < VPT; ++i) v[i] = ST == 0 && ok[i] ? ld4(xr + 4 * col[i]) : make_float4(0.f, 0.f, 0.f, 0.f);
   const bool pending = a.partials || a.comb_y;
   if (a.partials) {
     const float* pr = a.partials + (size_t)src * H;
@@ -419,7 +484,11 @@ row_norm_cluster_kernel(const __grid_constant__ RowArgs a, const int vec_per_blo
     for (int i = 0; i < VPT; ++i)
       if (ok[i]) add4(v[i], t[i]);
   }
-  if (pending) {
+  if constexpr (ST > 0) {
+#pragma unroll
+    for (int i = 0; i < VPT; ++i)
+      if (ok[i]) v[i] = stream_columns<ST>(xr + 4 * col[i], v[i], hw, a, pending);
+  } else if (pending) {
 #pragma unroll
     for (int i = 0; i < VPT; ++i)
       if (ok[i]) *reinterpret_cast<float4*>(xr + 4 * col[i]) = v[i];
@@ -531,8 +600,8 @@ row_norm_cluster_kernel(const __grid_constant__ RowArgs a, const int vec_per_blo
       if (a.router_logits) a.router_logits[(size_t)r * E + e] = t;
     }
     __syncwarp();
-    if (a.rule == 2)
-      select_sigmoid_grouped_by_warp(s, s + E, a.correction, lane, E, a.top, a.n_groups, a.keep, a.normalize, a.out_scale,
+    if (a.rule >= 2)
+      select_corrected_by_warp(s, s + E, a.correction, a.rule == 3, lane, E, a.top, a.n_groups, a.keep, a.normalize, a.out_scale,
                                      a.expert_ids + (size_t)a.top * r, a.gates + (size_t)a.top * r);
     else if (a.rule == 1)
       select_sigmoid_by_warp(s, lane, E - a.extra, a.extra, a.top, a.expert_ids + (size_t)a.top * r,
@@ -562,22 +631,22 @@ row_norm_cluster_kernel(const __grid_constant__ RowArgs a, const int vec_per_blo
   select_two_serial(s, E, a.jitter_eps, a.expert_ids + 2 * r, a.gates + 2 * r);
 }
 
-template <int VPT, typename TW>
+template <int VPT, typename TW, int ST>
 int launch_row(const RowArgs& a, int rows, int threads, size_t smem, cudaStream_t stream) {
   if (smem > 48 * 1024) {
     static bool configured = false;   // per instantiation
     if (!configured) {
-      cudaError_t e = cudaFuncSetAttribute(row_norm_kernel<VPT, TW>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+      cudaError_t e = cudaFuncSetAttribute(row_norm_kernel<VPT, TW, ST>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                            200 * 1024);
       if (e != cudaSuccess) return fail("row_norm: cannot raise shared memory: %s", cudaGetErrorString(e));
       configured = true;
     }
   }
-  launch_pdl(row_norm_kernel<VPT, TW>, dim3(rows), dim3(threads), smem, stream, a);
+  launch_pdl(row_norm_kernel<VPT, TW, ST>, dim3(rows), dim3(threads), smem, stream, a);
   return check_launch("row_norm");
 }
 
-template <int VPT, typename TW>
+template <int VPT, typename TW, int ST>
 int launch_row_cluster(const RowArgs& a, int rows, int cl, int vec_per_block, int threads, size_t smem, cudaStream_t stream) {
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3(rows * cl);
@@ -593,8 +662,44 @@ int launch_row_cluster(const RowArgs& a, int rows, int cl, int vec_per_block, in
   attr[1].val.clusterDim.z = 1;
   cfg.attrs = attr;
   cfg.numAttrs = 2;
-  cudaLaunchKernelEx(&cfg, row_norm_cluster_kernel<VPT, TW>, a, vec_per_block);
+  cudaLaunchKernelEx(&cfg, row_norm_cluster_kernel<VPT, TW, ST>, a, vec_per_block);
   return check_launch("row_norm (cluster)");
+}
+
+// Streams of any width: x brought up to date with what is pending (if it names mixing weights), u [rows, H] (or null) the
+// sum of the streams weighted by gather.  One block per row.
+__global__ void stream_update_kernel(const __grid_constant__ RowArgs a, float* __restrict__ u) {
+  __shared__ StreamWeights<MAX_STREAMS> w;
+  pdl_launch();
+  load_stream_weights<MAX_STREAMS>(w, a);
+  __syncthreads();
+  pdl_wait();
+  const int src = a.row_index ? a.row_index[blockIdx.x] : blockIdx.x;
+  const int H = a.H, n = a.n_streams;
+  const bool pending = a.partials || a.comb_y;
+  float* xr = a.x + (size_t)src * n * H;
+  for (int c = threadIdx.x; c < H; c += blockDim.x) {
+    float r = 0.f;
+    for (int z = 0; z < a.n_partials; ++z) r += a.partials[(size_t)z * a.partial_stride + (size_t)src * H + c];
+    if (a.add_bias) r += a.add_bias[c];
+    float e = 0.f;
+    for (int k = 0; k < a.comb_top; ++k)
+      e = fmaf(a.comb_gates[(size_t)a.comb_top * src + k], a.comb_y[(size_t)a.comb_row_of[(size_t)a.comb_top * src + k] * H + c], e);
+    r += e;
+    float x[MAX_STREAMS], g = 0.f;
+    for (int s = 0; s < n; ++s) x[s] = xr[(size_t)s * H + c];
+    for (int t = 0; t < n; ++t) {
+      float v = x[t];
+      if (pending) {
+        v = 0.f;
+        for (int s = 0; s < n; ++s) v = fmaf(w.mix[s * n + t], x[s], v);
+        v = fmaf(w.spread[t], r, v);
+        if (a.store) xr[(size_t)t * H + c] = v;
+      }
+      g = fmaf(w.gather[t], v, g);
+    }
+    if (u) u[(size_t)blockIdx.x * H + c] = g;
+  }
 }
 
 int g_cluster_rows = 16;      // up to this many rows a cluster of blocks shares each row; 0: never
@@ -618,7 +723,10 @@ extern "C" int flint_row_norm_set_cluster_rows(int rows) {
 // always-on parts, and aux [rows, top + extra] gets 1 for the chosen experts and those rows' sigmoids.  rule 2: a sigmoid
 // router limited to groups: choice scores sigmoid + correction [E] (or NULL), a group scores as the sum of its two
 // largest, `top` experts of the `keep` best of `n_groups` groups; gates the chosen sigmoids, over their sum if
-// `normalize`, times out_scale.
+// `normalize`, times out_scale.  rule 3: the same with softmax scores.
+// n_streams > 0: x is [T, n_streams, H]; what is pending goes into the streams by mix [n_streams, n_streams] ([from, to])
+// and spread [n_streams], and the norm reads their sum weighted by gather [n_streams].  With row_index the streams are
+// brought up to date for the norm only, not in memory.
 extern "C" int flint_row_norm(float* x, const int* row_index, int rows, int H, const float* partials,
                               int n_partials, long long partial_stride, const float* add_bias,
                               const float* comb_y, const int* comb_row_of, const float* comb_gates, int comb_top,
@@ -626,6 +734,7 @@ extern "C" int flint_row_norm(float* x, const int* row_index, int rows, int H, c
                               void* out_bf16, const void* wr, int w_dtype, int E, float jitter_eps,
                               int* expert_ids, float* gates, float* router_logits, int top, int n_groups, int keep,
                               float out_scale, int rule, int extra, float* aux, const float* correction, int normalize,
+                              int n_streams, const float* mix, const float* spread, const float* gather,
                               cudaStream_t stream) {
   if (rows <= 0) return 0;
   if (H <= 0 || (H & 3) || H > 4 * 1024 * MAX_VPT) return fail("row_norm: width %d (multiples of 4 up to %d)", H, 4096 * MAX_VPT);
@@ -636,16 +745,20 @@ extern "C" int flint_row_norm(float* x, const int* row_index, int rows, int H, c
   if (wr && rule == 1) {
     if (top < 1 || top > ROUTER_MAX_TOP || extra < 0 || top > E - extra || !aux)
       return fail("row_norm: a sigmoid router choosing %d of %d experts (%d gate rows) is not supported", top, E - extra, extra);
-  } else if (wr && rule != 0 && rule != 2) {
+  } else if (wr && rule != 0 && rule != 2 && rule != 3) {
     return fail("row_norm: unknown router rule %d", rule);
-  } else if (wr && rule == 2 && (top < 1 || 2 * E > H)) {
-    return fail("row_norm: the grouped sigmoid router needs top >= 1 and rows of at least twice the %d experts", E);
+  } else if (wr && rule >= 2 && (top < 1 || 2 * E > H)) {
+    return fail("row_norm: a router with corrected choice scores needs top >= 1 and rows of at least twice the %d experts", E);
   } else if (wr && top > 0 && (top > ROUTER_MAX_TOP || top > E || n_groups < 1 || n_groups > 64 || E % n_groups || keep < 1 ||
                         keep > n_groups || keep * (E / n_groups) < top))
     return fail("row_norm: %d of %d experts from %d of %d groups is not supported", top, E, keep, n_groups);
   if (wr && (row_index || !gamma || !expert_ids || !gates)) return fail("row_norm: the router needs a norm and all rows");
   if (wr && (((uintptr_t)wr & 15) != 0)) return fail("row_norm: router weights must be 16-byte aligned");
+  if (n_streams < 0 || n_streams > FUSED_STREAMS) return fail("row_norm: %d streams (up to %d)", n_streams, FUSED_STREAMS);
+  if (n_streams && (partials || comb_y) && (!mix || !spread)) return fail("row_norm: what is pending needs the streams' mixing weights");
+  if (n_streams && gamma && !gather) return fail("row_norm: the norm of several streams needs their weights");
   RowArgs a;
+  a.n_streams = n_streams; a.mix = mix; a.spread = spread; a.gather = gather; a.store = row_index == nullptr;
   a.x = x; a.row_index = row_index;
   a.partials = partials; a.n_partials = n_partials; a.partial_stride = partial_stride; a.add_bias = add_bias;
   a.comb_y = comb_y; a.comb_row_of = comb_row_of; a.comb_gates = comb_gates; a.comb_top = comb_top;
@@ -672,19 +785,22 @@ extern "C" int flint_row_norm(float* x, const int* row_index, int rows, int H, c
     const int k = wr ? (n_warps >= groups ? n_warps / groups : 1) : 0;
     const size_t smem = wr ? (size_t)(4 * vec_per_block + E * k + MAX_CL * E + 2 * E) * sizeof(float) : 0;
     if (smem <= 48 * 1024 && vpt <= MAX_VPT) {
-#define GOC(V) (wr && w_dtype == FLINT_BF16 ? launch_row_cluster<V, __nv_bfloat16>(a, rows, cl, vec_per_block, threads, smem, stream) \
-                                            : launch_row_cluster<V, float>(a, rows, cl, vec_per_block, threads, smem, stream))
+#define GOCS(V, S) (wr && w_dtype == FLINT_BF16 ? launch_row_cluster<V, __nv_bfloat16, S>(a, rows, cl, vec_per_block, threads, smem, stream) \
+                                                : launch_row_cluster<V, float, S>(a, rows, cl, vec_per_block, threads, smem, stream))
+#define GOC(V) (n_streams ? GOCS(V, FUSED_STREAMS) : GOCS(V, 0))
       switch (vpt) {
         case 1: return GOC(1);
         case 2: return GOC(2);
         default: return GOC(4);
       }
 #undef GOC
+#undef GOCS
     }
   }
   // few rows: a wide block per row (more warps share the router's rows); many rows: narrow blocks
   // with four vectors per thread, so that several blocks fit an SM and hide each other's latency
   int threads = rows < 148 ? ((n4 + 31) / 32) * 32 : ((n4 / 4 + 31) / 32) * 32;
+  if (n_streams && rows >= 148) threads = ((n4 + 31) / 32) * 32;      // the streams' columns already are several loads a thread
   if (threads > 1024) threads = 1024;
   if (threads < 32) threads = 32;
   if (wr && threads < 128) threads = 128;               // a few warps for the router's dot products
@@ -693,8 +809,9 @@ extern "C" int flint_row_norm(float* x, const int* row_index, int rows, int H, c
   const int groups = (E + 3) / 4;
   const int k = wr ? (n_warps >= groups ? n_warps / groups : 1) : 0;
   const size_t smem = wr ? (size_t)(H + E * k) * sizeof(float) : 0;
-#define GO(V) (wr && w_dtype == FLINT_BF16 ? launch_row<V, __nv_bfloat16>(a, rows, threads, smem, stream) \
-                                           : launch_row<V, float>(a, rows, threads, smem, stream))
+#define GOS(V, S) (wr && w_dtype == FLINT_BF16 ? launch_row<V, __nv_bfloat16, S>(a, rows, threads, smem, stream) \
+                                               : launch_row<V, float, S>(a, rows, threads, smem, stream))
+#define GO(V) (n_streams ? GOS(V, FUSED_STREAMS) : GOS(V, 0))
   if (smem > 200 * 1024) return fail("row_norm: width %d is too large for the fused router", H);
   switch (vpt) {
     case 1: return GO(1);
@@ -703,6 +820,28 @@ extern "C" int flint_row_norm(float* x, const int* row_index, int rows, int H, c
     default: return fail("row_norm: width %d is too large", H);
   }
 #undef GO
+#undef GOS
+}
+
+// The streams' part of flint_row_norm as a kernel of its own, for widths and numbers of streams that one does not take: x [T, n_streams, H]
+// updated in place (not with row_index), u [rows, H] the norm's input (or null).
+extern "C" int flint_stream_update(float* x, const int* row_index, int rows, int H, const float* partials, int n_partials,
+                                   long long partial_stride, const float* add_bias, const float* comb_y,
+                                   const int* comb_row_of, const float* comb_gates, int comb_top, int n_streams,
+                                   const float* mix, const float* spread, const float* gather, float* u,
+                                   cudaStream_t stream) {
+  if (rows <= 0) return 0;
+  if (n_streams < 1 || n_streams > MAX_STREAMS) return fail("stream_update: %d streams (up to %d)", n_streams, MAX_STREAMS);
+  if ((partials || comb_y) && (!mix || !spread)) return fail("stream_update: what is pending needs the streams' mixing weights");
+  if (u && !gather) return fail("stream_update: the sum of the streams needs their weights");
+  if (comb_y && comb_top < 1) return fail("stream_update: %d expert rows a token", comb_top);
+  RowArgs a = {};
+  a.x = x; a.row_index = row_index; a.H = H;
+  a.partials = partials; a.n_partials = partials ? n_partials : 0; a.partial_stride = partial_stride; a.add_bias = partials ? add_bias : nullptr;
+  a.comb_y = comb_y; a.comb_row_of = comb_row_of; a.comb_gates = comb_gates; a.comb_top = comb_y ? comb_top : 0;
+  a.n_streams = n_streams; a.mix = mix; a.spread = spread; a.gather = gather; a.store = row_index == nullptr;
+  launch_pdl(stream_update_kernel, dim3(rows), dim3(H >= 512 ? 256 : 128), 0, stream, a, u);
+  return check_launch("stream_update");
 }
 
 extern "C" const char* flint_row_fused_last_error() { return g_error; }

@@ -22,7 +22,7 @@ from ..config.spec import ModelSpec
 from ..errors import ConfigError, ModelError
 from ..parts.base import BuildContext, matmul_dtype
 from ..parts.block import run_norm
-from ..registry import ARCHITECTURES, BLOCKS, EMBED_ADDITIONS, FEED_FORWARDS, MIXERS, NORMS, POSITION_ENCODINGS
+from ..registry import ARCHITECTURES, BLOCKS, EMBED_ADDITIONS, FEED_FORWARDS, MIXERS, NORMS, POSITION_ENCODINGS, STREAM_MIXES
 from ..weights.loader import load_tensors
 from ..weights.sources import RenamedSource, SafetensorsSource, WeightSpec
 from .step import StepEntry, StepStaging
@@ -34,6 +34,8 @@ def registry_for_role(role: str):
         return MIXERS
     if role.startswith("ffn"):
         return FEED_FORWARDS
+    if role.startswith("hc"):
+        return STREAM_MIXES
     raise ConfigError(f"no part registry for role {role!r}")
 
 
@@ -146,6 +148,11 @@ class Model:
             raise ConfigError(f"max_context {self.max_context} exceeds the model's {spec.max_positions} positions")
         self.ctx = BuildContext(ops=ops, device=self.device, compute=dtype, max_context=self.max_context)
         self.layers = [Layer(ls, self.ctx) for ls in spec.layers]
+        if spec.streams and (spec.embed_norm is not None or spec.depth_mix or spec.pass_inputs or spec.embed_additions
+                             or spec.embed_position is not None):
+            raise ConfigError("a model with several residual streams adds nothing else to its embedded rows")
+        # what the final norm reads of several streams: their plain sum
+        self.stream_sum = torch.ones(spec.streams, dtype=torch.float32, device=self.device) if spec.streams else None
         self.final_norm = NORMS.get(spec.final_norm.kind)(spec.final_norm.params, self.ctx)
         self.embed_position = None
         if spec.embed_position is not None:
@@ -319,11 +326,13 @@ class Model:
     def forward(self, step) -> torch.Tensor:
         ops, spec = self.ops, self.spec
         T = step.n_tokens
-        h = torch.empty((T, spec.hidden_size), dtype=torch.float32, device=self.device)
+        shape = (T, spec.streams, spec.hidden_size) if spec.streams else (T, spec.hidden_size)
+        h = torch.empty(shape, dtype=torch.float32, device=self.device)
+        many = {"copies": spec.streams} if spec.streams else {}
         if self.fed_from is not None:
-            ops.embed(step.ids, self.embed_table, h, spec.embed_scale, fed_rows=step.fed_rows, fed_from=self.fed_from)
+            ops.embed(step.ids, self.embed_table, h, spec.embed_scale, fed_rows=step.fed_rows, fed_from=self.fed_from, **many)
         else:
-            ops.embed(step.ids, self.embed_table, h, spec.embed_scale)
+            ops.embed(step.ids, self.embed_table, h, spec.embed_scale, **many)
         if self.embed_position is not None:
             self.embed_position.after_embedding(h, step)
         for k, (part, _) in enumerate(self.embed_additions):
@@ -365,8 +374,11 @@ class Model:
             owner = i if call.cache_of is None else call.cache_of
             carry = layer.block.forward(h, step, self.cache.view(owner), self.cache.state_of(i),
                                         writes_cache=call.cache_of is None, carry=carry)
+            if step.record is not None and spec.streams and carry is not None:
+                ops.apply_pending(h, carry)       # a test asked for what every call leaves: the streams are finished here
+                carry = None
             if step.record is not None and carry is None and history is None:
-                step.record.setdefault("rows_after", []).append(h.clone())      # the rows as this call leaves them
+                step.record.setdefault("rows_after", []).append(h.sum(1) if spec.streams else h.clone())
             if history is not None:
                 if carry is not None:
                     ops.apply_pending(h, carry)
@@ -381,7 +393,7 @@ class Model:
         logits = torch.empty((R, spec.vocab_size), dtype=torch.float32, device=self.device)
         if R:
             wdt = self.head_weight.dtype
-            x, _ = run_norm(self.final_norm, h, (wdt,), carry, row_index=step.want_rows)
+            x, _ = run_norm(self.final_norm, h, (wdt,), carry, row_index=step.want_rows, gather=self.stream_sum)
             ops.gemm(x[wdt], self.head_weight, logits, bias=self.head_bias)
             if spec.logit_softcap:
                 ops.softcap(logits, spec.logit_softcap)

@@ -9,7 +9,8 @@ crates/thuban_model/src/ops/*.rs).
 Interfaces
 ----------
 Norm          ``forward(x, want, row_index=None, pending=None, router=None) -> {dtype: tensor}``
-              x is the float32 residual stream [T, H]; ``want`` is the set of element
+              x is the float32 residual stream [T, H] (or, with ``gather``, several streams [T, S, H] whose weighted
+              sum is normed); ``want`` is the set of element
               types the next part asked for.  A norm with ``supports_pending`` applies a
               ``Pending`` addition to x first; one with ``supports_router`` can fill a
               ``RouterRequest``.  Both are optional abilities; the block works without them.
@@ -26,6 +27,8 @@ PositionEncoding  ``rotary_dim``, ``style`` ("half": dims i and i + rotary_dim/2
               ``ModelSpec.embed_position`` instead has ``after_embedding(h, step)`` and adds to the embedded rows.
 Block         ``forward(residual, step, cache, state, writes_cache)``: the arrangement of
               the parts of one layer.
+StreamMix     ``weights()``, ``gather`` [S], ``mix`` [S, S] and ``spread`` [S] float32: how a part of a layer with several
+              residual streams reads them and how what it adds goes into them.
 EmbedAddition ``weights()``, ``state_spec()`` (per-request state, or None), ``forward(h, step, state)``: adds to the
               embedded rows h [T, H] in place (a table row chosen by the token and its predecessor, and the like).
 """
@@ -44,12 +47,16 @@ class Pending:
     kernel applies it while it reads the row anyway (or ``ops.apply_pending`` does, for a norm
     that cannot).  Either partial sums of a product whose K range was split
     (``partials`` [S, T, H] float32, plus an optional ``bias`` [H]), or the selected experts'
-    outputs (``y`` [kT, H] with ``row_of`` [T, k] and ``gates`` [T, k], k choices a token), or both."""
+    outputs (``y`` [kT, H] with ``row_of`` [T, k] and ``gates`` [T, k], k choices a token), or both.  For a residual of
+    several streams ``mix`` [S, S] ([from, to]) and ``spread`` [S] say how it goes into them: with r the addition,
+    x_t <- sum_s mix[s, t] x_s + spread[t] r for all t at once."""
     partials: torch.Tensor | None = None
     bias: torch.Tensor | None = None
     y: torch.Tensor | None = None
     row_of: torch.Tensor | None = None
     gates: torch.Tensor | None = None
+    mix: torch.Tensor | None = None
+    spread: torch.Tensor | None = None
 
 
 @dataclass
@@ -63,8 +70,10 @@ class RouterRequest:
     and ``weights`` [T, top + extra] gets 1 for every chosen expert and those rows' sigmoids.  With ``rule``
     "sigmoid_grouped": choice scores sigmoid(logit) + ``correction`` [E] (or None), a group of neighbouring experts scores
     as the sum of its two largest choice scores, ``top`` experts of the ``keep`` best of ``groups`` groups are chosen,
-    ``gates`` their sigmoids, over their sum if ``normalize``, times ``scale``.  ``logits`` ([T, E]
-    float32, optional): the logits the choice was made from are written there too (tests compare them)."""
+    ``gates`` their sigmoids, over their sum if ``normalize``, times ``scale``.  ``rule`` "softmax_corrected": the same with
+    the softmax of all logits as scores.  ``logits`` ([T, E]
+    float32, optional): the logits the choice was made from are written there too (tests compare them).  ``rows``
+    (optional, [*, H] float32): the float32 normalised rows are wanted as its last T rows."""
     weight: torch.Tensor
     jitter_eps: float
     expert_ids: torch.Tensor
@@ -79,6 +88,7 @@ class RouterRequest:
     weights: torch.Tensor | None = None
     correction: torch.Tensor | None = None
     normalize: bool = True
+    rows: torch.Tensor | None = None
 
 
 @dataclass
@@ -159,6 +169,11 @@ class Norm(Part):
 
     def forward(self, x, want, row_index=None, pending=None, router=None):
         raise NotImplementedError
+
+
+class StreamMix(Part):
+    """How one part of a layer reads and feeds the residual streams."""
+    gather = mix = spread = None
 
 
 class EmbedAddition(Part):

@@ -8,6 +8,8 @@
 the norms come after the sums (a and the scales s are the norms' ``residual_scale`` and ``branch_scale``).
 ``sandwich``: h += norm1b(mixer(norm1(h))); h += norm2b(ffn(norm2(h))): a norm before and one after each part, the
 second applied to what the part adds (RMS norms; the second half only with a feed-forward).
+``streams``: the residual is S streams; a part reads norm(sum_s gather[s] x_s) and what it adds, r, goes into all of
+them: x_t <- sum_s mix[s, t] x_s + spread[t] r (the second half only with a feed-forward).
 An arrangement only orders parts; it does not know what they are.
 """
 from __future__ import annotations
@@ -15,11 +17,12 @@ from __future__ import annotations
 import torch
 
 from ..errors import ConfigError
-from ..registry import BLOCKS
-from .base import Pending
+from ..registry import BLOCKS, STREAM_MIXES
+from ..weights.sources import WeightSpec
+from .base import Pending, StreamMix
 
 
-def run_norm(norm, residual, want, pending=None, router=None, row_index=None):
+def run_norm(norm, residual, want, pending=None, router=None, row_index=None, gather=None):
     """Run a norm; a pending addition or a routing request that the norm cannot take is served
     by separate kernels instead.  Returns (outputs, router or None if it still has to be done)."""
     if pending is not None and not norm.supports_pending:
@@ -34,6 +37,8 @@ def run_norm(norm, residual, want, pending=None, router=None, row_index=None):
         kw["router"] = router
     if row_index is not None:
         kw["row_index"] = row_index
+    if gather is not None:
+        kw["gather"] = gather
     return norm.forward(residual, want, **kw), router
 
 
@@ -233,3 +238,69 @@ class PostNormBlock(Block):
         fed = branch_of(ffn, residual, lambda rows: ffn.forward(y, rows, step))
         p["norm2"].post(residual, fed)
         return None
+
+
+@STREAM_MIXES.register("hyper_connection")
+class HyperConnection(StreamMix):
+    """params: streams (S).  tensors: in [S] (the weights of the streams in the part's input), mix [S, S] ([from, to]),
+    out [S] (the weights of what the part adds)."""
+
+    graph_safe = True
+
+    def __init__(self, params, ctx):
+        super().__init__(params, ctx)
+        self.streams = int(params["streams"])
+        if not 1 <= self.streams <= 16:
+            raise ConfigError(f"hyper connection: {self.streams} streams are not supported (1 to 16)")
+
+    def weights(self):
+        S = self.streams
+        return {"in": WeightSpec((S,), role="vector", init="gamma"), "out": WeightSpec((S,), role="vector", init="gamma"),
+                "mix": WeightSpec((S, S), role="vector", std=0.3)}
+
+    def load(self, t):
+        self.gather, self.spread, self.mix = t["in"], t["out"], t["mix"]
+
+
+@BLOCKS.register("streams")
+class StreamsBlock(Block):
+    """``residual`` [T, S, width].  A part's addition is left pending with the mixing weights of its half, and the
+    next norm's kernel brings the streams up to date while it forms its own input from them."""
+    roles = ("hc1", "norm1", "mixer")
+
+    @staticmethod
+    def _run(part, norm, hc, residual, pending, request, want, call):
+        T, W = residual.shape[0], residual.shape[-1]
+        kw = {}
+        if request is not None and request.rows is not None:       # the float32 rows go where the part wants them
+            out = {dt: torch.empty((T, W), dtype=dt, device=residual.device) for dt in set(want) if dt != torch.float32}
+            out[torch.float32] = request.rows[-T:]
+            kw["out"] = out
+        x = norm.forward(residual, want, pending=pending, router=request, gather=hc.gather, **kw)
+        if getattr(part, "returns_pending", False):
+            pend = call(x, None)
+        else:                         # a part that adds into the rows it is given gets rows of zeros
+            rows = torch.zeros((T, W), dtype=torch.float32, device=residual.device)
+            pend = call(x, rows)
+            if pend is not None:
+                part.ops.apply_pending(rows, pend)
+            pend = Pending(partials=rows.unsqueeze(0))
+        pend.mix, pend.spread = hc.mix, hc.spread
+        return pend
+
+    def forward(self, residual, step, cache, state, writes_cache=True, carry=None):
+        p = self.parts
+        mixer, ffn = p["mixer"], p.get("ffn")
+        pend = self._run(mixer, p["norm1"], p["hc1"], residual, carry, None, mixer.input_dtypes(),
+                         lambda x, rows: mixer.forward(x, rows, step, cache, state, writes_cache))
+        if ffn is None:
+            return pend
+        if "norm2" not in p or "hc2" not in p:
+            raise ConfigError("block 'streams': a feed-forward needs its norm and its stream mix (norm2, hc2)")
+        request = ffn.router_request(residual.shape[0]) if hasattr(ffn, "router_request") else None
+        if request is not None and step.record is not None and getattr(request, "logits", 0) is None:
+            request.logits = request.weight.new_empty((residual.shape[0], request.weight.shape[0]), dtype=torch.float32)
+        want = ffn.input_dtypes_when_routed() if request is not None else ffn.input_dtypes()
+        return self._run(ffn, p["norm2"], p["hc2"], residual, pend, request, want,
+                         lambda y, rows: ffn.forward(y, rows, step, routed=request) if request is not None
+                         else ffn.forward(y, rows, step))

@@ -20,7 +20,9 @@ from .base import FeedForward, Pending, RouterRequest, mat, matmul_dtype, vec
 class GatedMLP(FeedForward):
     """params: hidden_size, intermediate_size, act; tensors gate_proj/up_proj [I,H], down_proj [H,I].
     act ``silu`` or ``gelu_pytorch_tanh``: act(gate) * up.  act ``swish_clamped`` with ``act_slope`` s and
-    ``act_limit`` c: g = min(gate, c), u = clamp(up, -c, c), g sigmoid(s g) (u + 1)."""
+    ``act_limit`` c: g = min(gate, c), u = clamp(up, -c, c), g sigmoid(s g) (u + 1).  ``bias``: all three projections have
+    biases (gate_proj.bias, up_proj.bias [I], down_proj.bias [H]).  ``pending``: the down product is left as partial
+    sums for whoever applies it."""
 
     graph_safe = True
 
@@ -28,6 +30,8 @@ class GatedMLP(FeedForward):
         super().__init__(params, ctx)
         self.hidden, self.inter = int(params["hidden_size"]), int(params["intermediate_size"])
         self.act = params.get("act", "silu")
+        self.has_bias = bool(params.get("bias", False))
+        self.returns_pending = bool(params.get("pending", False))
         self.act_params = None
         if self.act == "swish_clamped":
             self.act_params = (float(params["act_slope"]), float(params["act_limit"]))
@@ -37,17 +41,24 @@ class GatedMLP(FeedForward):
             raise ConfigError(f"gated_mlp: unknown activation {self.act!r}")
 
     def weights(self):
-        return {"gate_proj.weight": mat(self.inter, self.hidden), "up_proj.weight": mat(self.inter, self.hidden),
-                "down_proj.weight": mat(self.hidden, self.inter)}
+        w = {"gate_proj.weight": mat(self.inter, self.hidden), "up_proj.weight": mat(self.inter, self.hidden),
+             "down_proj.weight": mat(self.hidden, self.inter)}
+        if self.has_bias:
+            w.update({"gate_proj.bias": vec(self.inter), "up_proj.bias": vec(self.inter), "down_proj.bias": vec(self.hidden)})
+        return w
 
     def fused(self):
         return {"gate_up_proj.weight": ["gate_proj.weight", "up_proj.weight"]}
 
     def load(self, t):
-        dt = matmul_dtype(*t.values())
+        dt = matmul_dtype(*(v for k, v in t.items() if k.endswith("weight")))
         # gate and up rows in the layout the kernels want: one product gives both
         self.w_gate_up = self.ops.pair_gate_up(t["gate_proj.weight"].to(dt), t["up_proj.weight"].to(dt)).contiguous()
         self.w_down = t["down_proj.weight"].to(dt)
+        self.b_gate_up = self.b_down = None
+        if self.has_bias:
+            self.b_gate_up = self.ops.pair_gate_up(t["gate_proj.bias"][:, None], t["up_proj.bias"][:, None]).reshape(-1).contiguous()
+            self.b_down = t["down_proj.bias"]
 
     def input_dtypes(self):
         return (self.w_gate_up.dtype,)
@@ -55,11 +66,14 @@ class GatedMLP(FeedForward):
     def forward(self, x, residual, step):
         xin = x[self.w_gate_up.dtype]
         a = torch.empty((xin.shape[0], self.inter), dtype=self.w_gate_up.dtype, device=xin.device)
+        kw = {} if self.b_gate_up is None else {"bias": self.b_gate_up}
         if self.act_params is None:
-            self.ops.gated_gemm(xin, self.w_gate_up, a, self.act)
+            self.ops.gated_gemm(xin, self.w_gate_up, a, self.act, **kw)
         else:
-            self.ops.gated_gemm(xin, self.w_gate_up, a, self.act, act_params=self.act_params)
-        self.ops.gemm(a, self.w_down, residual, accumulate=True)
+            self.ops.gated_gemm(xin, self.w_gate_up, a, self.act, act_params=self.act_params, **kw)
+        if self.returns_pending:
+            return Pending(partials=self.ops.gemm_partials(a, self.w_down), bias=self.b_down)
+        self.ops.gemm(a, self.w_down, residual, bias=self.b_down, accumulate=True)
 
 
 @FEED_FORWARDS.register("mlp")
@@ -174,10 +188,17 @@ class GroupedTopKMoE(FeedForward):
     chosen experts' down(act(gate x) * (up x)).  (No counterpart in the reference, whose feed-forward is dense:
     crates/thuban_model/src/ops/mlp.rs:24-79.)
 
-    params: hidden_size, intermediate_size, num_experts, top, groups, keep_groups, router_scale, act.
-    tensors: router [E, H]; e{i}.gate / e{i}.up [I, H], e{i}.down [H, I]."""
+    ``identity`` I: the router has I more outputs for experts without weights, whose output is x itself; all E + I take
+    part in the softmax and in the choice.  ``correction``: a stored offset per router output joins the scores for the
+    choice only (then no groups, or groups scored as the sum of their two best).  act ``swish_clamped`` with ``act_slope``
+    and ``act_limit`` as in ``gated_mlp``.
+
+    params: hidden_size, intermediate_size, num_experts, top, groups, keep_groups, router_scale, act (with its constants),
+    identity, correction.
+    tensors: router [E + I, H]; e{i}.gate / e{i}.up [I, H], e{i}.down [H, I]; correction [E + I]."""
 
     graph_safe = True
+    returns_pending = True        # the rows given are never touched: what the experts add goes back as a Pending
 
     def __init__(self, params, ctx):
         super().__init__(params, ctx)
@@ -187,17 +208,27 @@ class GroupedTopKMoE(FeedForward):
         self.groups, self.keep = int(p.get("groups", 1)), int(p.get("keep_groups", 1))
         self.router_scale = float(p.get("router_scale", 1.0))
         self.act = p.get("act", "silu")
-        if not 1 <= self.E <= 256:
-            raise ConfigError(f"num_experts {self.E} is not supported (1..256)")
-        if not 1 <= self.top <= min(self.E, 16):
-            raise ConfigError(f"{self.top} experts a token of {self.E} is not supported (1..16)")
-        if self.groups < 1 or self.groups > 64 or self.E % self.groups:
-            raise ConfigError(f"{self.E} experts do not form {self.groups} equal groups (up to 64)")
-        if not 1 <= self.keep <= self.groups or self.keep * (self.E // self.groups) < self.top:
+        self.act_params = (float(p["act_slope"]), float(p["act_limit"])) if self.act == "swish_clamped" else None
+        self.identity = int(p.get("identity", 0) or 0)
+        self.correction = bool(p.get("correction", False))
+        self.choices = self.E + self.identity          # what the router chooses from
+        if self.E < 1 or self.identity < 0 or self.choices > 256:
+            raise ConfigError(f"num_experts {self.E} (and {self.identity} identity experts) is not supported (1..256)")
+        if not 1 <= self.top <= min(self.choices, 16):
+            raise ConfigError(f"{self.top} experts a token of {self.choices} is not supported (1..16)")
+        if self.groups < 1 or self.groups > 64 or self.choices % self.groups:
+            raise ConfigError(f"{self.choices} experts do not form {self.groups} equal groups (up to 64)")
+        if not 1 <= self.keep <= self.groups or self.keep * (self.choices // self.groups) < self.top:
             raise ConfigError(f"{self.keep} of {self.groups} groups cannot give {self.top} experts a token")
+        if self.act_params is not None and self.act_params[1] <= 0:
+            raise ConfigError(f"grouped_topk_moe: act_limit must be positive, got {self.act_params[1]}")
+        if self.act_params is None and self.act not in ("silu", "gelu_pytorch_tanh"):
+            raise ConfigError(f"grouped_topk_moe: unknown activation {self.act!r}")
 
     def weights(self):
-        w = {"router": mat(self.E, self.hidden)}
+        w = {"router": mat(self.choices, self.hidden)}
+        if self.correction:
+            w["correction"] = vec(self.choices)
         for e in range(self.E):
             w[f"e{e}.gate"] = mat(self.inter, self.hidden)
             w[f"e{e}.up"] = mat(self.inter, self.hidden)
@@ -206,7 +237,8 @@ class GroupedTopKMoE(FeedForward):
 
     def load(self, t):
         self.w_router = t["router"]
-        dt = matmul_dtype(*(v for k, v in t.items() if k != "router"))
+        self.w_correction = t.get("correction")
+        dt = matmul_dtype(*(v for k, v in t.items() if k not in ("router", "correction")))
         self.w13 = torch.stack([self.ops.pair_gate_up(t[f"e{e}.gate"].to(dt), t[f"e{e}.up"].to(dt))
                                 for e in range(self.E)], 0).contiguous()
         self.w2 = torch.stack([t[f"e{e}.down"].to(dt) for e in range(self.E)], 0).contiguous()
@@ -216,30 +248,43 @@ class GroupedTopKMoE(FeedForward):
 
     def router_request(self, n_rows):
         """Routing can ride on the norm before this part (the normalised row is in registers there)."""
-        dev = self.w_router.device
-        return RouterRequest(self.w_router, 0.0, torch.empty((n_rows, self.top), dtype=torch.int32, device=dev),
-                             torch.empty((n_rows, self.top), dtype=torch.float32, device=dev), top=self.top,
-                             groups=self.groups, keep=self.keep, scale=self.router_scale)
+        dev, k = self.w_router.device, self.top
+        rows = None
+        if self.identity:      # the experts' rows and, after them, the rows as normalised: what identity experts hand on
+            rows = torch.empty(((k + 1) * n_rows, self.hidden), dtype=torch.float32, device=dev)
+        return RouterRequest(self.w_router, 0.0, torch.empty((n_rows, k), dtype=torch.int32, device=dev),
+                             torch.empty((n_rows, k), dtype=torch.float32, device=dev), top=k, groups=self.groups,
+                             keep=self.keep, scale=self.router_scale, rule="softmax_corrected" if self.correction else "",
+                             correction=self.w_correction, rows=rows)
 
     def input_dtypes_when_routed(self):
-        return (self.w13.dtype,)
+        return (torch.float32, self.w13.dtype) if self.identity else (self.w13.dtype,)
 
     def forward(self, x, residual, step, routed=None):
         ops = self.ops
         xa = x[self.w13.dtype]
         T, dev, k = xa.shape[0], xa.device, self.top
+        y = None
         if routed is not None:
-            ids, gates, logits = routed.expert_ids, routed.gates, routed.logits
+            ids, gates, logits, y = routed.expert_ids, routed.gates, routed.logits, routed.rows
         else:
             ids = torch.empty((T, k), dtype=torch.int32, device=dev)
             gates = torch.empty((T, k), dtype=torch.float32, device=dev)
-            logits = torch.empty((T, self.E), dtype=torch.float32, device=dev) if step.record is not None else None
-            ops.router_topk(x[torch.float32], self.w_router, k, self.groups, self.keep, self.router_scale, ids, gates, logits)
-        plan, xs = ops.moe_dispatch(ids, self.E, ops.moe_tile_rows(T, self.E, self.w13.dtype, k), xa)
+            logits = torch.empty((T, self.choices), dtype=torch.float32, device=dev) if step.record is not None else None
+            if self.correction:
+                ops.router_sigmoid_grouped(x[torch.float32], self.w_router, self.w_correction, k, self.groups, self.keep, True,
+                                           self.router_scale, ids, gates, logits, softmax=True)
+            else:
+                ops.router_topk(x[torch.float32], self.w_router, k, self.groups, self.keep, self.router_scale, ids, gates, logits)
+        if y is None:
+            y = torch.empty(((k + (1 if self.identity else 0)) * T, self.hidden), dtype=torch.float32, device=dev)
+        if self.identity and x[torch.float32].data_ptr() != y[k * T:].data_ptr():
+            y[k * T:].copy_(x[torch.float32])
+        plan, xs = ops.moe_dispatch(ids, self.E, ops.moe_tile_rows(T, self.choices, self.w13.dtype, k), xa)
         a = torch.empty((k * T, self.inter), dtype=self.w13.dtype, device=dev)
-        ops.gated_gemm(xs, self.w13, a, self.act, plan)
-        y = torch.empty((k * T, self.hidden), dtype=torch.float32, device=dev)
-        ops.grouped_gemm(a, self.w2, y, plan, plan_ready=True)
+        kw = {} if self.act_params is None else {"act_params": self.act_params}
+        ops.gated_gemm(xs, self.w13, a, self.act, plan, **kw)
+        ops.grouped_gemm(a, self.w2, y[:k * T], plan, plan_ready=True)
         if step.record is not None:
             step.record.setdefault("experts", []).append(ids)
             step.record.setdefault("gates", []).append(gates)

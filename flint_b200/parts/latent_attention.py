@@ -12,7 +12,11 @@ probability-weighted sum of the latents only.  So the mixer runs as attention of
 cached row per token whose first C numbers double as the value, with two small per-head products around
 it (W_uk folded into the query, W_uv applied to the result); keys and values are never materialised.
 A layer with ``own_cache`` False makes no latent: it reads the rows another layer call cached, with its
-own W_uk, W_uv, queries and output projection.
+own W_uk, W_uv, queries, window and output projection.
+
+Options: queries through a latent of their own, q = W_uq rmsnorm(W_dq x) (``q_rank``); a learned sink logit per head that
+joins the softmax's denominator and has no key (``sinks``); the heads' outputs multiplied number by number by
+sigmoid(W_g x) (``out_gate``).
 
 The reference's attention is grouped-query over cached keys and values
 (crates/thuban_architectures/src/transformer/forward.rs:114-365); it has no latent form.
@@ -33,11 +37,15 @@ class LatentAttention(Mixer):
     """params: hidden_size, num_heads, dim (unrotated q/k dims per head), rot_dim (rotated dims per head, one
     rotated key part for all heads), value_dim, kv_rank (latent size), scale, norm_eps (of the latent's RMS norm),
     window (0 = none), own_cache (False: reads another call's cache and has no down-projection),
-    position (PartSpec; its rotary_dim of the rot_dim dims rotate).
+    cache_window (the positions its cached rows stay reachable for, 0 = all; default: window; larger when another
+    call that reads them has a longer window), position (PartSpec; its rotary_dim of the rot_dim dims rotate);
+    q_rank (0: none), sinks, out_gate.
     tensors: q [H (dim + rot_dim), hidden], dkv [kv_rank + rot_dim, hidden], dkv.norm [kv_rank],
-    uk [H dim, kv_rank], uv [H value_dim, kv_rank], o [hidden, H value_dim]."""
+    uk [H dim, kv_rank], uv [H value_dim, kv_rank], o [hidden, H value_dim]; with q_rank dq [q_rank, hidden], dq.norm
+    [q_rank], uq [H (dim + rot_dim), q_rank] instead of q; sink [H]; g [H value_dim, hidden]."""
 
     graph_safe = True
+    returns_pending = True
 
     def __init__(self, params, ctx):
         super().__init__(params, ctx)
@@ -52,10 +60,19 @@ class LatentAttention(Mixer):
         self.scale = float(p["scale"])
         self.eps = float(p["norm_eps"])
         self.window = int(p.get("window", 0) or 0)
+        self.cache_window = int(p.get("cache_window", self.window) or 0)
+        self.q_rank = int(p.get("q_rank", 0) or 0)
+        self.sinks, self.out_gate = bool(p.get("sinks", False)), bool(p.get("out_gate", False))
+        if self.cache_window and (not self.window or self.cache_window < self.window):
+            raise ConfigError("latent attention: the cached rows must stay reachable for the layer's own window")
         self.own_cache = bool(p.get("own_cache", True))
         self.position = shared_position_encoding(p["position"], ctx) if p.get("position") is not None else None
         self.rot = self.position.rotary_dim if self.position is not None else 0
         self.rot_style = self.position.style if self.position is not None else "half"
+        if self.q_rank < 0:
+            raise ConfigError("latent attention: q_rank must not be negative")
+        if self.out_gate and not self.q_rank:
+            raise ConfigError("latent attention: the output gate goes with queries through a latent (q_rank)")
         if self.rot > self.R:
             raise ConfigError(f"latent attention: {self.rot} rotating dims exceed rot_dim {self.R}")
         self.Dk = self.C + self.R
@@ -63,18 +80,31 @@ class LatentAttention(Mixer):
 
     def weights(self):
         H, D, R, V, C, W = self.H, self.D, self.R, self.V, self.C, self.hidden
-        w = {"q": mat(H * (D + R), W), "uk": mat(H * D, C), "uv": mat(H * V, C), "o": mat(W, H * V)}
+        w = {"uk": mat(H * D, C), "uv": mat(H * V, C), "o": mat(W, H * V)}
+        if self.q_rank:
+            w.update({"dq": mat(self.q_rank, W), "dq.norm": vec(self.q_rank, init="gamma"), "uq": mat(H * (D + R), self.q_rank)})
+        else:
+            w["q"] = mat(H * (D + R), W)
         if self.own_cache:
             w["dkv"] = mat(C + R, W)
             w["dkv.norm"] = vec(C, init="gamma")
+        if self.sinks:
+            w["sink"] = vec(H)
+        if self.out_gate:
+            w["g"] = mat(H * V, W)
         return w
 
     def load(self, t):
         H, D, V, C = self.H, self.D, self.V, self.C
-        dt = matmul_dtype(*(v for k, v in t.items() if k != "dkv.norm"))
-        # q and the latent's down-projection are one product
-        self.w_in = torch.cat([t["q"].to(dt)] + ([t["dkv"].to(dt)] if self.own_cache else []), 0).contiguous()
+        dt = matmul_dtype(*(v for k, v in t.items() if k not in ("dkv.norm", "dq.norm", "sink")))
+        # q (or its latent), the latent's down-projection and the output gate are one product
+        names = ["dq" if self.q_rank else "q"] + (["dkv"] if self.own_cache else []) + (["g"] if self.out_gate else [])
+        self.w_in = torch.cat([t[n].to(dt) for n in names], 0).contiguous()
         self.w_norm = t.get("dkv.norm")
+        self.w_q_norm, self.w_uq = t.get("dq.norm"), t["uq"].to(dt) if self.q_rank else None
+        self.w_sink = t.get("sink")
+        # where the gate's columns start in that product
+        self.gate_col = (self.q_rank or H * (D + self.R)) + (C + self.R if self.own_cache else 0)
         # W_uk per head, transposed: the product that folds it into the query takes [C, D] per head
         self.w_ukT = t["uk"].to(dt).view(H, D, C).transpose(1, 2).contiguous()
         self.w_uv = t["uv"].to(dt).view(H, V, C).contiguous()
@@ -89,7 +119,7 @@ class LatentAttention(Mixer):
 
     def cache_spec(self):
         # one row per token for all heads, no separate values: the latent is the start of the row
-        return KVSpec(1, self.row_w, self.window, value_dim=0) if self.own_cache else None
+        return KVSpec(1, self.row_w, self.cache_window, value_dim=0) if self.own_cache else None
 
     def plan_step(self, step, captured):
         """A batch of decoded tokens that is captured as a CUDA graph has its key ranges cut for a bucketed
@@ -111,18 +141,28 @@ class LatentAttention(Mixer):
         xin = x[self.w_in.dtype]
         T, dev = xin.shape[0], xin.device
         act = self.ctx.act_dtype if self.w_in.dtype == torch.bfloat16 else torch.float32
-        proj = ops.gemm_partials(xin, self.w_in)                 # [S, T, H (D + R) (+ C + R)] partial sums
+        proj = ops.gemm_partials(xin, self.w_in)      # [S, T, H (D + R) or q_rank (+ C + R) (+ H V)] partial sums
+        gate = proj[:, :, self.gate_col:] if self.out_gate else None
         q_plain = torch.empty((T, H, D), dtype=act, device=dev)
         qa = torch.empty((T, H, self.Dk), dtype=act, device=dev)
-        ops.latent_prepare(proj, step.pos, step.slot, self.cos, self.sin, self.rot, self.rot_style, self.w_norm, self.eps,
+        if self.q_rank:
+            c_q = torch.empty((T, self.q_rank), dtype=act, device=dev)
+            ops.latent_down(proj, self.q_rank, self.w_q_norm, step.pos, step.slot, self.cos, self.sin, self.rot, self.rot_style,
+                            self.w_norm, self.eps, c_q, cache, R, C, writes_cache, step.status)
+            q_proj, writes_cache = ops.gemm_partials(c_q, self.w_uq), False
+        else:
+            q_proj = proj
+        ops.latent_prepare(q_proj, step.pos, step.slot, self.cos, self.sin, self.rot, self.rot_style, self.w_norm, self.eps,
                            q_plain, qa, cache, H, D, R, C, writes_cache, step.status)
         if D:
             ops.head_products(q_plain, self.w_ukT, qa[:, :, :C])     # qa[t, h, :C] = W_uk_h^T q_plain[t, h]
         else:
             qa[:, :, :C].zero_()
         o_lat = torch.empty((T, H, C), dtype=act, device=dev)
-        ops.latent_attention(qa, cache, step, o_lat, H, C, self.window, self.scale)
+        kw = {} if self.w_sink is None else {"sinks": self.w_sink}
+        ops.latent_attention(qa, cache, step, o_lat, H, C, self.window, self.scale, **kw)
         attn = torch.empty((T, H, V), dtype=act, device=dev)
-        ops.head_products(o_lat, self.w_uv, attn)                    # attn[t, h] = W_uv_h o_lat[t, h]
+        kw = {} if gate is None else {"gate": gate}
+        ops.head_products(o_lat, self.w_uv, attn, **kw)              # attn[t, h] = W_uv_h o_lat[t, h] (* sigmoid(gate))
         # the output projection is handed on as partial sums
         return Pending(partials=ops.gemm_partials(attn.view(T, H * V), self.w_o))

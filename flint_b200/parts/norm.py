@@ -4,7 +4,8 @@ LayerNorm: y = (x - mean) * rsqrt(var + eps) * gamma + beta with var = mean((x-m
 RMSNorm: y = x * rsqrt(mean(x^2) + eps) * gamma; with ``weight_offset`` c the stored scale w is an offset,
 gamma = c + w (formed once, in float32, when the tensors are loaded).  Statistics are float32.  With
 ``branch_scale`` the norm also stores a scale s per channel for what a block adds before it, and ``post`` runs the
-norm after the sum: x <- norm(a x + s * branch) with a = ``residual_scale``, in place.  The
+norm after the sum: x <- norm(a x + s * branch) with a = ``residual_scale``, in place.  ``output_scale`` c multiplies the
+result (folded into gamma and beta when they are loaded).  The
 reference's norm shader has both as modes (crates/thuban_kernel/wgsl/norm.wgsl:66-83,
 112-121) and picks by config key (crates/thuban_architectures/src/phi.rs:55-63).
 """
@@ -30,6 +31,7 @@ class _RowNorm(Norm):
         # for a block that norms after the sum: the residual's weight, and whether a scale of the branch is stored
         self.residual_scale = float(params.get("residual_scale", 1.0))
         self.has_branch_scale = bool(params.get("branch_scale", False))
+        self.output_scale = float(params.get("output_scale", 1.0))
         self.gamma = self.beta = self.branch_scale = None
 
     def weights(self):
@@ -45,6 +47,9 @@ class _RowNorm(Norm):
         if self.weight_offset:
             self.gamma = (self.gamma.to(torch.float32) + self.weight_offset).contiguous()
         self.beta = tensors.get("bias")
+        if self.output_scale != 1.0:
+            self.gamma = (self.gamma.to(torch.float32) * self.output_scale).contiguous()
+            self.beta = (self.beta.to(torch.float32) * self.output_scale).contiguous() if self.beta is not None else None
         self.branch_scale = tensors.get("branch_scale")
 
     supports_pending = True
@@ -56,15 +61,17 @@ class _RowNorm(Norm):
         self.ops.post_norm(x, branch.partials, branch.bias, self.branch_scale, self.residual_scale, self.gamma, self.beta,
                            self.eps, self.mode, out_copy=copy)
 
-    def forward(self, x, want, row_index=None, pending=None, router=None, out=None):
-        """``out``: {element type: tensor} to write into instead of new tensors (then ``want`` is ignored)."""
+    def forward(self, x, want, row_index=None, pending=None, router=None, out=None, gather=None):
+        """``out``: {element type: tensor} to write into instead of new tensors (then ``want`` is ignored).  ``gather``
+        [S]: x is [T, S, width] and its weighted sum over the streams is normed."""
         rows = row_index.numel() if row_index is not None else x.shape[0]
         if out is None:
             out = {}
             for dt in set(want):
                 out[dt] = torch.empty((rows, self.width), dtype=dt, device=x.device)
+        kw = {} if gather is None else {"gather": gather}
         self.ops.row_norm(x, self.gamma, self.beta, self.eps, self.mode, out_f32=out.get(torch.float32),
-                          out_bf16=out.get(torch.bfloat16), row_index=row_index, pending=pending, router=router)
+                          out_bf16=out.get(torch.bfloat16), row_index=row_index, pending=pending, router=router, **kw)
         return out
 
 

@@ -4,8 +4,11 @@ model with a scalar decay per head (the state-space duality form of Mamba-2).
 A third, ``retention``, is linear attention with a fixed decay per head: S <- decay_h S + k v^T, o = S^T q, with q and
 k rotated by the position; it runs the state-space form of the same kernel with the decay and the step size constant.
 
-Both keep, per request, a float32 matrix S per head and the last ``taps - 1`` inputs of a short causal convolution
-in one row of the cache manager's state slab (zeroed on admission), and both run the same recurrence kernel
+A fourth, ``rglru``, carries one number per channel: Griffin's recurrent block with a real-gated linear recurrent unit,
+S <- a S + sqrt(1 - a^2) i u with a and i from block-diagonal gates; it has kernels of its own.
+
+The first two keep, per request, a float32 matrix S per head and the last ``taps - 1`` inputs of a short causal convolution
+in one row of the cache manager's state slab (zeroed on admission), and run the same recurrence kernel
 (``ops.recurrence_scan``), which walks every request's rows of the step in order from the state its earlier steps
 left: the result does not depend on how a prompt was cut.  With k, q of a key head (or B, C of a group), a value
 row v and S [dim, value_dim]:
@@ -274,4 +277,72 @@ class StateSpaceDuality(_Recurrent):
         act = self.ctx.act_dtype if self.w_o.dtype == torch.bfloat16 else torch.float32
         out = torch.empty((T, inner), dtype=act, device=dev)
         ops.gated_norm(o, proj[:, :inner], "silu", True, self.w_norm, self.eps, self.norm_groups, out)
+        return Pending(partials=ops.gemm_partials(out, self.w_o))
+
+
+@MIXERS.register("rglru")
+class RealGatedLRU(_Recurrent):
+    """Griffin's recurrent block: y = gelu_tanh(W_y x + b_y); u = causal convolution (with a bias, no activation) of
+    W_x x + b_x; r, i = sigmoid(ra u + ra.b), sigmoid(ri u + ri.b) with block-diagonal ra, ri; log a = -c r softplus(lam);
+    S <- a S + sqrt(1 - a^2) i u from zero; output W_o (S * y).  From the convolution to S everything is float32.  The
+    state (S and the convolution's last inputs) is a ``StateSpec`` slab zeroed at admission.
+
+    params: hidden_size, width, blocks, conv_taps, decay_scale (c).
+    tensors: y, x [width, hidden] with y.b, x.b [width]; conv [width, taps], conv.b [width]; ra, ri [blocks, width / blocks,
+    width / blocks] with ra.b, ri.b [blocks, width / blocks]; lam [width]; o [hidden, width]."""
+
+    def __init__(self, params, ctx):
+        super().__init__(params, ctx)
+        p = params
+        self.hidden, self.W, self.blocks = int(p["hidden_size"]), int(p["width"]), int(p["blocks"])
+        self.taps, self.decay_scale = int(p["conv_taps"]), float(p["decay_scale"])
+        if self.W < 1 or self.blocks < 1 or self.W % self.blocks:
+            raise ConfigError(f"rglru: width {self.W} is not a multiple of {self.blocks} blocks")
+        if not 1 <= self.taps <= 64:
+            raise ConfigError(f"rglru: {self.taps} taps are not supported (1 to 64)")
+
+    def weights(self):
+        W, H, B, n = self.W, self.hidden, self.blocks, self.W // self.blocks
+        return {"y": mat(W, H), "y.b": vec(W), "x": mat(W, H), "x.b": vec(W), "conv": conv_weight(W, self.taps), "conv.b": vec(W),
+                "ra": mat(B, n, n), "ra.b": WeightSpec((B, n), role="vector"), "ri": mat(B, n, n),
+                "ri.b": WeightSpec((B, n), role="vector"), "lam": vec(W), "o": mat(H, W)}
+
+    def load(self, t):
+        dt = matmul_dtype(t["y"], t["x"], t["o"])
+        self.w_in = torch.cat([t["y"].to(dt), t["x"].to(dt)], 0).contiguous()      # one product gives both branches
+        self.b_in = torch.cat([t["y.b"], t["x.b"]], 0).contiguous()
+        self.w_conv, self.b_conv = t["conv"], t["conv.b"]
+        gdt = matmul_dtype(t["ra"], t["ri"])
+        self.w_r, self.w_i = t["ra"].to(gdt).contiguous(), t["ri"].to(gdt).contiguous()
+        self.b_r, self.b_i = t["ra.b"].reshape(-1).contiguous(), t["ri.b"].reshape(-1).contiguous()
+        # log a = rate * r
+        self.rate = (-self.decay_scale * torch.nn.functional.softplus(t["lam"].to(torch.float32))).contiguous()
+        self.w_o = t["o"].to(dt)
+
+    def input_dtypes(self):
+        return (self.w_in.dtype,)
+
+    def state_spec(self):
+        # S, then `taps` rows of the convolution's inputs (the input at p in row p mod taps: the row a token writes is
+        # none that its own convolution reads)
+        return StateSpec((self.W * (1 + self.taps),), torch.float32)
+
+    def forward(self, x, residual, step, cache, state, writes_cache=True):
+        ops, W = self.ops, self.W
+        S, ring = self._split_state(state, W)
+        xin = x[self.w_in.dtype]
+        T, dev = xin.shape[0], xin.device
+        act = self.ctx.act_dtype if self.w_o.dtype == torch.bfloat16 else torch.float32
+        out = torch.empty((T, W), dtype=act, device=dev)
+        if T == len(step.entries) and W // self.blocks <= ops.RGLRU_STEP_BLOCK:          # single tokens: one launch
+            ops.rglru_step(ops.gemm_partials(xin, self.w_in), self.b_in, self.w_conv, self.b_conv, self.w_r, self.b_r, self.w_i,
+                           self.b_i, self.rate, step.pos, step.slot, state, out)
+            return Pending(partials=ops.gemm_partials(out, self.w_o))
+        f32 = dict(dtype=torch.float32, device=dev)
+        proj = torch.empty((T, 2 * W), **f32)
+        ops.gemm(xin, self.w_in, proj, bias=self.b_in)
+        u, a, b = torch.empty((T, W), **f32), torch.empty((T, W), **f32), torch.empty((T, W), **f32)
+        ops.short_conv(proj, W, self.w_conv, self.b_conv, "none", step.pos, step.slot, ring, u, ring_rows=self.taps)
+        ops.rglru_gates(u, self.w_r, self.b_r, self.w_i, self.b_i, self.rate, a, b)
+        ops.rglru_scan(a, b, proj[:, :W], step.slot, request_starts(step), len(step.entries), step.longest_entry, S, out)
         return Pending(partials=ops.gemm_partials(out, self.w_o))

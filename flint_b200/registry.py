@@ -49,5 +49,6 @@ FEED_FORWARDS = Registry("feed-forward")
 NORMS = Registry("norm")
 POSITION_ENCODINGS = Registry("position encoding")
 BLOCKS = Registry("block arrangement")
+STREAM_MIXES = Registry("stream mix")
 EMBED_ADDITIONS = Registry("embedding addition")
 ARCHITECTURES = Registry("architecture")

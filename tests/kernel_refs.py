@@ -38,12 +38,13 @@ class RefOps:
         self.tc_error, self.page_error, self.token_out = self.readback[0:1], self.readback[1:2], self.readback[2:]
 
     # ------------------------------------------------------------------ row-wise
-    def embed(self, ids, table, out, scale=1.0, fed_rows=None, fed_from=None):
+    def embed(self, ids, table, out, scale=1.0, fed_rows=None, fed_from=None, copies=1):
         ids = ids.long()
         if fed_rows is not None:
             fed = fed_rows.long()
             ids = torch.where(fed >= 0, fed_from.to(fed.device).long()[fed.clamp(min=0)], ids)
-        out.copy_((table[ids].to(self.cd) * scale).to(out.dtype))
+        rows = (table[ids].to(self.cd) * scale).to(out.dtype)
+        out.copy_(rows[:, None, :].expand(-1, copies, -1) if out.dim() == 3 else rows)
 
     def norm(self, x, gamma, beta, eps, mode, out_f32=None, out_bf16=None, row_index=None):
         xs = x[row_index.long()] if row_index is not None else x
@@ -62,7 +63,17 @@ class RefOps:
             out_bf16.copy_(y.to(torch.float32).to(torch.bfloat16))
 
     def row_norm(self, x, gamma, beta, eps, mode, out_f32=None, out_bf16=None, row_index=None, pending=None,
-                 router=None):
+                 router=None, gather=None):
+        if x.dim() == 3:                       # several streams of every row
+            xs = x
+            if pending is not None:
+                if row_index is not None:
+                    xs = x.clone()             # brought up to date for this norm only
+                self.apply_pending(xs, pending)
+            if gamma is None:
+                return
+            u = torch.einsum("s,tsw->tw", gather.to(self.cd), xs.to(self.cd)).to(x.dtype)
+            return self.row_norm(u, gamma, beta, eps, mode, out_f32, out_bf16, row_index, None, router)
         if pending is not None:
             self.apply_pending(x, pending)
         if gamma is None:
@@ -72,10 +83,10 @@ class RefOps:
             tmp = torch.empty((x.shape[0], x.shape[1]), dtype=torch.float32)
         self.norm(x, gamma, beta, eps, mode, out_f32=tmp, out_bf16=out_bf16, row_index=row_index)
         if router is not None:
-            if getattr(router, "rule", "") == "sigmoid_grouped":
+            if getattr(router, "rule", "") in ("sigmoid_grouped", "softmax_corrected"):
                 self.router_sigmoid_grouped(tmp, router.weight, router.correction, router.top, router.groups, router.keep,
                                             router.normalize, router.scale, router.expert_ids, router.gates,
-                                            getattr(router, "logits", None))
+                                            getattr(router, "logits", None), softmax=router.rule == "softmax_corrected")
             elif getattr(router, "rule", "") == "sigmoid":
                 self.router_sigmoid(tmp, router.weight, router.weight.shape[0] - router.extra, router.top, router.expert_ids,
                                     router.gates, router.weights, getattr(router, "logits", None))
@@ -87,6 +98,18 @@ class RefOps:
                                         getattr(router, "logits", None))
 
     def apply_pending(self, x, pending):
+        if x.dim() == 3:
+            r = torch.zeros((x.shape[0], x.shape[2]), dtype=self.cd)
+            if pending.partials is not None:
+                r = r + pending.partials.to(self.cd).sum(0)
+                if pending.bias is not None:
+                    r = r + pending.bias.to(self.cd)
+            if pending.y is not None:
+                self.moe_combine(r, pending.y, pending.row_of, pending.gates)
+            new = torch.einsum("sk,tsw->tkw", pending.mix.to(self.cd), x.to(self.cd)) \
+                + pending.spread.to(self.cd)[None, :, None] * r[:, None, :]
+            x.copy_(new.to(x.dtype))
+            return
         if pending.partials is not None:
             add = pending.partials.to(self.cd).sum(0)
             if pending.bias is not None:
@@ -167,23 +190,25 @@ class RefOps:
         """This implementation keeps the gate rows before the up rows."""
         return torch.cat([w_gate, w_up], -2)
 
-    def gated_gemm(self, x, w13, out, act="silu", plan=None, act_params=None):
-        """w13 = pair_gate_up(gate, up): [2N, K] or [E, 2N, K]."""
+    def gated_gemm(self, x, w13, out, act="silu", plan=None, act_params=None, bias=None):
+        """w13 = pair_gate_up(gate, up): [2N, K] or [E, 2N, K]; bias = pair_gate_up of the two biases, [2N]."""
         xs = x.to(self.cd)
         n = w13.shape[-2] // 2
-        if act == "swish_clamped":
-            slope, limit = act_params
-            g = torch.clamp(xs @ w13[:n].to(self.cd).T, max=limit)
-            u = torch.clamp(xs @ w13[n:].to(self.cd).T, -limit, limit)
-            out.copy_((g * torch.sigmoid(slope * g) * (u + 1.0)).to(out.dtype))
-            return
+
+        def unit(g, u):
+            if act == "swish_clamped":
+                slope, limit = act_params
+                g, u = torch.clamp(g, max=limit), torch.clamp(u, -limit, limit)
+                return (g * torch.sigmoid(slope * g) * (u + 1.0)).to(out.dtype)
+            return (_act(g, act) * u).to(out.dtype)
         if plan is None:
-            out.copy_((_act(xs @ w13[:n].to(self.cd).T, act) * (xs @ w13[n:].to(self.cd).T)).to(out.dtype))
+            g, u = xs @ w13[:n].to(self.cd).T, xs @ w13[n:].to(self.cd).T
+            if bias is not None:
+                g, u = g + bias[:n].to(self.cd), u + bias[n:].to(self.cd)
+            out.copy_(unit(g, u))
             return
         for e, lo, hi in self._rows_by_expert(plan):
-            g = xs[lo:hi] @ w13[e, :n].to(self.cd).T
-            u = xs[lo:hi] @ w13[e, n:].to(self.cd).T
-            out[lo:hi] = (_act(g, act) * u).to(out.dtype)
+            out[lo:hi] = unit(xs[lo:hi] @ w13[e, :n].to(self.cd).T, xs[lo:hi] @ w13[e, n:].to(self.cd).T)
 
     def grouped_gemm(self, x, w, out, plan, plan_ready=False):
         xs = x.to(self.cd)
@@ -346,8 +371,9 @@ class RefOps:
                 a = t
         return runs
 
-    def short_conv(self, u, col0, w, bias, act, pos, slot, state, y):
+    def short_conv(self, u, col0, w, bias, act, pos, slot, state, y, ring_rows=None):
         C, taps = w.shape
+        R = ring_rows or taps - 1
         x = u[:, col0:col0 + C].to(self.cd)
         ww = w.to(self.cd)
         res = torch.zeros(x.shape, dtype=self.cd)
@@ -356,13 +382,13 @@ class RefOps:
             past = torch.zeros(taps - 1, C, dtype=self.cd)       # inputs of positions p0 - taps + 1 .. p0 - 1
             for d in range(1, taps):
                 if p0 - d >= 0:
-                    r = (p0 - d) % (taps - 1)
+                    r = (p0 - d) % R
                     past[taps - 1 - d] = state[sl, r * C:(r + 1) * C].to(self.cd)
             seq = torch.cat([past, x[a:b]], 0)
             for j in range(taps):
                 res[a:b] += ww[:, j] * seq[j:j + b - a]
             for t in range(max(a, b - (taps - 1)), b):
-                r = int(pos[t]) % (taps - 1)
+                r = int(pos[t]) % R
                 state[sl, r * C:(r + 1) * C] = x[t].to(state.dtype)
         if bias is not None:
             res = res + bias.to(self.cd)
@@ -559,10 +585,10 @@ class RefOps:
         dt.fill_(dt_value)
 
     def router_sigmoid_grouped(self, x, wr, correction, top, n_groups, keep, normalize, scale, expert_ids, gates,
-                               logits_out=None):
+                               logits_out=None, softmax=False):
         z = x.to(self.cd) @ wr.to(self.cd).T
         T, E = z.shape
-        s = torch.sigmoid(z)
+        s = torch.softmax(z, -1) if softmax else torch.sigmoid(z)
         c = s + correction.to(self.cd) if correction is not None else s.clone()
         per = E // n_groups
         if keep < n_groups:
@@ -601,8 +627,71 @@ class RefOps:
         out.copy_(_act(x, act).to(out.dtype))
 
     # ------------------------------------------------------------------ attention over a cached latent
-    def head_products(self, x, w, out):
-        out.copy_(torch.einsum("thk,hnk->thn", x.to(self.cd), w.to(self.cd)).to(out.dtype))
+    def head_products(self, x, w, out, gate=None):
+        y = torch.einsum("thk,hnk->thn", x.to(self.cd), w.to(self.cd))
+        if gate is not None:
+            y = y * torch.sigmoid(gate.to(self.cd).sum(0)).view(y.shape)
+        out.copy_(y.to(out.dtype))
+
+    def latent_down(self, proj, q_rank, q_norm, pos, slot, cos, sin, rot_dims, style, norm_w, eps, c_q, cache, R, C, write_kv,
+                    status):
+        x = proj.to(self.cd).sum(0)
+        q = x[:, :q_rank]
+        c_q.copy_((q / torch.sqrt((q * q).mean(-1, keepdim=True) + eps) * q_norm.to(self.cd)).to(c_q.dtype))
+        if not write_kv:
+            return
+        T, p = x.shape[0], pos.long()
+        c = x[:, q_rank:q_rank + C]
+        row = torch.zeros(T, cache.k.shape[-1], dtype=self.cd)
+        row[:, :C] = c / torch.sqrt((c * c).mean(-1, keepdim=True) + eps) * norm_w.to(self.cd)
+        r = x[:, None, q_rank + C:q_rank + C + R]
+        row[:, C:C + R] = self._turn(r, cos[p].to(self.cd), sin[p].to(self.cd), style)[:, 0] if rot_dims else r[:, 0]
+        pages = cache.block_table[slot.long(), p // cache.page_size].long()
+        assert (pages >= 0).all(), "write to a position without a page"
+        cache.k[pages, 0, p % cache.page_size, :] = row.to(cache.k.dtype)
+
+    # ------------------------------------------------------------------ real-gated linear recurrent unit
+    def _rglru_ab(self, u, w_r, b_r, w_i, b_i, rate):
+        B, n = w_r.shape[0], w_r.shape[1]
+        ub = u.view(-1, B, n)
+        gate = lambda w, b: torch.sigmoid(torch.einsum("bij,tbj->tbi", w.to(self.cd), ub).reshape(u.shape) + b.to(self.cd))
+        a = torch.exp(rate.to(self.cd) * gate(w_r, b_r))
+        return a, torch.sqrt(1 - a * a) * gate(w_i, b_i) * u
+
+    def rglru_gates(self, u, w_r, b_r, w_i, b_i, rate, a, b, kernel=None):
+        ra, rb = self._rglru_ab(u.to(self.cd), w_r, b_r, w_i, b_i, rate)
+        a.copy_(ra.to(a.dtype))
+        b.copy_(rb.to(b.dtype))
+
+    def rglru_scan(self, a, b, y, slot, seq_start, n_seq, longest, state, out):
+        W = a.shape[1]
+        starts = list(range(n_seq + 1)) if seq_start is None else seq_start.tolist()
+        g = _act(y.to(self.cd), "gelu_pytorch_tanh")
+        for e in range(n_seq):
+            sl = int(slot[starts[e]])
+            S = state[sl, :W].to(self.cd).clone()
+            for t in range(starts[e], starts[e + 1]):
+                S = a[t].to(self.cd) * S + b[t].to(self.cd)
+                out[t] = (S * g[t]).to(out.dtype)
+            state[sl, :W] = S.to(state.dtype)
+
+    RGLRU_STEP_BLOCK = 4096
+
+    def rglru_step(self, proj, bias, conv_w, conv_b, w_r, b_r, w_i, b_i, rate, pos, slot, state, out):
+        x = proj.to(self.cd).sum(0) + bias.to(self.cd)
+        W, taps = conv_w.shape
+        for t in range(x.shape[0]):
+            p, home = int(pos[t]), state[int(slot[t])]
+            u = conv_b.to(self.cd) + conv_w[:, -1].to(self.cd) * x[t, W:]
+            for d in range(1, taps):
+                if p - d >= 0:
+                    r = (p - d) % taps
+                    u = u + conv_w[:, taps - 1 - d].to(self.cd) * home[W + r * W:W + (r + 1) * W].to(self.cd)
+            a, b = self._rglru_ab(u[None], w_r, b_r, w_i, b_i, rate)
+            S = a[0] * home[:W].to(self.cd) + b[0]
+            home[:W] = S.to(home.dtype)
+            home[W + (p % taps) * W:W + (p % taps + 1) * W] = x[t, W:].to(home.dtype)
+            out[t] = (S * _act(x[t, :W], "gelu_pytorch_tanh")).to(out.dtype)
 
     def latent_prepare(self, proj, pos, slot, cos, sin, rot_dims, style, norm_w, eps, q_plain, qa, cache, H, D, R, C,
                        write_kv, status):
@@ -639,7 +728,7 @@ class RefOps:
         assert (pages >= 0).all(), "write to a position without a page"
         cache.k[pages, 0, p % P, :] = row.to(cache.k.dtype)
 
-    def latent_attention(self, qa, cache, step, out, H, C, window, scale, splits=None, rows=None):
+    def latent_attention(self, qa, cache, step, out, H, C, window, scale, splits=None, rows=None, sinks=None):
         T, Dk = qa.shape[0], qa.shape[2]
         P = cache.page_size
         for t in (range(T) if rows is None else rows.tolist()):
@@ -650,7 +739,9 @@ class RefOps:
             assert (pages >= 0).all(), f"row {t}: key without a page"
             k = cache.k[pages, 0, js % P, :].to(self.cd)            # [n, row]
             s = (qa[t].to(self.cd) @ k[:, :Dk].T) * scale            # [H, n]
-            out[t] = (torch.softmax(s, -1) @ k[:, :C]).to(out.dtype)
+            if sinks is not None:
+                s = torch.cat([s, sinks.to(self.cd)[:, None]], -1)
+            out[t] = (torch.softmax(s, -1)[:, :k.shape[0]] @ k[:, :C]).to(out.dtype)
 
     def pair_embed_add(self, ids, pos, slot, last, table, out, mul_prev, mul_cur, fed_rows=None, fed_from=None):
         ids = ids.long().clone()
@@ -720,13 +811,16 @@ class RefOps:
     def moe_plan(self, expert_ids, n_experts, tile_rows):
         ids = expert_ids.reshape(-1).long()
         n = ids.numel()
-        counts = torch.bincount(ids, minlength=n_experts)
+        counts = torch.bincount(ids, minlength=n_experts)[:n_experts]
         offsets = torch.zeros(n_experts + 1, dtype=torch.long)
         offsets[1:] = torch.cumsum(counts, 0)
         order = torch.argsort(ids, stable=True)
         row_of = torch.empty(n, dtype=torch.long)
         row_of[order] = torch.arange(n)
-        token_of = order // (expert_ids.shape[-1] if expert_ids.dim() > 1 else 2)
+        per = expert_ids.shape[-1] if expert_ids.dim() > 1 else 2
+        token_of = order // per
+        row_of[ids >= n_experts] = n + (torch.arange(n) // per)[ids >= n_experts]      # identity experts
+        token_of[int(offsets[-1]):] = -1
         tiles_e, tiles_r = [], []
         for e in range(n_experts):
             for r in range(0, int(counts[e]), tile_rows):
@@ -741,7 +835,9 @@ class RefOps:
 
     def moe_dispatch(self, expert_ids, n_experts, tile_rows, x):
         plan = self.moe_plan(expert_ids, n_experts, tile_rows)
-        return plan, x[plan.token_of.long()].clone()
+        xs = torch.empty((plan.token_of.numel(), x.shape[1]), dtype=x.dtype)
+        self.gather_rows(x, plan.token_of, xs)
+        return plan, xs
 
     # ------------------------------------------------------------------ sampling
     def argmax(self, logits, out):
