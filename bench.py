@@ -731,6 +731,111 @@ def run_dumizen_pair(args, pk, rng):
     return out
 
 
+def sinilorn_config(width, heads, dim, rot, vdim, kv_rank, q_rank, window, streams, unit, blocks, ff, experts, identity, top,
+                    dense_ff, layers, vocab, taps=4):
+    """A Sinilorn configuration of ``layers`` layers: recurrent unit, latent attention with rows of its own, recurrent unit,
+    latent attention that reads the rows two layers before it, ...; the recurrent layers with the dense feed-forward, the
+    others with the mixture of experts."""
+    out = []
+    for i in range(layers):
+        if i % 2 == 0:
+            out.append({"type": "rglru", "mixer": {"width": unit, "blocks": blocks, "conv": taps}, "mlp": {"kind": "dense", "ff": dense_ff}})
+            continue
+        m = {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": vdim, "kv_rank": kv_rank, "q_rank": q_rank,
+             "scale": (dim + rot) ** -0.5, "rot": {"base": 5e5, "dims": rot, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+        if window:
+            m["mask"] = {"size": window}
+        if i % 4 == 3:
+            m["kv_from"] = i - 2
+        out.append({"type": "latent_attention", "mixer": m,
+                    "mlp": {"kind": "moe", "expert": {"ff": ff, "limit": 7.0}, "router": {"experts": experts, "identity": identity, "top": top}}})
+    return {"architecture": "Sinilorn", "vocab": vocab, "width": width, "streams": streams, "norm": {"eps": 1e-5}, "logit_scale": 1.0,
+            "layers": out}
+
+
+# layer sizes that resemble real models of this kind, beside a Puledra of equal width, heads, head sizes, latent and experts.
+# The first point's window is shorter than the prompt, the second's attention sees all of it, as Puledra's does.
+SINILORN_SIZES = {
+    "2048x16": dict(width=2048, heads=16, dim=128, rot=64, vdim=128, kv_rank=512, q_rank=1536, window=1024, streams=4, unit=2048, blocks=8,
+                    ff=1408, experts=64, identity=16, top=6, dense_ff=8192,
+                    puledra=dict(width=2048, heads=16, dim=128, rot=64, vdim=128, kv_rank=512, ff=1408, experts=64, top=6, groups=8, keep=3)),
+    "4096x32": dict(width=4096, heads=32, dim=128, rot=64, vdim=128, kv_rank=512, q_rank=1536, window=0, streams=4, unit=4096, blocks=16,
+                    ff=960, experts=16, identity=4, top=2, dense_ff=12288,
+                    puledra=dict(width=4096, heads=32, dim=128, rot=64, vdim=128, kv_rank=512, ff=960, experts=16, top=2, groups=1, keep=1)),
+}
+
+
+def run_sinilorn_pair(args, pk, rng):
+    """Prefill and decode of Sinilorn at layer sizes that resemble real models, beside Puledra at equal width, heads, latent
+    and experts: tokens/s, every kernel's time a layer of its kind, and the distance from the roofline of the attention
+    kernels (decode: cache bytes over the measured copy bandwidth; prefill: flops over the sustained library product
+    rate), of the recurrence and of the row kernel (bytes over the copy bandwidth) and of the block-diagonal gates
+    (flops of the products as float32 over the sustained product rate)."""
+    import torch
+    layers = args.layers or 8
+    vocab = args.vocab or 32064
+    batch, ctx = args.batch, args.prompt_tokens
+    out = {"design": "Sinilorn", "beside": "Puledra", "layers": layers, "batch": batch, "prompt_tokens": ctx, "dtype": "bf16",
+           "data": "synthetic: seeded random weights, uniform-random token ids",
+           "peaks": {k: pk[k] for k in ("hbm_gbs", "bf16_tflops_sustained", "source")}, "sizes": {}}
+    for name, sz in SINILORN_SIZES.items():
+        if args.design_sizes and name not in args.design_sizes:
+            continue
+        cfgs = {"sinilorn": sinilorn_config(**{k: v for k, v in sz.items() if k != "puledra"}, layers=layers, vocab=vocab),
+                "puledra": puledra_config(**sz["puledra"], layers=layers, vocab=vocab)}
+        row = {}
+        for which, cfg in cfgs.items():
+            cfg.setdefault("vocab_size", cfg.get("vocab"))
+            model = build_model(cfg, max(batch, 1), ctx + 256)
+            pre_ms = run_prefill(model, cfg, ctx, reps=3, warmup=3, rng=rng)
+            dec = run_decode(model, cfg, batch, ctx, args.steps, max(args.warmup, 3), rng, count_experts=False)
+            pre_t, dec_t, _ = profile_tables(model, cfg, batch, ctx, rng)
+            kv = ctx + 2
+            mixers = [l.parts["mixer"] for l in model.layers]
+            att = next(m for m in mixers if hasattr(m, "row_w"))
+            n_att = sum(1 for m in mixers if hasattr(m, "row_w"))
+            seen = lambda k: min(k, att.window) if att.window else k
+            att_bytes = batch * seen(kv) * att.row_w * 2
+            att_flops = sum(2 * att.H * (att.Dk + att.C) * seen(k) for k in range(1, ctx + 1))
+            unit = next((m for m in mixers if hasattr(m, "blocks")), None)
+            W, S = cfg["width"], cfg.get("streams", 1)
+            kern = {}
+            for kind, table in (("prefill", pre_t), ("decode", dec_t)):
+                rows = ctx if kind == "prefill" else batch
+                for kname, (n, ms) in sorted(table.items()):
+                    recurrent = kname.startswith(("flint_rglru", "flint_short_conv"))
+                    latent = kname.startswith(("flint_latent", "flint_head_products"))
+                    per = layers - n_att if recurrent else n_att if latent else layers
+                    secs = ms / per * 1e-3
+                    e = {"launches": n, "us_per_layer": round(ms * 1000.0 / per, 2)}
+                    if kname.startswith("flint_latent_attention"):
+                        if kind == "decode":
+                            e["frac_of_copy_bandwidth"] = round(att_bytes / secs / 1e9 / pk["hbm_gbs"], 4)
+                        else:
+                            e["frac_of_sustained_product_rate"] = round(att_flops / secs / (pk["bf16_tflops_sustained"] * 1e12), 4)
+                    elif kname.startswith("flint_rglru_gates"):
+                        e["frac_of_sustained_product_rate"] = round(rows * unit.W * (unit.W // unit.blocks) * 4 / secs / (pk["bf16_tflops_sustained"] * 1e12), 4)
+                        e["frac_of_copy_bandwidth"] = round(rows * unit.W * 12 / secs / 1e9 / pk["hbm_gbs"], 4)
+                    elif kname.startswith("flint_rglru_scan"):            # a, b, y in, the output out; the state in and out
+                        e["frac_of_copy_bandwidth"] = round(rows * unit.W * 14 / secs / 1e9 / pk["hbm_gbs"], 4)
+                    elif kname.startswith("flint_rglru_step"):            # both gates' blocks, the state and the ring in and out
+                        e["frac_of_copy_bandwidth"] = round((2 * unit.W * (unit.W // unit.blocks) * 2 + rows * unit.W * (2 + unit.taps) * 4 + rows * unit.W * 10)
+                                                            / secs / 1e9 / pk["hbm_gbs"], 4)
+                    elif kname.startswith("flint_row_norm"):              # streams in and out, what is pending (one set of sums), the normed row
+                        halves = n - 1
+                        e["us_per_launch"] = round(ms * 1000.0 / n, 2)
+                        if kind == "prefill":
+                            e["frac_of_copy_bandwidth"] = round(rows * W * (8 * S + 4 + 2) * halves / (ms * 1e-3) / 1e9 / pk["hbm_gbs"], 4)
+                    kern[f"{kind}: {kname}"] = e
+            row[which] = {"prefill_tok_s": round(ctx * 1000.0 / pre_ms, 1), "prefill_ms": round(pre_ms, 3),
+                          "decode_tok_s": round(dec["tok_s"], 1), "decode_ms_per_step": round(dec["ms"], 4),
+                          "decode_launches": dec["launches"], "weight_gb": round(model.weight_bytes() / 1e9, 2), "kernels": kern}
+            del model
+            torch.cuda.empty_cache()
+        out["sizes"][name] = row
+    return out
+
+
 def run_design_pair(args, pk, rng):
     """Prefill and decode of Puledra or Gepadra at layer sizes that resemble real models, beside Phi-MoE at equal width, heads
     and active expert parameters: tokens/s, and for the attention kernels of both the time a layer and the
@@ -1051,9 +1156,9 @@ def main():
     ap.add_argument("--sweep", action="store_true",
                     help="instead of the default run: decode at batch 1 and 8 with contexts of 16,384 and 65,536 tokens, "
                          "batch 1 with 131,008, and batch 128 and 256 with 2,048, each with its roofline fraction")
-    ap.add_argument("--design", choices=["puledra", "gepadra", "tefovik", "dumizen"], default=None,
+    ap.add_argument("--design", choices=["puledra", "gepadra", "tefovik", "dumizen", "sinilorn"], default=None,
                     help="prefill and decode of this design at layer sizes that resemble real models, beside the closest "
-                         "earlier model at equal sizes (Phi-MoE; for tefovik and dumizen Gepadra), with its kernels' shares of the peaks")
+                         "earlier model at equal sizes (Phi-MoE; for tefovik and dumizen Gepadra, for sinilorn Puledra), with its kernels' shares of the peaks")
     ap.add_argument("--design-sizes", nargs="+", default=None, help="which of the design's size points to run")
     ap.add_argument("--profile", action="store_true",
                     help="print per-kernel device times of one prefill and one decode step to stderr and exit")
@@ -1085,7 +1190,7 @@ def main():
         print(json.dumps(run_tiny(args.tiny)))
         return 0
     if args.design:
-        run = {"tefovik": run_tefovik_pair, "dumizen": run_dumizen_pair}.get(args.design, run_design_pair)
+        run = {"tefovik": run_tefovik_pair, "dumizen": run_dumizen_pair, "sinilorn": run_sinilorn_pair}.get(args.design, run_design_pair)
         print(json.dumps(run(args, pk, rng)))
         return 0
     if args.sweep:

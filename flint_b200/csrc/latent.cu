@@ -32,6 +32,15 @@ constexpr int GC = 4;           // heads per warp
 constexpr int WARPS = 4;
 constexpr int MAX_DPL = 16;     // output dims per lane: latent size <= 512
 
+__device__ __forceinline__ void store4(float* dst, float4 v) { *reinterpret_cast<float4*>(dst) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* dst, float4 v) {
+  const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+  uint2 w;
+  w.x = *reinterpret_cast<const uint32_t*>(&lo);
+  w.y = *reinterpret_cast<const uint32_t*>(&hi);
+  *reinterpret_cast<uint2*>(dst) = w;
+}
+
 // One column's partial sums, added in order with up to eight loads in flight.
 __device__ __forceinline__ float sum_partials(const float* col, int n_partials, long long stride) {
   float s = 0.f;
@@ -87,15 +96,16 @@ latent_prepare_kernel(const float* __restrict__ proj, int n_partials, long long 
                       const float* __restrict__ cos_t, const float* __restrict__ sin_t, int rot_dims, int interleaved,
                       const float* __restrict__ norm_w, float eps, TQ* __restrict__ q_plain, TQ* __restrict__ qa,
                       TC* __restrict__ k_cache, const int* __restrict__ block_table, int max_pages, int page_size,
-                      int H, int D, int R, int C, int row_w, int write_kv, int* __restrict__ status) {
+                      int H, int D, int R, int C, int row_w, int write_kv, int vec, int* __restrict__ status) {
   extern __shared__ float sm[];         // C floats of the latent before its norm
   __shared__ float red[32];
   pdl_launch();
   const int t = blockIdx.x;
   const int p = pos[t];
+  const bool writes = write_kv && blockIdx.y == gridDim.y - 1;
   long long cache_row = -1;
   bool missing = false;
-  if (write_kv) {
+  if (writes) {
     const int page = block_table[(size_t)slot[t] * max_pages + p / page_size];
     if (page >= 0) cache_row = (long long)page * page_size + p % page_size;
     else missing = true;
@@ -111,11 +121,26 @@ latent_prepare_kernel(const float* __restrict__ proj, int n_partials, long long 
     if (interleaved) { d0 = 2 * u; d1 = 2 * u + 1; }
     else { d0 = u; d1 = u + half; }
   };
-  for (int i = threadIdx.x; i < H * D; i += blockDim.x) {
-    const int h = i / D, d = i - h * D;
-    q_plain[((size_t)t * H + h) * D + d] = from_f32<TQ>(total(h * DR + d));
+  const int first = blockIdx.y * blockDim.x + threadIdx.x, stride = gridDim.y * blockDim.x;
+  if (vec) {                    // four neighbouring dims at a time
+    const int D4 = D / 4;
+    for (int i = first; i < H * D4; i += stride) {
+      const int h = i / D4, d = 4 * (i - h * D4);
+      const float* src = row + h * DR + d;
+      float4 v = *reinterpret_cast<const float4*>(src);
+      for (int z = 1; z < n_partials; ++z) {
+        const float4 o = *reinterpret_cast<const float4*>(src + (size_t)z * partial_stride);
+        v.x += o.x; v.y += o.y; v.z += o.z; v.w += o.w;
+      }
+      store4(q_plain + ((size_t)t * H + h) * D + d, v);
+    }
+  } else {
+    for (int i = first; i < H * D; i += stride) {
+      const int h = i / D, d = i - h * D;
+      q_plain[((size_t)t * H + h) * D + d] = from_f32<TQ>(total(h * DR + d));
+    }
   }
-  for (int i = threadIdx.x; i < H * units; i += blockDim.x) {
+  for (int i = first; i < H * units; i += stride) {
     const int h = i / units, u = i - h * units;
     const int src = h * DR + D;
     TQ* dst = qa + ((size_t)t * H + h) * Dk + C;
@@ -131,27 +156,28 @@ latent_prepare_kernel(const float* __restrict__ proj, int n_partials, long long 
       dst[d] = from_f32<TQ>(total(src + d));
     }
   }
-  if (!write_kv) return;
+  if (!writes) return;
   write_latent_row(total, H * DR, norm_w, eps, cos_t, sin_t, rot_dims, interleaved, p, cache_row, k_cache, R, C, row_w, sm, red);
 }
 
 // proj [S][T, W], columns [q latent (Q) | latent (C) | rotated key part (R) | ...]: c_q = rmsnorm(q latent) out, and, with
-// write_kv, the token's cache row.  One block per row.
+// write_kv, the token's cache row.  Blocks (row, 0) make c_q, blocks (row, 1) the cache row.
 template <typename TQ, typename TC>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(512)
 latent_down_kernel(const float* __restrict__ proj, int n_partials, long long partial_stride, int W, int Q,
                    const float* __restrict__ q_norm, const int* __restrict__ pos, const int* __restrict__ slot,
                    const float* __restrict__ cos_t, const float* __restrict__ sin_t, int rot_dims, int interleaved,
                    const float* __restrict__ norm_w, float eps, TQ* __restrict__ c_q, TC* __restrict__ k_cache,
                    const int* __restrict__ block_table, int max_pages, int page_size, int R, int C, int row_w,
                    int write_kv, int* __restrict__ status) {
-  extern __shared__ float sm[];         // Q floats of the q latent, then C of the latent, before their norms
+  extern __shared__ float sm[];         // Q floats of the q latent, or C of the latent, before their norms
   __shared__ float red[32];
   pdl_launch();
   const int t = blockIdx.x, p = pos[t];
+  const bool writes = write_kv && blockIdx.y == 1;
   long long cache_row = -1;
   bool missing = false;
-  if (write_kv) {
+  if (writes) {
     const int page = block_table[(size_t)slot[t] * max_pages + p / page_size];
     if (page >= 0) cache_row = (long long)page * page_size + p % page_size;
     else missing = true;
@@ -160,6 +186,10 @@ latent_down_kernel(const float* __restrict__ proj, int n_partials, long long par
   if (missing && threadIdx.x == 0) atomicExch(status, 1);
   const float* row = proj + (size_t)t * W;
   auto total = [&](int col) { return sum_partials(row + col, n_partials, partial_stride); };
+  if (writes) {
+    write_latent_row(total, Q, norm_w, eps, cos_t, sin_t, rot_dims, interleaved, p, cache_row, k_cache, R, C, row_w, sm, red);
+    return;
+  }
   float ss = 0.f;
   for (int i = threadIdx.x; i < Q; i += blockDim.x) {
     const float v = total(i);
@@ -169,8 +199,6 @@ latent_down_kernel(const float* __restrict__ proj, int n_partials, long long par
   ss = block_sum(ss, red);
   const float inv = 1.0f / sqrtf(ss / (float)Q + eps);
   for (int i = threadIdx.x; i < Q; i += blockDim.x) c_q[(size_t)t * Q + i] = from_f32<TQ>(sm[i] * inv * q_norm[i]);
-  if (!write_kv) return;
-  write_latent_row(total, Q, norm_w, eps, cos_t, sin_t, rot_dims, interleaved, p, cache_row, k_cache, R, C, row_w, sm + Q, red);
 }
 
 template <typename TQ, typename TC, typename TO>
@@ -764,10 +792,15 @@ extern "C" int flint_latent_prepare(const float* proj, int n_partials, long long
   const int W = H * (D + R) + (write_kv ? C + R : 0);
   const size_t smem = (size_t)C * sizeof(float);
   if (smem > 48 * 1024) return fail("latent_prepare: latent size %d is too large", C);
+  const int vec = D % 4 == 0 && R % 4 == 0 && W % 4 == 0 && partial_stride % 4 == 0 && !((uintptr_t)proj & 15) && !((uintptr_t)q_plain & 15);
+  // few rows: several blocks share one, so that the device is filled
+  int per_row = T >= 148 ? 1 : (148 + T - 1) / T;
+  const int most = (H * (D / (vec ? 4 : 1)) + 255) / 256 + (write_kv ? 1 : 0);
+  if (per_row > most) per_row = most < 1 ? 1 : most;
   FLINT_DISPATCH_DTYPE(q_dtype, TQ, FLINT_DISPATCH_DTYPE(cache_dtype, TC,
-      (launch_pdl(latent_prepare_kernel<TQ, TC>, dim3(T), dim3(256), smem, stream, proj, n_partials, partial_stride, W,
+      (launch_pdl(latent_prepare_kernel<TQ, TC>, dim3(T, per_row), dim3(256), smem, stream, proj, n_partials, partial_stride, W,
                   pos, slot, cos_t, sin_t, rot_dims, interleaved, norm_w, eps, (TQ*)q_plain, (TQ*)qa, (TC*)k_cache,
-                  block_table, max_pages, page_size, H, D, R, C, row_w, write_kv, status))));
+                  block_table, max_pages, page_size, H, D, R, C, row_w, write_kv, vec, status))));
   return check_launch("latent_prepare");
 }
 
@@ -901,10 +934,10 @@ extern "C" int flint_latent_down(const float* proj, int n_partials, long long pa
   if (rot_dims < 0 || rot_dims > R || (rot_dims & 1)) return fail("latent_down: %d rotating dims do not fit %d", rot_dims, R);
   if (write_kv && (row_w < C + R || (row_w & 7))) return fail("latent_down: cache rows of %d numbers do not hold %d", row_w, C + R);
   if (write_kv && (!k_cache || !norm_w || page_size <= 0)) return fail("latent_down: no cache to write to");
-  const size_t smem = (size_t)(Q + C) * sizeof(float);
+  const size_t smem = (size_t)(Q > C ? Q : C) * sizeof(float);
   if (smem > 48 * 1024) return fail("latent_down: latents of %d and %d numbers are too large", Q, C);
   FLINT_DISPATCH_DTYPE(q_dtype, TQ, FLINT_DISPATCH_DTYPE(cache_dtype, TC,
-      (launch_pdl(latent_down_kernel<TQ, TC>, dim3(T), dim3(256), smem, stream, proj, n_partials, partial_stride, W, Q,
+      (launch_pdl(latent_down_kernel<TQ, TC>, dim3(T, write_kv ? 2 : 1), dim3(T >= 148 ? 256 : 512), smem, stream, proj, n_partials, partial_stride, W, Q,
                   q_norm, pos, slot, cos_t, sin_t, rot_dims, interleaved, norm_w, eps, (TQ*)c_q, (TC*)k_cache, block_table,
                   max_pages, page_size, R, C, row_w, write_kv, status))));
   return check_launch("latent_down");

@@ -64,6 +64,53 @@ __global__ void short_conv_kernel(const float* __restrict__ u, long long in_stri
   }
 }
 
+// The same for many rows of whole 16-byte units: a block takes CONV_ROWS rows, a thread four neighbouring channels, whose
+// weights stay in registers; the rows a convolution shares with its neighbours come from L1.  The same sums in the same
+// order.
+constexpr int CONV_ROWS = 8, CONV_TAPS = 8;
+__global__ void __launch_bounds__(128)
+short_conv_rows_kernel(const float* __restrict__ u, long long in_stride, int col0, const float* __restrict__ w,
+                       const float* __restrict__ bias, int act, const int* __restrict__ pos, const int* __restrict__ slot,
+                       const float* __restrict__ ring, long long ring_stride, float* __restrict__ y, int T, int C, int taps,
+                       int R) {
+  __shared__ int have_s[CONV_ROWS], pos_s[CONV_ROWS];
+  pdl_launch();
+  pdl_wait();
+  const int t0 = blockIdx.x * CONV_ROWS, nt = min(CONV_ROWS, T - t0);
+  if (threadIdx.x < nt) {
+    const int t = t0 + threadIdx.x;
+    int have = 0;
+    while (have < taps - 1 && same_request(pos, slot, t, have + 1, T)) ++have;
+    have_s[threadIdx.x] = have;
+    pos_s[threadIdx.x] = pos[t];
+  }
+  __syncthreads();
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * 4;
+  if (c >= C) return;
+  float4 wt[CONV_TAPS];                       // the tap d positions back
+#pragma unroll
+  for (int d = 0; d < CONV_TAPS; ++d) {
+    const float* p = w + (size_t)c * taps + (taps - 1 - d);
+    wt[d] = d < taps ? make_float4(p[0], p[taps], p[2 * taps], p[3 * taps]) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  const float4 b = bias ? *reinterpret_cast<const float4*>(bias + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int r = 0; r < nt; ++r) {
+    const int t = t0 + r, p = pos_s[r], have = have_s[r];
+    const float* row = u + (size_t)t * in_stride + col0 + c;
+    float4 acc = b;
+#pragma unroll
+    for (int d = CONV_TAPS - 1; d >= 0; --d) {
+      if (d >= taps || p - d < 0) continue;
+      const float* src = d <= have ? row - (long long)d * in_stride : ring + (size_t)slot[t] * ring_stride + (size_t)((p - d) % R) * C + c;
+      const float4 x = *reinterpret_cast<const float4*>(src);
+      acc.x = fmaf(wt[d].x, x.x, acc.x); acc.y = fmaf(wt[d].y, x.y, acc.y);
+      acc.z = fmaf(wt[d].z, x.z, acc.z); acc.w = fmaf(wt[d].w, x.w, acc.w);
+    }
+    if (act == 1) acc = make_float4(siluf_(acc.x), siluf_(acc.y), siluf_(acc.z), siluf_(acc.w));
+    *reinterpret_cast<float4*>(y + (size_t)t * C + c) = acc;
+  }
+}
+
 // The inputs that outlive the step: a row that is among the last taps - 1 of its request's rows stores its input.
 __global__ void short_conv_keep_kernel(const float* __restrict__ u, long long in_stride, int col0,
                                        const int* __restrict__ pos, const int* __restrict__ slot, float* __restrict__ ring,
@@ -700,8 +747,14 @@ extern "C" int flint_short_conv(const float* u, long long in_stride, int col0, c
   // few rows (decoded tokens): a thread a channel, so that the rows spread over the chip; many rows: four channels a thread
   const int threads = C >= 1024 ? 256 : 128, per = T >= 256 ? 4 : 1;
   const dim3 grid((unsigned)T, (unsigned)min((C + threads * per - 1) / (threads * per), 65535));
-  launch_pdl(short_conv_kernel, grid, dim3(threads), 0, stream, u, in_stride, col0, w, bias, act, pos, slot,
-             (const float*)ring, ring_stride, y, T, C, taps, ring_rows);
+  const bool lined = C % 4 == 0 && col0 % 4 == 0 && in_stride % 4 == 0 && ring_stride % 4 == 0 &&
+                     !(((uintptr_t)u | (uintptr_t)ring | (uintptr_t)y | (uintptr_t)bias) & 15);
+  if (T >= 128 && taps <= CONV_TAPS && lined)
+    launch_pdl(short_conv_rows_kernel, dim3((unsigned)((T + CONV_ROWS - 1) / CONV_ROWS), (unsigned)((C + 511) / 512)), dim3(128), 0,
+               stream, u, in_stride, col0, w, bias, act, pos, slot, (const float*)ring, ring_stride, y, T, C, taps, ring_rows);
+  else
+    launch_pdl(short_conv_kernel, grid, dim3(threads), 0, stream, u, in_stride, col0, w, bias, act, pos, slot,
+               (const float*)ring, ring_stride, y, T, C, taps, ring_rows);
   if (taps > 1)
     launch_pdl(short_conv_keep_kernel, grid, dim3(threads), 0, stream, u, in_stride, col0, pos, slot, ring, ring_stride, T, C,
                taps, ring_rows);

@@ -285,129 +285,163 @@ __global__ void rglru_walk_kernel(const float* __restrict__ a, const float* __re
 }
 
 // ------------------------------------------------------------------------------------------- single tokens
-// Block: SO outputs of one diagonal block for up to ST tokens.  Every warp forms the sums of SO / 8 outputs, both gates,
-// for all the block's tokens: lanes share the channels of a weight row, a butterfly leaves every lane one sum or
-// two.
-constexpr int SO = 32, ST = 8, STEP_THREADS = 256;
+// Block: SO outputs of one diagonal block for up to ST tokens.  The threads first form the convolved input of the
+// block's channels, a channel a thread, all tokens' operands in flight together; then every warp forms both gates'
+// sums of SO / 8 outputs for all tokens: lanes share the channels of a weight row (asked for before the wait for the
+// projection while it fits: no kernel writes it), and a butterfly leaves every lane one sum.
+constexpr int SO = 32, ST = 4, STEP_THREADS = 256, OW = SO / 8;
+static_assert(OW * 2 * ST == 32, "one sum a lane");
 
 template <typename TW> struct Unit { static constexpr int N = 4; };
 template <> struct Unit<__nv_bfloat16> { static constexpr int N = 8; };
-__device__ __forceinline__ void load_unit(const float* p, float* f) {
-  const float4 v = *reinterpret_cast<const float4*>(p);
-  f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+__device__ __forceinline__ void unpack(const uint4 v, float* f, float) {
+  f[0] = __uint_as_float(v.x); f[1] = __uint_as_float(v.y); f[2] = __uint_as_float(v.z); f[3] = __uint_as_float(v.w);
 }
-__device__ __forceinline__ void load_unit(const __nv_bfloat16* p, float* f) { flint_attn::load8<__nv_bfloat16>(p, f); }
+__device__ __forceinline__ void unpack(const uint4 v, float* f, __nv_bfloat16) {
+  const uint32_t w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    f[2 * i] = __uint_as_float(w[i] << 16);
+    f[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+  }
+}
 
 template <typename TW, typename TO>
-__global__ void __launch_bounds__(STEP_THREADS)
+__global__ void __launch_bounds__(STEP_THREADS, 2)
 rglru_step_kernel(const float* __restrict__ proj, int n_partials, long long partial_stride, const float* __restrict__ bias,
                   const float* __restrict__ conv_w, const float* __restrict__ conv_b, int taps, const TW* __restrict__ wr,
                   const float* __restrict__ br, const TW* __restrict__ wi, const float* __restrict__ bi,
                   const float* __restrict__ rate, const int* __restrict__ pos, const int* __restrict__ slot,
                   float* __restrict__ state, long long state_stride, TO* __restrict__ out, int T, int W, int n, int vec) {
-  extern __shared__ float sm[];               // us [ST][n], then xs [ST][SO], then z [ST][SO][2]
+  extern __shared__ __align__(16) float sm[];  // us [ST][n], then xs [ST][SO], then z [ST][SO][2]
+  __shared__ long long home_s[ST];
+  __shared__ long long ring_s[64][ST];         // where the input d positions back lies (a tap that looks before the start: -1)
   float* us = sm;
   float* xs = us + (size_t)ST * n;
   float* z = xs + ST * SO;
+  constexpr int VN = Unit<TW>::N;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int slices = (n + SO - 1) / SO;
   const int blk = blockIdx.x / slices, o0 = (blockIdx.x % slices) * SO, t0 = blockIdx.y * ST;
   const int nt = min(ST, T - t0);
-  pdl_launch();
-  pdl_wait();
-  // the convolved input of the block's channels; beside it the raw input of this block's own outputs
-  for (int i = tid; i < nt * n; i += STEP_THREADS) {
-    const int tt = i / n, k = i - tt * n, t = t0 + tt, c = blk * n + k, p = pos[t];
-    const float* src = proj + (size_t)t * 2 * W + W + c;
-    float x = 0.f;
-    for (int q0 = 0; q0 < n_partials; q0 += 8) {
-      float v[8];
+  // the first (for short rows: the only) units of this warp's weight rows
+  uint4 first[OW][2];
 #pragma unroll
-      for (int q = 0; q < 8; ++q) v[q] = q0 + q < n_partials ? src[(size_t)(q0 + q) * partial_stride] : 0.f;
+  for (int j = 0; j < OW; ++j)
 #pragma unroll
-      for (int q = 0; q < 8; ++q) x += v[q];
+    for (int g = 0; g < 2; ++g) {
+      const int o = o0 + warp * OW + j;
+      first[j][g] = make_uint4(0u, 0u, 0u, 0u);
+      if (vec && o < n && lane * VN < n)
+        first[j][g] = *reinterpret_cast<const uint4*>((g ? wi : wr) + ((size_t)blk * n + o) * n + lane * VN);
     }
-    x += bias[W + c];
-    const float* ring = state + (size_t)slot[t] * state_stride + W + c;
-    float acc = conv_b[c];
-    for (int d = taps - 1; d >= 1; --d)
-      acc = fmaf(conv_w[(size_t)c * taps + taps - 1 - d], p - d >= 0 ? ring[(size_t)((p - d) % taps) * W] : 0.f, acc);
-    us[tt * n + k] = fmaf(conv_w[(size_t)c * taps + taps - 1], x, acc);
-    if (k >= o0 && k < o0 + SO) xs[tt * SO + k - o0] = x;
+  if (tid < ST) {
+    const int t = t0 + min(tid, nt - 1);
+    home_s[tid] = (long long)slot[t] * state_stride;
+  }
+  for (int i = tid; i < taps * ST; i += STEP_THREADS) {
+    const int d = i / ST, t = t0 + min(i % ST, nt - 1), p = pos[t];
+    ring_s[d][i % ST] = p >= d ? (long long)slot[t] * state_stride + W + (long long)((p - d) % taps) * W : -1;
   }
   __syncthreads();
-  constexpr int VN = Unit<TW>::N;
-#pragma unroll 1
-  for (int j = 0; j < SO / 8; ++j) {
-    const int o = o0 + warp * (SO / 8) + j;
-    if (o >= n) break;
-    const TW* rr = wr + ((size_t)blk * n + o) * n;
-    const TW* ir = wi + ((size_t)blk * n + o) * n;
-    float ar[ST], ai[ST];
+  pdl_launch();
+  pdl_wait();
+  for (int k = tid; k < n; k += STEP_THREADS) {
+    const int c = blk * n + k;
+    const float* src = proj + (size_t)t0 * 2 * W + W + c;
+    float x[ST], u[ST];
 #pragma unroll
-    for (int t = 0; t < ST; ++t) ar[t] = ai[t] = 0.f;
-    if (vec) {
-#pragma unroll 2
-      for (int k = lane * VN; k < n; k += 32 * VN) {
-        float r[VN], q[VN];
-        load_unit(rr + k, r);
-        load_unit(ir + k, q);
+    for (int t = 0; t < ST; ++t) { x[t] = 0.f; u[t] = conv_b[c]; }
+#pragma unroll 4
+    for (int q = 0; q < n_partials; ++q)
 #pragma unroll
-        for (int t = 0; t < ST; ++t)
-          if (t < nt) {
+      for (int t = 0; t < ST; ++t)
+        if (t < nt) x[t] += src[(size_t)q * partial_stride + (size_t)t * 2 * W];
+#pragma unroll 3
+    for (int d = taps - 1; d >= 1; --d) {
+      const float w = conv_w[(size_t)c * taps + taps - 1 - d];
 #pragma unroll
-            for (int v = 0; v < VN; v += 4) {
-              const float4 x = *reinterpret_cast<const float4*>(us + t * n + k + v);
-              ar[t] = fmaf(r[v], x.x, ar[t]); ar[t] = fmaf(r[v + 1], x.y, ar[t]);
-              ar[t] = fmaf(r[v + 2], x.z, ar[t]); ar[t] = fmaf(r[v + 3], x.w, ar[t]);
-              ai[t] = fmaf(q[v], x.x, ai[t]); ai[t] = fmaf(q[v + 1], x.y, ai[t]);
-              ai[t] = fmaf(q[v + 2], x.z, ai[t]); ai[t] = fmaf(q[v + 3], x.w, ai[t]);
-            }
-          }
-      }
-    } else {
-      for (int k = lane; k < n; k += 32) {
-        const float r = to_f32(rr[k]), q = to_f32(ir[k]);
-#pragma unroll
-        for (int t = 0; t < ST; ++t)
-          if (t < nt) {
-            ar[t] = fmaf(r, us[t * n + k], ar[t]);
-            ai[t] = fmaf(q, us[t * n + k], ai[t]);
-          }
-      }
+      for (int t = 0; t < ST; ++t)
+        if (t < nt && ring_s[d][t] >= 0) u[t] = fmaf(w, state[ring_s[d][t] + c], u[t]);
     }
-    // 2 ST = 16 sums over 32 lanes: each exchange halves how many a lane holds; lane l ends with the sum of index l / 2
-    float v[2 * ST];
+    const float w = conv_w[(size_t)c * taps + taps - 1], bx = bias[W + c];
 #pragma unroll
-    for (int t = 0; t < ST; ++t) { v[t] = ar[t]; v[ST + t] = ai[t]; }
-#pragma unroll
-    for (int m = 2 * ST / 2, bit = 16; m >= 1; m >>= 1, bit >>= 1) {
-      const bool up = lane & bit;
-#pragma unroll
-      for (int i = 0; i < m; ++i) {
-        const float give = up ? v[i] : v[i + m], keep = up ? v[i + m] : v[i];
-        v[i] = keep + __shfl_xor_sync(0xffffffffu, give, bit);
-      }
+    for (int t = 0; t < ST; ++t) {
+      x[t] += bx;
+      us[t * n + k] = t < nt ? fmaf(w, x[t], u[t]) : 0.f;
+      if (k >= o0 && k < o0 + SO) xs[t * SO + k - o0] = x[t];
     }
-    const float s = v[0] + __shfl_xor_sync(0xffffffffu, v[0], 1);
-    const int idx = lane >> 1;                // 0 .. ST - 1: the recurrence gate of token idx; then the input gate
-    if (!(lane & 1)) z[((idx % ST) * SO + warp * (SO / 8) + j) * 2 + idx / ST] = s;
   }
+  __syncthreads();
+  float acc[OW * 2 * ST];                     // index (j * 2 + gate) * ST + token
+#pragma unroll
+  for (int i = 0; i < OW * 2 * ST; ++i) acc[i] = 0.f;
+  if (vec) {
+    for (int k = lane * VN; k < n; k += 32 * VN) {
+      float w[OW][2][VN];
+#pragma unroll
+      for (int j = 0; j < OW; ++j)
+#pragma unroll
+        for (int g = 0; g < 2; ++g) {
+          const int o = min(o0 + warp * OW + j, n - 1);
+          const uint4 v = k == lane * VN ? first[j][g]
+                                         : *reinterpret_cast<const uint4*>((g ? wi : wr) + ((size_t)blk * n + o) * n + k);
+          unpack(v, w[j][g], TW());
+        }
+#pragma unroll
+      for (int t = 0; t < ST; ++t)
+#pragma unroll
+        for (int v = 0; v < VN; v += 4) {
+          const float4 x = *reinterpret_cast<const float4*>(us + t * n + k + v);
+#pragma unroll
+          for (int j = 0; j < OW; ++j)
+#pragma unroll
+            for (int g = 0; g < 2; ++g) {
+              float& s = acc[(j * 2 + g) * ST + t];
+              s = fmaf(w[j][g][v], x.x, s); s = fmaf(w[j][g][v + 1], x.y, s);
+              s = fmaf(w[j][g][v + 2], x.z, s); s = fmaf(w[j][g][v + 3], x.w, s);
+            }
+        }
+    }
+  } else {
+    for (int k = lane; k < n; k += 32)
+#pragma unroll
+      for (int j = 0; j < OW; ++j)
+#pragma unroll
+        for (int g = 0; g < 2; ++g) {
+          const int o = min(o0 + warp * OW + j, n - 1);
+          const float w = to_f32((g ? wi : wr)[((size_t)blk * n + o) * n + k]);
+#pragma unroll
+          for (int t = 0; t < ST; ++t) acc[(j * 2 + g) * ST + t] = fmaf(w, us[t * n + k], acc[(j * 2 + g) * ST + t]);
+        }
+  }
+  // 32 sums over 32 lanes: each exchange halves how many a lane holds; lane l ends with the sum of index l
+#pragma unroll
+  for (int m = 16; m >= 1; m >>= 1) {
+    const bool up = lane & m;
+#pragma unroll
+    for (int i = 0; i < m; ++i) {
+      const float give = up ? acc[i] : acc[i + m], keep = up ? acc[i + m] : acc[i];
+      acc[i] = keep + __shfl_xor_sync(0xffffffffu, give, m);
+    }
+  }
+  z[((lane % ST) * SO + warp * OW + lane / (2 * ST)) * 2 + (lane / ST) % 2] = acc[0];
   __syncthreads();
   for (int i = tid; i < nt * SO; i += STEP_THREADS) {
     const int tt = i / SO, j = i % SO, o = o0 + j, t = t0 + tt;
     if (o >= n) continue;
     const int c = blk * n + o;
+    const float* src = proj + (size_t)t * 2 * W + c;
+    float y = bias[c];
+#pragma unroll 4
+    for (int q = 0; q < n_partials; ++q) y += src[(size_t)q * partial_stride];
     float a, b;
     unit(z[i * 2] + br[c], z[i * 2 + 1] + bi[c], rate[c], us[tt * n + o], a, b);
-    float* home = state + (size_t)slot[t] * state_stride;
+    float* home = state + home_s[tt];
     const float S = fmaf(a, home[c], b);
     home[c] = S;
-    home[W + (size_t)(pos[t] % taps) * W + c] = xs[tt * SO + j];
-    const float* src = proj + (size_t)t * 2 * W + c;
-    float y = 0.f;
-    for (int q = 0; q < n_partials; ++q) y += src[(size_t)q * partial_stride];
-    out[(size_t)t * W + c] = from_f32<TO>(S * gelu_tanhf_(y + bias[c]));
+    state[ring_s[0][tt] + c] = xs[i];
+    out[(size_t)t * W + c] = from_f32<TO>(S * gelu_tanhf_(y));
   }
 }
 

@@ -374,11 +374,12 @@ class Model:
             owner = i if call.cache_of is None else call.cache_of
             carry = layer.block.forward(h, step, self.cache.view(owner), self.cache.state_of(i),
                                         writes_cache=call.cache_of is None, carry=carry)
-            if step.record is not None and spec.streams and carry is not None:
-                ops.apply_pending(h, carry)       # a test asked for what every call leaves: the streams are finished here
+            if spec.streams and step.record is not None and "rows_after" in step.record:
+                ops.apply_pending(h, carry)       # asked for what every call leaves (the streams' sum): finished here
                 carry = None
-            if step.record is not None and carry is None and history is None:
-                step.record.setdefault("rows_after", []).append(h.sum(1) if spec.streams else h.clone())
+                step.record["rows_after"].append(h.sum(1))
+            if step.record is not None and carry is None and history is None and not spec.streams:
+                step.record.setdefault("rows_after", []).append(h.clone())      # the rows as this call leaves them
             if history is not None:
                 if carry is not None:
                     ops.apply_pending(h, carry)
