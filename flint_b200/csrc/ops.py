@@ -583,11 +583,14 @@ class CudaOps:
                 return bn
         return 256
 
-    def moe_tile_rows(self, n_tokens, n_experts, weight_dtype, top=2):
-        """Row-tile size the plan should use for grouped products over these weights (``top`` choices a token)."""
+    def moe_tile_rows(self, n_tokens, n_experts, weight_dtype, top=2, sums=()):
+        """Row-tile size the plan should use for grouped products over these weights (``top`` choices a token; ``sums``:
+        how many numbers the products over the plan sum over).  A product that cannot run on the tensor cores takes
+        tiles of up to 64 rows, and all products over a plan share its tiles."""
         if weight_dtype != torch.bfloat16:
             return 64
-        return self.token_tile(-(-top * n_tokens // n_experts))
+        rows = self.token_tile(-(-top * n_tokens // n_experts))
+        return min(rows, 64) if any(k % 8 for k in sums) else rows
 
     def _gemm_tc(self, x, w, gated, out, bias, accumulate, act_code, plan, M, N, K, plan_ready=False, act_params=(0.0, 0.0)):
         if plan is not None:

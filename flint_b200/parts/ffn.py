@@ -165,7 +165,7 @@ class SparseMixerMoE(FeedForward):
             gates = torch.empty((T, 2), dtype=torch.float32, device=dev)
             logits = torch.empty((T, self.E), dtype=torch.float32, device=dev) if step.record is not None else None
             ops.router_sparsemixer(x[torch.float32], self.w_router, self.eps, ids, gates, logits)
-        plan, xs = ops.moe_dispatch(ids, self.E, ops.moe_tile_rows(T, self.E, self.w13.dtype), xa)
+        plan, xs = ops.moe_dispatch(ids, self.E, ops.moe_tile_rows(T, self.E, self.w13.dtype, sums=(self.hidden, self.inter)), xa)
         a = torch.empty((2 * T, self.inter), dtype=self.w13.dtype, device=dev)
         ops.gated_gemm(xs, self.w13, a, self.act, plan)
         y = torch.empty((2 * T, self.hidden), dtype=torch.float32, device=dev)
@@ -280,7 +280,7 @@ class GroupedTopKMoE(FeedForward):
             y = torch.empty(((k + (1 if self.identity else 0)) * T, self.hidden), dtype=torch.float32, device=dev)
         if self.identity and x[torch.float32].data_ptr() != y[k * T:].data_ptr():
             y[k * T:].copy_(x[torch.float32])
-        plan, xs = ops.moe_dispatch(ids, self.E, ops.moe_tile_rows(T, self.choices, self.w13.dtype, k), xa)
+        plan, xs = ops.moe_dispatch(ids, self.E, ops.moe_tile_rows(T, self.choices, self.w13.dtype, k, (self.hidden, self.inter)), xa)
         a = torch.empty((k * T, self.inter), dtype=self.w13.dtype, device=dev)
         kw = {} if self.act_params is None else {"act_params": self.act_params}
         ops.gated_gemm(xs, self.w13, a, self.act, plan, **kw)
@@ -412,7 +412,7 @@ class SigmoidTopKMoE(FeedForward):
             weights = torch.empty((T, k + extra), dtype=torch.float32, device=dev)
             logits = torch.empty((T, self.E + extra), dtype=torch.float32, device=dev) if step.record is not None else None
             ops.router_sigmoid(x[torch.float32], self.w_router, self.E, k, ids, scores, weights, logits)
-        plan, xs = ops.moe_dispatch(ids, self.E, ops.moe_tile_rows(T, self.E, self.w_up.dtype, k), xa)
+        plan, xs = ops.moe_dispatch(ids, self.E, ops.moe_tile_rows(T, self.E, self.w_up.dtype, k, (self.hidden, self.inter)), xa)
         a = torch.empty((k * T, self.inter), dtype=self.w_up.dtype, device=dev)
         ops.row_act(ops.gemm_partials(xs, self.w_up, plan=plan), a, self.act, row_of=plan.row_of, row_scale=scores)
         y = torch.empty(((k + extra) * T, self.hidden), dtype=torch.float32, device=dev)
@@ -443,7 +443,7 @@ class SigmoidTopKMoE(FeedForward):
             logits = torch.empty((T, self.E), dtype=torch.float32, device=dev) if step.record is not None else None
             ops.router_sigmoid_grouped(x[torch.float32], self.w_router, self.w_correction, k, self.groups, self.keep,
                                        self.normalize, self.router_scale, ids, gates, logits)
-        plan, xs = ops.moe_dispatch(ids, self.E, ops.moe_tile_rows(T, self.E, self.w_up.dtype, k), xa)
+        plan, xs = ops.moe_dispatch(ids, self.E, ops.moe_tile_rows(T, self.E, self.w_up.dtype, k, (self.hidden, self.inter)), xa)
         a = torch.empty((k * T, self.inter), dtype=self.w_up.dtype, device=dev)
         ops.row_act(ops.gemm_partials(xs, self.w_up, plan=plan), a, self.act)
         y = torch.empty((k * T, self.hidden), dtype=torch.float32, device=dev)

@@ -239,7 +239,7 @@ class RefOps:
                 res[t, h] = torch.softmax(s, 0) @ v[:, h // G, :]
         out.copy_(res.reshape(T, nq * hd).to(out.dtype))
 
-    def moe_tile_rows(self, n_tokens, n_experts, weight_dtype, top=2):
+    def moe_tile_rows(self, n_tokens, n_experts, weight_dtype, top=2, sums=()):
         return 64
 
     # ------------------------------------------------------------------ attention with kept first tokens and a sink
@@ -655,8 +655,8 @@ class RefOps:
         B, n = w_r.shape[0], w_r.shape[1]
         ub = u.view(-1, B, n)
         gate = lambda w, b: torch.sigmoid(torch.einsum("bij,tbj->tbi", w.to(self.cd), ub).reshape(u.shape) + b.to(self.cd))
-        a = torch.exp(rate.to(self.cd) * gate(w_r, b_r))
-        return a, torch.sqrt(1 - a * a) * gate(w_i, b_i) * u
+        log_a = rate.to(self.cd) * gate(w_r, b_r)
+        return torch.exp(log_a), torch.sqrt(-torch.expm1(2 * log_a)) * gate(w_i, b_i) * u
 
     def rglru_gates(self, u, w_r, b_r, w_i, b_i, rate, a, b, kernel=None):
         ra, rb = self._rglru_ab(u.to(self.cd), w_r, b_r, w_i, b_i, rate)
