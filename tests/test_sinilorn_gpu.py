@@ -83,8 +83,8 @@ def step_of(pos, slot, n_entries):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("C,R,H", [(40, 8, 5), (20, 6, 1), (96, 16, 6), (256, 64, 33)])
-@pytest.mark.parametrize("window", [0, 1, 7, 64, 72, 200])
+@pytest.mark.parametrize("C,R,H", [(40, 8, 5), (20, 6, 1), (104, 24, 7), (256, 64, 33)])
+@pytest.mark.parametrize("window", [0, 1, 7, 64, 77, 200])
 def test_latent_attention_with_sinks_finds_planted_keys(ops, dtype, C, R, H, window):
     """Single rows whose query points at one key (the row's own, the window's first, the one that has just left it, page
     borders, the first token), with sinks from negligible to dominant: a key too many or too few, or a sink that is
@@ -117,8 +117,8 @@ def test_latent_attention_with_sinks_finds_planted_keys(ops, dtype, C, R, H, win
             assert err.max().item() < (3e-5 if dtype == torch.float32 else 4e-2), (kernel, splits, rows[int(err.argmax())], err.max().item())
 
 
-@pytest.mark.parametrize("C,R,H", [(96, 16, 6), (48, 16, 1), (24, 8, 3), (512, 64, 16), (128, 32, 32)])
-@pytest.mark.parametrize("window", [0, 5, 64, 72, 128, 130])
+@pytest.mark.parametrize("C,R,H", [(104, 24, 7), (48, 16, 1), (24, 8, 3), (512, 64, 16), (128, 32, 32)])
+@pytest.mark.parametrize("window", [0, 5, 64, 77, 128, 130])
 def test_latent_attention_windows_over_tiles_of_tokens(ops, C, R, H, window):
     """Portions of prompts on the tensor cores: a block's tokens see a window each, so between them more keys than one
     window (a window of exactly a key tile, one more, one less than a multiple)."""
@@ -181,7 +181,7 @@ def test_the_latents_on_their_way_in(ops, dtype, T, Q, C, R, rot, H, D, S):
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("T", [1, 8, 16, 17, 150])
-@pytest.mark.parametrize("H,N,K,S", [(3, 24, 40, 1), (6, 80, 96, 4), (2, 7, 13, 3), (5, 33, 16, 2)])
+@pytest.mark.parametrize("H,N,K,S", [(3, 24, 40, 1), (7, 72, 104, 4), (2, 7, 13, 3), (5, 33, 16, 2)])
 def test_products_per_head_with_a_gate(ops, dtype, T, H, N, K, S):
     rn = gen(T + N)
     x, w, proj = rn(T, H, K).to(dtype), (rn(H, N, K) / math.sqrt(K)).to(dtype), rn(S, T, 5 + H * N)
@@ -335,7 +335,7 @@ def pend_on(p, device):
 
 
 @pytest.mark.parametrize("S", [1, 2, 3, 4, 6])
-@pytest.mark.parametrize("T,W", [(1, 192), (8, 2048), (16, 1024), (300, 200), (2048, 512), (5, 8192), (40, 37)])
+@pytest.mark.parametrize("T,W", [(1, 208), (8, 2048), (16, 1024), (300, 200), (2048, 512), (5, 8192), (40, 37)])
 def test_streams_are_mixed_and_normed(ops, S, T, W):
     """One kernel for the mixing of what is pending and the norm of the streams' weighted sum: a block a row, a cluster a
     row, many rows, widths and numbers of streams that go to the separate kernels; the additions alone; the final
@@ -366,8 +366,8 @@ def test_streams_are_mixed_and_normed(ops, S, T, W):
                 assert torch.equal(b.cpu(), x)
 
 
-@pytest.mark.parametrize("S,T,W", [(2, 1, 192), (4, 8, 2048), (3, 300, 200), (6, 40, 72), (4, 2048, 256), (2, 9, 38)])
-@pytest.mark.parametrize("E,top", [(12, 4), (80, 6), (5, 1)])
+@pytest.mark.parametrize("S,T,W", [(2, 1, 208), (4, 8, 2048), (3, 300, 200), (6, 40, 72), (4, 2048, 256), (2, 9, 38)])
+@pytest.mark.parametrize("E,top", [(13, 3), (80, 6), (5, 1)])
 def test_the_corrected_softmax_router_rides_on_the_streams_norm(ops, S, T, W, E, top):
     """The choice is exactly the rule applied to the logits the kernel reports, and those agree with the plain product;
     the weights are the scores without the correction."""
@@ -391,7 +391,7 @@ def test_the_corrected_softmax_router_rides_on_the_streams_norm(ops, S, T, W, E,
 
 
 # ------------------------------------------------------------------------------------------------ experts
-@pytest.mark.parametrize("T,E,identity,top", [(1, 2, 2, 3), (8, 8, 4, 4), (60, 3, 5, 4), (64, 4, 4, 4), (65, 4, 4, 4), (500, 16, 4, 2), (40, 1, 6, 2)])
+@pytest.mark.parametrize("T,E,identity,top", [(1, 2, 2, 3), (8, 10, 3, 4), (60, 3, 5, 4), (64, 4, 4, 4), (65, 4, 4, 4), (500, 16, 4, 2), (40, 1, 6, 2)])
 @pytest.mark.parametrize("kind", ["drawn", "all identity", "no identity"])
 def test_identity_experts_take_no_rows_of_the_plan(ops, T, E, identity, top, kind):
     if (kind == "all identity" and identity < top) or (kind == "no identity" and E < top):
@@ -420,7 +420,7 @@ def test_identity_experts_take_no_rows_of_the_plan(ops, T, E, identity, top, kin
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("M", [1, 8, 100, 130, 300])
-@pytest.mark.parametrize("N,K", [(40, 64), (96, 192), (23, 40), (17, 21)])
+@pytest.mark.parametrize("N,K", [(40, 64), (112, 208), (23, 40), (17, 21)])
 def test_gated_products_with_biases_and_clamps(ops, dtype, M, N, K):
     """Dense: biases of gate and up before the activation, plain and clamped; few rows (partial sums and an activation
     kernel) and many (the tile's epilogue)."""
@@ -439,7 +439,7 @@ def test_gated_products_with_biases_and_clamps(ops, dtype, M, N, K):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("T,E,identity,top,N,K", [(1, 4, 4, 2, 32, 64), (1, 2, 6, 4, 16, 64), (7, 8, 4, 4, 96, 192), (200, 8, 4, 4, 96, 192), (90, 3, 2, 3, 13, 40),
+@pytest.mark.parametrize("T,E,identity,top,N,K", [(1, 4, 4, 2, 32, 64), (1, 2, 6, 4, 16, 64), (7, 10, 3, 4, 112, 208), (200, 10, 3, 4, 112, 208), (90, 3, 2, 3, 13, 40),
                                                    (300, 2, 1, 2, 20, 36), (300, 2, 1, 2, 20, 40)])
 def test_a_mixture_with_identity_experts_beside_the_plain_one(ops, dtype, T, E, identity, top, N, K):
     """The whole part, from the normalised rows to the pending rows, beside the plain mixture following its choices; also
