@@ -232,17 +232,30 @@ __global__ void moe_plan_kernel(const int* __restrict__ expert_ids, int n_assign
 // Few assignments (decode): the plan and the gather of the rows in one launch.  Every block works the
 // (tiny) plan out again in shared memory, with ranks by position so that all blocks agree; block r then
 // copies the row of its token to sorted row r, and block 0 also writes the plan out.
+// scale (or null): the score of every assignment, which multiplies the row it sends: then x holds float32 rows and xs receives
+// their multiples as TO, else whole rows are copied 16 bytes at a time (row_vecs units a row).
 constexpr int DISPATCH_MAX = 256;      // assignments
+__device__ __forceinline__ void scaled4(float* dst, const float4 v, float s) {
+  *reinterpret_cast<float4*>(dst) = make_float4(v.x * s, v.y * s, v.z * s, v.w * s);
+}
+__device__ __forceinline__ void scaled4(__nv_bfloat16* dst, const float4 v, float s) {
+  const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x * s, v.y * s), hi = __floats2bfloat162_rn(v.z * s, v.w * s);
+  uint2 pk;
+  pk.x = *reinterpret_cast<const uint32_t*>(&lo);
+  pk.y = *reinterpret_cast<const uint32_t*>(&hi);
+  *reinterpret_cast<uint2*>(dst) = pk;
+}
+template <typename TO>
 __global__ void __launch_bounds__(256)
 moe_dispatch_kernel(const int* __restrict__ expert_ids, int n_assign, int E, int tile_rows,
                     int* __restrict__ counts, int* __restrict__ offsets, int* __restrict__ row_of,
                     int* __restrict__ token_of, int* __restrict__ tile_expert, int* __restrict__ tile_row0,
-                    int* __restrict__ n_tiles, int max_tiles, const uint4* __restrict__ x,
-                    uint4* __restrict__ xs, int row_vecs, int top) {
+                    int* __restrict__ n_tiles, int max_tiles, const void* __restrict__ x,
+                    void* __restrict__ xs, int row_vecs, int top, const float* __restrict__ scale) {
   __shared__ int ids[DISPATCH_MAX];
   __shared__ int cnt[MAX_E];
   __shared__ int off[MAX_E + 1];
-  __shared__ int my_token;
+  __shared__ int my_token, my_choice;
   pdl_launch();
   pdl_wait();
   const int tid = threadIdx.x;
@@ -291,15 +304,41 @@ moe_dispatch_kernel(const int* __restrict__ expert_ids, int n_assign, int E, int
       row_of[tid] = row;
       token_of[row] = tid / top;
     }
-    if (row == (int)blockIdx.x) my_token = tid / top;
+    if (row == (int)blockIdx.x) { my_token = tid / top; my_choice = tid; }
   }
   if (blockIdx.x == 0)
     for (int r = off[E] + tid; r < n_assign; r += blockDim.x) token_of[r] = -1;
   __syncthreads();
   if (my_token < 0) return;                     // a sorted row that no choice takes
-  const uint4* src = x + (size_t)my_token * row_vecs;
-  uint4* dst = xs + (size_t)blockIdx.x * row_vecs;
+  if (scale) {
+    const float s = scale[my_choice];
+    const float4* src = (const float4*)x + (size_t)my_token * row_vecs;
+    TO* dst = (TO*)xs + (size_t)blockIdx.x * row_vecs * 4;
+    for (int i = tid; i < row_vecs; i += blockDim.x) scaled4(dst + 4 * i, src[i], s);
+    return;
+  }
+  const uint4* src = (const uint4*)x + (size_t)my_token * row_vecs;
+  uint4* dst = (uint4*)xs + (size_t)blockIdx.x * row_vecs;
   for (int i = tid; i < row_vecs; i += blockDim.x) dst[i] = src[i];
+}
+
+// xs[row_of[a]] = scale[a] * x[a / top] for every assignment a (sorted rows of a plan; a token's identity choices, whose places
+// lie behind the n_assign sorted rows, send nothing).  One block per assignment.
+template <typename TO>
+__global__ void scatter_scaled_kernel(const float* __restrict__ x, const int* __restrict__ row_of, const float* __restrict__ scale,
+                                      TO* __restrict__ xs, int n_assign, int H, int top, int vec) {
+  pdl_launch();
+  pdl_wait();
+  const int a = blockIdx.x, row = row_of[a];
+  if (row >= n_assign) return;
+  const float s = scale[a];
+  const float* src = x + (size_t)(a / top) * H;
+  TO* dst = xs + (size_t)row * H;
+  if (vec) {
+    for (int i = threadIdx.x; i < H / 4; i += blockDim.x) scaled4(dst + 4 * i, reinterpret_cast<const float4*>(src)[i], s);
+  } else {
+    for (int i = threadIdx.x; i < H; i += blockDim.x) dst[i] = from_f32<TO>(src[i] * s);
+  }
 }
 }  // namespace
 
@@ -502,11 +541,12 @@ extern "C" int flint_moe_plan(const int* expert_ids, int n_assign, int E, int ti
 }
 
 // The plan of flint_moe_plan and xs[r, :] = x[token_of[r], :] in one launch, for up to 256 assignments and rows
-// of a multiple of 16 bytes (x and xs 16-byte aligned).
+// of a multiple of 16 bytes (x and xs 16-byte aligned).  With scale [n_assign] (then x is float32 and row_bytes its row):
+// xs[r, :] = scale[assignment of r] * x[token_of[r], :] in out_dtype.
 extern "C" int flint_moe_dispatch(const int* expert_ids, int n_assign, int E, int tile_rows, int* counts,
                                   int* offsets, int* row_of, int* token_of, int* tile_expert, int* tile_row0,
                                   int* n_tiles, int max_tiles, const void* x, void* xs, int row_bytes, int top,
-                                  cudaStream_t stream) {
+                                  const float* scale, int out_dtype, cudaStream_t stream) {
   if (n_assign <= 0) return 0;
   if (top < 1) return fail("moe_dispatch: %d choices a token", top);
   if (n_assign > DISPATCH_MAX) return fail("moe_dispatch: %d assignments (up to %d)", n_assign, DISPATCH_MAX);
@@ -516,10 +556,23 @@ extern "C" int flint_moe_dispatch(const int* expert_ids, int n_assign, int E, in
     return fail("moe_dispatch: tile map of %d entries is too small", max_tiles);
   if (row_bytes <= 0 || (row_bytes & 15) || ((uintptr_t)x & 15) || ((uintptr_t)xs & 15))
     return fail("moe_dispatch: rows must be a multiple of 16 bytes and 16-byte aligned");
-  launch_pdl(moe_dispatch_kernel, dim3(n_assign), dim3(256), 0, stream, expert_ids, n_assign, E, tile_rows, counts,
-             offsets, row_of, token_of, tile_expert, tile_row0, n_tiles, max_tiles, (const uint4*)x, (uint4*)xs,
-             row_bytes / 16, top);
+  FLINT_DISPATCH_DTYPE(out_dtype, TO,
+      launch_pdl(moe_dispatch_kernel<TO>, dim3(n_assign), dim3(256), 0, stream, expert_ids, n_assign, E, tile_rows, counts,
+                 offsets, row_of, token_of, tile_expert, tile_row0, n_tiles, max_tiles, x, xs, row_bytes / 16, top, scale));
   return check_launch("moe_dispatch");
+}
+
+// The rows of a plan, each multiplied by the score of the choice that sends it: x [*, H] float32, row_of and scale [n_assign],
+// xs [n_assign, H] in out_dtype.
+extern "C" int flint_scatter_scaled(const float* x, const int* row_of, const float* scale, void* xs, int out_dtype, int n_assign,
+                                    int H, int top, cudaStream_t stream) {
+  if (n_assign <= 0) return 0;
+  if (top < 1 || H < 1) return fail("scatter_scaled: %d choices a token of rows of %d", top, H);
+  const int vec = H % 4 == 0 && !(((uintptr_t)x | (uintptr_t)xs) & 15);
+  FLINT_DISPATCH_DTYPE(out_dtype, TO,
+      launch_pdl(scatter_scaled_kernel<TO>, dim3((unsigned)n_assign), dim3(H >= 1024 ? 256 : 128), 0, stream, x, row_of, scale,
+                 (TO*)xs, n_assign, H, top, vec));
+  return check_launch("scatter_scaled");
 }
 
 extern "C" const char* flint_moe_last_error() { return g_error; }

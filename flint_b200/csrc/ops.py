@@ -276,39 +276,117 @@ class CudaOps:
                 top = row_of.numel() // max(T, 1)
                 if y.shape[1] != H or top < 1 or row_of.numel() != top * T or gts.numel() != top * T:
                     raise KernelError("row_norm: pending expert rows do not match the residual")
-        wr = logits = None
-        E, jit, ids, gates = 0, 0.0, None, None
-        r_top, r_groups, r_keep, r_scale = 0, 1, 1, 1.0
-        r_rule, r_extra, r_aux = 0, 0, None
-        r_corr, r_norm = None, 0
-        if router is not None:
-            wr, E, jit, ids, gates = router.weight, router.weight.shape[0], router.jitter_eps, router.expert_ids, router.gates
-            logits = getattr(router, "logits", None)
-            r_top, r_groups = int(getattr(router, "top", 0)), int(getattr(router, "groups", 1))
-            r_keep, r_scale = int(getattr(router, "keep", 1)), float(getattr(router, "scale", 1.0))
-            if logits is not None:
-                _check(logits, "router logits", torch.float32, 2)
-                if tuple(logits.shape) != (T, E):
-                    raise KernelError(f"row_norm: router logits must be [{T}, {E}]")
-            _check(wr, "router weight", dims=2)
-            if wr.shape[1] != H or ids.numel() != (r_top or 2) * T or gates.numel() != (r_top or 2) * T:
-                raise KernelError("row_norm: router shapes do not match")
-            if getattr(router, "rule", "") == "sigmoid":
-                r_rule, r_extra, r_aux = 1, int(router.extra), router.weights
-                _check(r_aux, "router weights out", torch.float32, 2)
-                if tuple(r_aux.shape) != (T, r_top + r_extra) or r_top < 1:
-                    raise KernelError(f"row_norm: the sigmoid router's weights must be [{T}, {r_top + r_extra}]")
-            elif getattr(router, "rule", "") in ("sigmoid_grouped", "softmax_corrected"):
-                r_rule = 2 if router.rule == "sigmoid_grouped" else 3
-                r_corr, r_norm = router.correction, 1 if router.normalize else 0
-                if r_corr is not None and (r_corr.dtype != torch.float32 or r_corr.numel() != E):
-                    raise KernelError("row_norm: the router's correction must be float32, one per expert")
+        wr, E, jit, ids, gates, logits, rest = self._router_args(router, T, H, "row_norm")
         self._run("row_fused", "flint_row_norm", _ptr(x), _ptr(row_index), c_int(rows), c_int(H), _ptr(partials),
                   c_int(S), c_longlong(stride), _ptr(bias), _ptr(y), _ptr(row_of), _ptr(gts), c_int(top), _ptr(gamma), _ptr(beta),
                   c_float(eps), c_int({"layer": 0, "rms": 1}[mode]), _ptr(out_f32), _ptr(out_bf16), _ptr(wr),
                   c_int(_code(wr.dtype) if wr is not None else 0), c_int(E), c_float(jit), _ptr(ids), _ptr(gates),
-                  _ptr(logits), c_int(r_top), c_int(r_groups), c_int(r_keep), c_float(r_scale), c_int(r_rule), c_int(r_extra),
-                  _ptr(r_aux), _ptr(r_corr), c_int(r_norm), c_int(streams), _ptr(mix), _ptr(spread), _ptr(gather))
+                  _ptr(logits), *rest, c_int(streams), _ptr(mix), _ptr(spread), _ptr(gather))
+
+    @staticmethod
+    def _router_args(router, T, H, who):
+        """(weight, E, jitter_eps, ids, gates, logits, the launchers' remaining arguments) of a ``RouterRequest`` or None."""
+        wr = logits = aux = corr = ids = gates = None
+        E, jit, top, groups, keep, scale, rule, extra, normalize = 0, 0.0, 0, 1, 1, 1.0, 0, 0, 0
+        if router is not None:
+            wr, E, jit, ids, gates = router.weight, router.weight.shape[0], router.jitter_eps, router.expert_ids, router.gates
+            logits = getattr(router, "logits", None)
+            top, groups = int(getattr(router, "top", 0)), int(getattr(router, "groups", 1))
+            keep, scale = int(getattr(router, "keep", 1)), float(getattr(router, "scale", 1.0))
+            if logits is not None:
+                _check(logits, "router logits", torch.float32, 2)
+                if tuple(logits.shape) != (T, E):
+                    raise KernelError(f"{who}: router logits must be [{T}, {E}]")
+            _check(wr, "router weight", dims=2)
+            if wr.shape[1] != H or ids.numel() != (top or 2) * T or gates.numel() != (top or 2) * T:
+                raise KernelError(f"{who}: router shapes do not match")
+            if getattr(router, "rule", "") == "sigmoid":
+                rule, extra, aux = 1, int(router.extra), router.weights
+                _check(aux, "router weights out", torch.float32, 2)
+                if tuple(aux.shape) != (T, top + extra) or top < 1:
+                    raise KernelError(f"{who}: the sigmoid router's weights must be [{T}, {top + extra}]")
+            elif getattr(router, "rule", "") in ("sigmoid_grouped", "softmax_corrected"):
+                rule = 2 if router.rule == "sigmoid_grouped" else 3
+                corr, normalize = router.correction, 1 if router.normalize else 0
+                if corr is not None and (corr.dtype != torch.float32 or corr.numel() != E):
+                    raise KernelError(f"{who}: the router's correction must be float32, one per expert")
+        return wr, E, jit, ids, gates, logits, (c_int(top), c_int(groups), c_int(keep), c_float(scale), c_int(rule), c_int(extra),
+                                                _ptr(aux), _ptr(corr), c_int(normalize))
+
+    def row_post(self, x, pending=None, out=None, router=None, conv=None):
+        """x [T, H] float32 += what is pending, in place, with ``pending.gamma`` divided by its root mean square and scaled
+        first; ``out`` [T, H] (float32 or bfloat16) receives the new rows; ``router``: the routing of the new rows.  ``conv`` =
+        (w [H, taps], ring, pos, slot), for a batch of single tokens: ``out`` receives the new rows plus their convolution
+        over time, whose earlier rows lie in ``ring`` [slots, >= (taps - 1) H] (a view) as in ``short_conv``.  Widths that
+        the row kernel does not take go through separate kernels."""
+        _check(x, "x", torch.float32, 2)
+        T, H = x.shape
+        branches, rows = self._pending_branches(pending)
+        gamma, eps = (pending.gamma, pending.eps) if pending is not None else (None, 0.0)
+        if gamma is not None and (gamma.dtype != torch.float32 or gamma.numel() != H):
+            raise KernelError("row_post: scale must be float32 of the row width")
+        if out is not None:
+            _check(out, "out", dims=2)
+            if tuple(out.shape) != (T, H):
+                raise KernelError(f"row_post: out must be [{T}, {H}]")
+        if conv is not None:
+            w, ring, pos, slot = conv
+            _check(w, "conv weight", torch.float32, 2)
+            taps = w.shape[1]
+            if out is None or w.shape[0] != H:
+                raise KernelError("row_post: a convolution needs an output and taps for every channel")
+            if taps > 1:
+                _check(ring, "ring", torch.float32, 2, contiguous=False)
+                if ring.stride(1) != 1 or ring.shape[1] < (taps - 1) * H or pos.numel() != T or slot.numel() != T:
+                    raise KernelError("row_post: the convolution's state does not match")
+        if H % 4 or H > 16384 or (router is not None and not self._router_rides(router, H)):
+            if branches or rows is not None:
+                self.sum_norm_add(x, [b[:2] for b in branches], [b[2] for b in branches], expert_rows=rows, gamma=gamma, eps=eps)
+            if conv is not None:
+                self.short_conv(x, 0, w, None, "plus_input", pos, slot, ring, out)
+            elif out is not None:
+                self.cast_rows(x, out)
+            if router is not None:
+                self.route(x, router)
+            return
+        ptrs, strides, counts, biases = [], [], [], []
+        for part, bias, _ in branches:
+            _check(part, "partials", torch.float32, 3)
+            if tuple(part.shape[1:]) != (T, H) or (bias is not None and (bias.dtype != torch.float32 or bias.numel() != H)):
+                raise KernelError("row_post: pending partial sums do not match the rows")
+            ptrs.append(part.data_ptr())
+            strides.append(part.stride(0))
+            counts.append(part.shape[0])
+            biases.append(bias.data_ptr() if bias is not None else 0)
+        y = row_of = gts = None
+        top = 0
+        if rows is not None:
+            y, row_of, gts = rows
+            _check(y, "pending expert rows", torch.float32, 2)
+            top = row_of.numel() // max(T, 1)
+            if y.shape[1] != H or top < 1 or row_of.numel() != top * T or gts.numel() != top * T:
+                raise KernelError("row_post: pending expert rows do not match the rows")
+        n = len(branches)
+        arr = lambda ctype, vals: (ctype * max(n, 1))(*vals)
+        wr, E, _, ids, gates, logits, rest = self._router_args(router, T, H, "row_post")
+        conv_args = ((_ptr(w), c_int(taps), _ptr(ring if taps > 1 else None), c_longlong(ring.stride(0) if taps > 1 else 0), _ptr(pos),
+                      _ptr(slot)) if conv is not None else (_ptr(None), c_int(0), _ptr(None), c_longlong(0), _ptr(None), _ptr(None)))
+        self._run("row_fused", "flint_row_post", _ptr(x), c_int(T), c_int(H), c_int(n), arr(c_void_p, ptrs), arr(c_int, counts),
+                  arr(c_longlong, strides), arr(c_void_p, biases), arr(c_float, [float(b[2]) for b in branches]), _ptr(y),
+                  _ptr(row_of), _ptr(gts), c_int(top), _ptr(gamma), c_float(eps),
+                  _ptr(out if out is not None and out.dtype == torch.float32 else None),
+                  _ptr(out if out is not None and out.dtype == torch.bfloat16 else None), *conv_args, _ptr(wr),
+                  c_int(_code(wr.dtype) if wr is not None else 0), c_int(E), _ptr(ids), _ptr(gates), _ptr(logits), *rest)
+
+    @staticmethod
+    def _pending_branches(pending):
+        """([(partial sums, bias, scale)], (expert rows, places, weights) or None) of a ``Pending`` or None."""
+        if pending is None:
+            return [], None
+        branches = ([(pending.partials, pending.bias, 1.0)] if pending.partials is not None else []) + list(pending.branches)
+        if len(branches) > 4:
+            raise KernelError("row_post: up to four products can be pending")
+        return branches, (pending.y, pending.row_of, pending.gates) if pending.y is not None else None
 
     @staticmethod
     def _router_rides(router, H):
@@ -342,6 +420,8 @@ class CudaOps:
         _check(x, "x", torch.float32)
         if x.dim() == 3:
             return self.row_norm(x, None, None, 0.0, "layer", pending=pending)
+        if pending.alone:
+            return self.row_post(x, pending)
         T, H = x.shape
         if H % 4 == 0 and H <= 16384:
             return self.row_norm(x, None, None, 0.0, "layer", pending=pending)
@@ -997,17 +1077,18 @@ class CudaOps:
         before its start: u [T, >= col0 + C] float32 rows (a view; rows may be strided), w [C, taps], y [T, C] float32.
         ``state`` [slots, >= (taps - 1) C] float32 (a view of the slab's rows) holds each request's last taps - 1
         inputs and is brought up to date (``ring_rows``, default taps - 1: the rows of C inputs it has; the input at
-        position p lies in row p mod ring_rows).  act: "none" or "silu"."""
+        position p lies in row p mod ring_rows).  act: "none", "silu", or "plus_input" (y = u + its convolution).  y may
+        be of another element type."""
         _check(u, "u", torch.float32, 2, contiguous=False)
         _check(w, "w", torch.float32, 2)
-        _check(y, "y", torch.float32, 2)
+        _check(y, "y", dims=2)
         C, taps = w.shape
         T = u.shape[0]
         if u.stride(1) != 1 or u.shape[1] < col0 + C or tuple(y.shape) != (T, C):
             raise KernelError("short_conv: shapes do not match")
         if bias is not None and (bias.dtype != torch.float32 or bias.numel() != C):
             raise KernelError("short_conv: bias must be float32, one per channel")
-        if act not in ("none", "silu"):
+        if act not in ("none", "silu", "plus_input"):
             raise KernelError(f"short_conv: unknown activation {act!r}")
         if taps > 1:
             if state is None:
@@ -1016,27 +1097,29 @@ class CudaOps:
             if state.stride(1) != 1 or state.shape[1] < (ring_rows or taps - 1) * C:
                 raise KernelError("short_conv: the state's rows are too short")
         self._run("recurrent", "flint_short_conv", _ptr(u), c_longlong(u.stride(0)), c_int(col0), _ptr(w), _ptr(bias),
-                  c_int(1 if act == "silu" else 0), _ptr(pos), _ptr(slot), _ptr(state),
-                  c_longlong(state.stride(0) if state is not None else 0), _ptr(y), c_int(T), c_int(C), c_int(taps),
+                  c_int(("none", "silu", "plus_input").index(act)), _ptr(pos), _ptr(slot), _ptr(state),
+                  c_longlong(state.stride(0) if state is not None else 0), _ptr(y), c_int(_code(y.dtype)), c_int(T), c_int(C), c_int(taps),
                   c_int(ring_rows or taps - 1))
         self.launches += 1 if taps > 1 else 0
 
     def delta_prepare(self, y, b, a, dt_bias, a_log, qk, decay, beta, H, G, D, unit_eps):
         """Operands of the gated delta rule from y [T, 2 G D + H V] (q | k | v after their convolution): qk [T, 2 G D]
         = q and k as unit vectors per head (x / sqrt(sum x^2 + unit_eps); q also times D^(-1/2)); beta [T, H] =
-        sigmoid(b) (b a [T, H] view); decay [T, H D] = exp(-exp(a_log[h]) softplus(a + dt_bias))."""
+        sigmoid(b) (b a [T, H] view); decay [T, H D] = exp(-exp(a_log[h]) softplus(a + dt_bias)), or with one decay a head
+        a (a view) and decay [T, H]."""
         _check(y, "y", torch.float32, 2)
         _check(b, "b", torch.float32, 2, contiguous=False)
-        for name, t in (("a", a), ("qk", qk), ("decay", decay), ("beta", beta)):
+        _check(a, "a", torch.float32, 2, contiguous=False)
+        for name, t in (("qk", qk), ("decay", decay), ("beta", beta)):
             _check(t, name, torch.float32, 2)
-        T = y.shape[0]
-        if y.shape[1] < 2 * G * D or tuple(b.shape) != (T, H) or b.stride(1) != 1 or tuple(a.shape) != (T, H * D) \
-                or tuple(qk.shape) != (T, 2 * G * D) or tuple(decay.shape) != (T, H * D) or tuple(beta.shape) != (T, H) \
-                or dt_bias.numel() != H * D or a_log.numel() != H:
+        T, A = y.shape[0], decay.shape[1] // H
+        if y.shape[1] < 2 * G * D or tuple(b.shape) != (T, H) or b.stride(1) != 1 or tuple(a.shape) != (T, H * A) \
+                or a.stride(1) != 1 or A not in (1, D) or tuple(qk.shape) != (T, 2 * G * D) or tuple(decay.shape) != (T, H * A) \
+                or tuple(beta.shape) != (T, H) or dt_bias.numel() != H * A or a_log.numel() != H:
             raise KernelError("delta_prepare: shapes do not match")
         self._run("recurrent", "flint_delta_prepare", _ptr(y), c_longlong(y.stride(0)), _ptr(b), c_longlong(b.stride(0)),
-                  _ptr(a), _ptr(dt_bias), _ptr(a_log), _ptr(qk), _ptr(decay), _ptr(beta), c_int(T), c_int(H), c_int(G),
-                  c_int(D), c_float(unit_eps))
+                  _ptr(a), c_longlong(a.stride(0)), _ptr(dt_bias), _ptr(a_log), _ptr(qk), _ptr(decay), _ptr(beta), c_int(T),
+                  c_int(H), c_int(G), c_int(D), c_int(A), c_float(unit_eps))
 
     def ssd_prepare(self, raw, dt_bias, a_log, dt, decay):
         """dt = softplus(raw + dt_bias), decay = exp(-exp(a_log) dt): raw a [T, H] float32 view, dt and decay [T, H]."""
@@ -1053,7 +1136,8 @@ class CudaOps:
     def recurrence_scan(self, q, k, v, decay, delta, beta, dt, skip, slot, seq_start, n_seq, state, out, H, G, D, V):
         """Walks every request's rows in order (request e owns rows seq_start[e] .. seq_start[e + 1] - 1;
         ``seq_start`` None: row e alone) from and into ``state`` [slots, >= H D V] float32, per head a matrix S [D, V]:
-        ``delta``: S <- diag(decay_t) S; u = beta_t (v_t - S^T k_t); S <- S + k_t u^T; o_t = S^T q_t (decay [T, H D]);
+        ``delta``: S <- diag(decay_t) S; u = beta_t (v_t - S^T k_t); S <- S + k_t u^T; o_t = S^T q_t (decay [T, H D], or [T, H]:
+                   one a head);
         else:      S <- decay_t S + k_t (dt_t v_t)^T; o_t = S^T q_t + skip v_t (decay, dt [T, H]; skip [H] or None).
         q, k [T, G D] and v [T, H V] are float32 views (rows may be strided); out [T, H V] float32."""
         for name, t in (("q", q), ("k", k), ("v", v)):
@@ -1066,7 +1150,7 @@ class CudaOps:
         _check(state, "state", torch.float32, 2, contiguous=False)
         T = q.shape[0]
         if tuple(q.shape) != (T, G * D) or tuple(k.shape) != (T, G * D) or tuple(v.shape) != (T, H * V) \
-                or tuple(decay.shape) != (T, H * D if delta else H) or tuple(w1.shape) != (T, H) \
+                or tuple(decay.shape) not in ((T, H), (T, H * D if delta else H)) or tuple(w1.shape) != (T, H) \
                 or tuple(out.shape) != (T, H * V) or state.stride(1) != 1 or state.shape[1] < H * D * V:
             raise KernelError("recurrence_scan: shapes do not match")
         if skip is not None and (skip.dtype != torch.float32 or skip.numel() != H):
@@ -1077,9 +1161,10 @@ class CudaOps:
                 raise KernelError("recurrence_scan: seq_start must have one entry more than there are requests")
         elif n_seq != T:
             raise KernelError("recurrence_scan: without seq_start every request brings one row")
-        self._label = f"{'delta' if delta else 'ssd'} H{H} D{D} V{V}"
+        rule = (1 if D > 1 and decay.shape[1] == H * D else 2) if delta else 0
+        self._label = f"{('ssd', 'delta', 'delta, a decay a head')[rule]} H{H} D{D} V{V}"
         self._run("recurrent", "flint_recurrence_scan", _ptr(q), c_longlong(q.stride(0)), _ptr(k), c_longlong(k.stride(0)),
-                  _ptr(v), c_longlong(v.stride(0)), _ptr(decay), c_int(1 if delta else 0), _ptr(w1), _ptr(skip), _ptr(slot),
+                  _ptr(v), c_longlong(v.stride(0)), _ptr(decay), c_int(rule), _ptr(w1), _ptr(skip), _ptr(slot),
                   _ptr(seq_start), c_int(n_seq), _ptr(state), c_longlong(state.stride(0)), _ptr(out), c_int(H), c_int(G),
                   c_int(D), c_int(V))
 
@@ -1655,22 +1740,32 @@ class CudaOps:
                   c_int(tile_rows), *ptrs, c_int(plan.max_tiles), c_int(plan.top))
         return plan
 
-    def moe_dispatch(self, expert_ids, n_experts, tile_rows, x):
+    def moe_dispatch(self, expert_ids, n_experts, tile_rows, x, scale=None, out_dtype=None):
         """The plan for these choices and the rows of x in its order: (plan, xs) with
         xs[r] = x[plan.token_of[r]].  Few rows take one fused launch.  Choices from ``n_experts`` on name experts without
         weights (identity): they take no row, plan.row_of gives them choices + token, and as many rows at the end of
-        xs belong to nobody."""
-        _check(x, "x", dims=2)
+        xs belong to nobody.  ``scale`` [T, top] float32 (then x is float32): xs[r] is the token's row times the score of the
+        choice that sends it, in ``out_dtype``."""
+        _check(x, "x", torch.float32 if scale is not None else None, 2)
         n = expert_ids.numel()
-        xs = torch.empty((n, x.shape[1]), dtype=x.dtype, device=x.device)
+        xs = torch.empty((n, x.shape[1]), dtype=x.dtype if scale is None else out_dtype or x.dtype, device=x.device)
         row_bytes = x.shape[1] * x.element_size()
+        if scale is not None:
+            _check(scale, "scale", torch.float32, 2)
+            if scale.shape != expert_ids.shape:
+                raise KernelError("moe_dispatch: one score a choice")
         if n > 256 or row_bytes % 16 or x.data_ptr() % 16:
             plan = self.moe_plan(expert_ids, n_experts, tile_rows)
-            self.gather_rows(x, plan.token_of, xs)
+            if scale is None:
+                self.gather_rows(x, plan.token_of, xs)
+            else:
+                self._run("moe", "flint_scatter_scaled", _ptr(x), _ptr(plan.row_of), _ptr(scale), _ptr(xs), c_int(_code(xs.dtype)),
+                          c_int(n), c_int(x.shape[1]), c_int(plan.top))
             return plan, xs
         plan, ptrs = self._plan_buffers(expert_ids, n_experts, tile_rows)
         self._run("moe", "flint_moe_dispatch", _ptr(expert_ids), c_int(n), c_int(n_experts), c_int(tile_rows), *ptrs,
-                  c_int(plan.max_tiles), _ptr(x), _ptr(xs), c_int(row_bytes), c_int(plan.top))
+                  c_int(plan.max_tiles), _ptr(x), _ptr(xs), c_int(row_bytes), c_int(plan.top), _ptr(scale),
+                  c_int(_code(xs.dtype)))
         return plan, xs
 
     # ------------------------------------------------------------------ sampling

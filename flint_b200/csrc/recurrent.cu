@@ -2,13 +2,14 @@
 // the gated delta rule and of a state-space model with a scalar decay per head, and what surrounds them.
 //
 // Short convolution.  y[t, c] = act(b[c] + sum_j w[c, j] u[t - taps + 1 + j, c]) over the rows of one request, zeros
-// before its first position.  The inputs of earlier steps come from the request's state, R >= taps - 1 rows: the input at
+// before its first position (act: none, SiLU, or "plus input", u[t, c] + sum).  The inputs of earlier steps come from the request's state, R >= taps - 1 rows: the input at
 // position p lives in state row p mod R.  The convolution's kernel only reads the state; a second kernel,
 // launched behind it, stores the inputs of every request's last taps - 1 rows of the step.  So every row of the batch
 // is worked independently, and no row of the state is read and written in one launch.
 //
 // Recurrence.  Per request and head a float32 matrix S [D, V] (key dims by value dims) lives in the state slab.
 //   gated delta rule:  S <- diag(g_t) S;  u = beta_t (v_t - S^T k_t);  S <- S + k_t u^T;  o_t = S^T q_t
+//                      (g_t a decay per key channel, or one number for the head)
 //   state space:       S <- a_t S + k_t (dt_t v_t)^T;                                     o_t = S^T q_t + skip v_t
 // (for the state-space form k is the input matrix B and q the read-out C).  Columns of S are independent, so a block
 // takes a request, a head and a run of columns; a column is held by 1, 2, 4 or 8 neighbouring lanes, 32 rows each in
@@ -38,10 +39,11 @@ __device__ __forceinline__ bool same_request(const int* pos, const int* slot, in
 
 // ------------------------------------------------------------------------------------------- short convolution
 // u: float32 rows of `in_stride` floats, the convolved channels start at column col0.  Grid: (rows, blocks of channels).
+template <typename TO>
 __global__ void short_conv_kernel(const float* __restrict__ u, long long in_stride, int col0, const float* __restrict__ w,
                                   const float* __restrict__ bias, int act, const int* __restrict__ pos,
                                   const int* __restrict__ slot, const float* __restrict__ ring, long long ring_stride,
-                                  float* __restrict__ y, int T, int C, int taps, int R) {
+                                  TO* __restrict__ y, int T, int C, int taps, int R) {
   pdl_launch();
   pdl_wait();
   const int t = blockIdx.x;
@@ -60,7 +62,7 @@ __global__ void short_conv_kernel(const float* __restrict__ u, long long in_stri
       acc = fmaf(w[(size_t)c * taps + (taps - 1 - d)], x, acc);
     }
     acc = fmaf(w[(size_t)c * taps + taps - 1], row[c], acc);
-    y[(size_t)t * C + c] = act == 1 ? siluf_(acc) : acc;
+    y[(size_t)t * C + c] = from_f32<TO>(act == 1 ? siluf_(acc) : act == 2 ? row[c] + acc : acc);
   }
 }
 
@@ -68,10 +70,19 @@ __global__ void short_conv_kernel(const float* __restrict__ u, long long in_stri
 // weights stay in registers; the rows a convolution shares with its neighbours come from L1.  The same sums in the same
 // order.
 constexpr int CONV_ROWS = 8, CONV_TAPS = 8;
+__device__ __forceinline__ void store4(float* p, const float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, const float4 v) {
+  const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+  uint2 pk;
+  pk.x = *reinterpret_cast<const uint32_t*>(&lo);
+  pk.y = *reinterpret_cast<const uint32_t*>(&hi);
+  *reinterpret_cast<uint2*>(p) = pk;
+}
+template <typename TO>
 __global__ void __launch_bounds__(128)
 short_conv_rows_kernel(const float* __restrict__ u, long long in_stride, int col0, const float* __restrict__ w,
                        const float* __restrict__ bias, int act, const int* __restrict__ pos, const int* __restrict__ slot,
-                       const float* __restrict__ ring, long long ring_stride, float* __restrict__ y, int T, int C, int taps,
+                       const float* __restrict__ ring, long long ring_stride, TO* __restrict__ y, int T, int C, int taps,
                        int R) {
   __shared__ int have_s[CONV_ROWS], pos_s[CONV_ROWS];
   pdl_launch();
@@ -107,7 +118,11 @@ short_conv_rows_kernel(const float* __restrict__ u, long long in_stride, int col
       acc.z = fmaf(wt[d].z, x.z, acc.z); acc.w = fmaf(wt[d].w, x.w, acc.w);
     }
     if (act == 1) acc = make_float4(siluf_(acc.x), siluf_(acc.y), siluf_(acc.z), siluf_(acc.w));
-    *reinterpret_cast<float4*>(y + (size_t)t * C + c) = acc;
+    if (act == 2) {
+      const float4 x = *reinterpret_cast<const float4*>(row);
+      acc = make_float4(x.x + acc.x, x.y + acc.y, x.z + acc.z, x.w + acc.w);
+    }
+    store4(y + (size_t)t * C + c, acc);
   }
 }
 
@@ -126,11 +141,13 @@ __global__ void short_conv_keep_kernel(const float* __restrict__ u, long long in
 
 // ------------------------------------------------------------------------------------------- gated delta rule: operands
 // y [T, 2 G D + H V]: q | k | v after the convolution.  q and k become unit vectors per head (q times D^(-1/2));
-// beta = sigmoid(b); decay[t, h, d] = exp(-exp(A_log[h]) softplus(a[t, h, d] + dt_bias[h, d])).  One block per row.
+// beta = sigmoid(b); decay[t, h, d] = exp(-exp(A_log[h]) softplus(a[t, h, d] + dt_bias[h, d])), d over A = D key channels or
+// over A = 1 (one decay per head).  One block per row.
 __global__ void delta_prepare_kernel(const float* __restrict__ y, long long y_stride, const float* __restrict__ b,
-                                     long long b_stride, const float* __restrict__ a, const float* __restrict__ dt_bias,
-                                     const float* __restrict__ a_log, float* __restrict__ qk, float* __restrict__ decay,
-                                     float* __restrict__ beta, int H, int G, int D, float unit_eps) {
+                                     long long b_stride, const float* __restrict__ a, long long a_stride,
+                                     const float* __restrict__ dt_bias, const float* __restrict__ a_log,
+                                     float* __restrict__ qk, float* __restrict__ decay, float* __restrict__ beta, int H, int G,
+                                     int D, int A, float unit_eps) {
   pdl_launch();
   pdl_wait();
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
@@ -144,9 +161,9 @@ __global__ void delta_prepare_kernel(const float* __restrict__ y, long long y_st
     const float inv = (1.0f / sqrtf(ss + unit_eps)) * (g < G ? q_scale : 1.0f);
     for (int d = lane; d < D; d += 32) qk[(size_t)t * 2 * G * D + (size_t)g * D + d] = src[d] * inv;
   }
-  for (int e = threadIdx.x; e < H * D; e += blockDim.x) {
-    const float rate = expf(a_log[e / D]);
-    decay[(size_t)t * H * D + e] = expf(-rate * softplusf_(a[(size_t)t * H * D + e] + dt_bias[e]));
+  for (int e = threadIdx.x; e < H * A; e += blockDim.x) {
+    const float rate = expf(a_log[e / A]);
+    decay[(size_t)t * H * A + e] = expf(-rate * softplusf_(a[(size_t)t * a_stride + e] + dt_bias[e]));
   }
   for (int h = threadIdx.x; h < H; h += blockDim.x) beta[(size_t)t * H + h] = sigmoidf_(b[(size_t)t * b_stride + h]);
 }
@@ -179,13 +196,14 @@ __device__ __forceinline__ void copy16(float* dst, const float* src) {
 
 constexpr int SEG = RPT + 4;     // floats between the rows of neighbouring lanes of a column: their 16-byte reads miss each other's banks
 
-// TPC: threads per column (D <= 32 TPC).  DELTA: the gated delta rule (a decay per key channel, the write corrected
-// by what the state already returns for the key), else the state-space form (one decay per head, plain write).
-// q, k [T, G D] and v [T, H V] are float32 views with row strides; decay [T, H D] (DELTA) or [T, H]; w1 [T, H]: beta
-// (DELTA) or dt; skip [H] or null.  seq_start [n_seq + 1] or null (row e is request e).  Grid: (column blocks, H, n_seq).
+// TPC: threads per column (D <= 32 TPC).  RULE: the state-space form (one decay per head, plain write) or the gated delta
+// rule (the write corrected by what the state already returns for the key) with a decay per key channel or per head.
+// q, k [T, G D] and v [T, H V] are float32 views with row strides; decay [T, H D] (DELTA_CHANNEL) or [T, H]; w1 [T, H]: dt
+// (STATE_SPACE) or beta; skip [H] or null.  seq_start [n_seq + 1] or null (row e is request e).  Grid: (column blocks, H, n_seq).
 // VEC: every row of q, k, v and decay starts on a 16-byte boundary and D and V are multiples of 4, so the operands are
 // staged 16 bytes a copy; else 4 bytes a copy.  Both leave the same numbers in the same places.
-template <int TPC, bool DELTA, bool VEC>
+enum { STATE_SPACE = 0, DELTA_CHANNEL = 1, DELTA_HEAD = 2 };
+template <int TPC, int RULE, bool VEC>
 __global__ void __launch_bounds__(SCAN_THREADS)
 recurrence_scan_kernel(const float* __restrict__ q, long long q_stride, const float* __restrict__ k, long long k_stride,
                        const float* __restrict__ v, long long v_stride, const float* __restrict__ decay,
@@ -194,7 +212,8 @@ recurrence_scan_kernel(const float* __restrict__ q, long long q_stride, const fl
                        float* __restrict__ o, int H, int G, int D, int V, int TB) {
   extern __shared__ __align__(16) float sm[];
   constexpr int DP = TPC * SEG;                  // floats of a staged vector of key dims: lane s of a column reads from s SEG
-  constexpr int NV = DELTA ? 3 : 2;              // staged vectors a token: q, k (and the decay per channel)
+  constexpr bool CHANNEL = RULE == DELTA_CHANNEL;
+  constexpr int NV = CHANNEL ? 3 : 2;            // staged vectors a token: q, k (and the decay per channel)
   constexpr int COLS = SCAN_THREADS / TPC;       // columns a block takes
   const int tid = threadIdx.x, sub = tid % TPC, col = blockIdx.x * COLS + tid / TPC;
   const int h = blockIdx.y, e = blockIdx.z, kh = h / (H / G);
@@ -205,7 +224,7 @@ recurrence_scan_kernel(const float* __restrict__ q, long long q_stride, const fl
   float* stage[2] = {sm, sm + (size_t)TB * per_tok};
   for (int i = tid; i < 2 * TB * per_tok; i += SCAN_THREADS) {      // dims beyond D: q = k = 0, decay = 1
     const int w = i % per_tok;
-    sm[i] = (DELTA && w >= 2 * DP && w < 3 * DP) ? 1.f : 0.f;
+    sm[i] = (CHANNEL && w >= 2 * DP && w < 3 * DP) ? 1.f : 0.f;
   }
   __syncthreads();
   pdl_wait();
@@ -220,7 +239,7 @@ recurrence_scan_kernel(const float* __restrict__ q, long long q_stride, const fl
   const int c0 = blockIdx.x * COLS, nc = min(COLS, V - c0);
   const float* q_h = q + (size_t)kh * D;
   const float* k_h = k + (size_t)kh * D;
-  const float* g_h = DELTA ? decay + (size_t)h * D : nullptr;
+  const float* g_h = CHANNEL ? decay + (size_t)h * D : nullptr;
   const float* v_h = v + (size_t)h * V + c0;
   auto fetch = [&](int t0, int st) {
     const int n = min(TB, r1 - t0);
@@ -232,7 +251,7 @@ recurrence_scan_kernel(const float* __restrict__ q, long long q_stride, const fl
         int a = 0, x = j;                        // which vector, which piece of it
         if (x >= d4) { x -= d4; a = 1; }
         if (a == 1 && x >= d4) { x -= d4; a = 2; }
-        if (DELTA && a == 2 && x >= d4) { x -= d4; a = 3; }
+        if (CHANNEL && a == 2 && x >= d4) { x -= d4; a = 3; }
         const bool val = a == NV;
         const int d = 4 * x;
         const int off = val ? NV * DP + d : a * DP + (d / RPT) * SEG + d % RPT;
@@ -246,7 +265,7 @@ recurrence_scan_kernel(const float* __restrict__ q, long long q_stride, const fl
         float* dst = base + (size_t)tt * per_tok + (d / RPT) * SEG + d % RPT;
         copy4(dst, q_h + (size_t)t * q_stride + d);
         copy4(dst + DP, k_h + (size_t)t * k_stride + d);
-        if (DELTA) copy4(dst + 2 * DP, g_h + (size_t)t * H * D + d);
+        if (CHANNEL) copy4(dst + 2 * DP, g_h + (size_t)t * H * D + d);
       }
       for (int i = tid; i < n * nc; i += SCAN_THREADS) {
         const int tt = i / nc, c = i % nc;
@@ -256,7 +275,7 @@ recurrence_scan_kernel(const float* __restrict__ q, long long q_stride, const fl
     for (int tt = tid; tt < n; tt += SCAN_THREADS) {
       float* dst = base + (size_t)tt * per_tok + NV * DP + COLS;
       copy4(dst, w1 + (size_t)(t0 + tt) * H + h);
-      if (!DELTA) copy4(dst + 1, decay + (size_t)(t0 + tt) * H + h);
+      if (!CHANNEL) copy4(dst + 1, decay + (size_t)(t0 + tt) * H + h);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
@@ -282,12 +301,13 @@ recurrence_scan_kernel(const float* __restrict__ q, long long q_stride, const fl
 #pragma unroll
       for (int i = 0; i < RPT / 4; ++i) kr[i] = k4[i];
       float u;
-      if (DELTA) {
+      if (RULE != STATE_SPACE) {
         const float4* g4 = reinterpret_cast<const float4*>(tok + 2 * DP + sub * SEG);
+        const float a = CHANNEL ? 0.f : rest[COLS + 1];
         float d0 = 0.f, d1 = 0.f, d2 = 0.f, d3 = 0.f;
 #pragma unroll
         for (int i = 0; i < RPT / 4; ++i) {
-          const float4 gg = g4[i];
+          const float4 gg = CHANNEL ? g4[i] : make_float4(a, a, a, a);
           S[4 * i] *= gg.x; S[4 * i + 1] *= gg.y; S[4 * i + 2] *= gg.z; S[4 * i + 3] *= gg.w;
           d0 = fmaf(S[4 * i], kr[i].x, d0); d1 = fmaf(S[4 * i + 1], kr[i].y, d1);
           d2 = fmaf(S[4 * i + 2], kr[i].z, d2); d3 = fmaf(S[4 * i + 3], kr[i].w, d3);
@@ -709,13 +729,14 @@ __global__ void head_finish_kernel(const TA* __restrict__ attn, const int* __res
                                    long long gate_stride, int gate_each, TA* __restrict__ out, int T, int nq, int vd) {
   pdl_launch();
   pdl_wait();
-  const int half = vd / 2;
+  const int half = (vd + 1) / 2;          // an odd size (never with a rotation) leaves one dim without a partner
   const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
   if (idx >= (long long)T * nq * half) return;
   const int i = (int)(idx % half), head = (int)((idx / half) % nq), t = (int)(idx / ((long long)half * nq));
   const int a = interleaved ? 2 * i : i, b = interleaved ? 2 * i + 1 : i + half;
   const size_t base = ((size_t)t * nq + head) * vd;
-  float u = to_f32(attn[base + a]), v = to_f32(attn[base + b]);
+  const bool pair = b < vd;
+  float u = to_f32(attn[base + a]), v = pair ? to_f32(attn[base + b]) : 0.f;
   if (vcos) {
     const float c = vcos[(size_t)pos[t] * half + i], s = vsin[(size_t)pos[t] * half + i];
     const float u2 = u * c + v * s, v2 = v * c - u * s;       // the angle's sign turned round
@@ -725,9 +746,9 @@ __global__ void head_finish_kernel(const TA* __restrict__ attn, const int* __res
   // a gate per head, or one per number of every head
   const float* gr = gate + (size_t)t * gate_stride;
   const float ga = !gate ? 1.f : sigmoidf_(gate_each ? gr[(size_t)head * vd + a] : gr[head]);
-  const float gb = !gate ? 1.f : (gate_each ? sigmoidf_(gr[(size_t)head * vd + b]) : ga);
+  const float gb = !gate ? 1.f : (gate_each ? sigmoidf_(gr[(size_t)head * vd + (pair ? b : a)]) : ga);
   out[base + a] = from_f32<TA>(u * ga);
-  out[base + b] = from_f32<TA>(v * gb);
+  if (pair) out[base + b] = from_f32<TA>(v * gb);
 }
 
 }  // namespace
@@ -738,8 +759,8 @@ __global__ void head_finish_kernel(const TA* __restrict__ attn, const int* __res
 static int row_threads(int W) { return W >= 2048 ? 1024 : W >= 1024 ? 512 : W >= 512 ? 256 : 128; }
 
 extern "C" int flint_short_conv(const float* u, long long in_stride, int col0, const float* w, const float* bias, int act,
-                                const int* pos, const int* slot, float* ring, long long ring_stride, float* y, int T,
-                                int C, int taps, int ring_rows, cudaStream_t stream) {
+                                const int* pos, const int* slot, float* ring, long long ring_stride, void* y,
+                                int y_dtype, int T, int C, int taps, int ring_rows, cudaStream_t stream) {
   if (T <= 0 || C <= 0) return 0;
   if (ring_rows < taps - 1) return fail("short_conv: %d rows of state do not hold the last %d inputs", ring_rows, taps - 1);
   if (taps < 1 || taps > 64) return fail("short_conv: %d taps are not supported (1 to 64)", taps);
@@ -750,11 +771,14 @@ extern "C" int flint_short_conv(const float* u, long long in_stride, int col0, c
   const bool lined = C % 4 == 0 && col0 % 4 == 0 && in_stride % 4 == 0 && ring_stride % 4 == 0 &&
                      !(((uintptr_t)u | (uintptr_t)ring | (uintptr_t)y | (uintptr_t)bias) & 15);
   if (T >= 128 && taps <= CONV_TAPS && lined)
-    launch_pdl(short_conv_rows_kernel, dim3((unsigned)((T + CONV_ROWS - 1) / CONV_ROWS), (unsigned)((C + 511) / 512)), dim3(128), 0,
-               stream, u, in_stride, col0, w, bias, act, pos, slot, (const float*)ring, ring_stride, y, T, C, taps, ring_rows);
+    FLINT_DISPATCH_DTYPE(y_dtype, TO,
+        launch_pdl(short_conv_rows_kernel<TO>, dim3((unsigned)((T + CONV_ROWS - 1) / CONV_ROWS), (unsigned)((C + 511) / 512)),
+                   dim3(128), 0, stream, u, in_stride, col0, w, bias, act, pos, slot, (const float*)ring, ring_stride, (TO*)y, T,
+                   C, taps, ring_rows));
   else
-    launch_pdl(short_conv_kernel, grid, dim3(threads), 0, stream, u, in_stride, col0, w, bias, act, pos, slot,
-               (const float*)ring, ring_stride, y, T, C, taps, ring_rows);
+    FLINT_DISPATCH_DTYPE(y_dtype, TO,
+        launch_pdl(short_conv_kernel<TO>, grid, dim3(threads), 0, stream, u, in_stride, col0, w, bias, act, pos, slot,
+                   (const float*)ring, ring_stride, (TO*)y, T, C, taps, ring_rows));
   if (taps > 1)
     launch_pdl(short_conv_keep_kernel, grid, dim3(threads), 0, stream, u, in_stride, col0, pos, slot, ring, ring_stride, T, C,
                taps, ring_rows);
@@ -762,12 +786,13 @@ extern "C" int flint_short_conv(const float* u, long long in_stride, int col0, c
 }
 
 extern "C" int flint_delta_prepare(const float* y, long long y_stride, const float* b, long long b_stride, const float* a,
-                                   const float* dt_bias, const float* a_log, float* qk, float* decay, float* beta, int T,
-                                   int H, int G, int D, float unit_eps, cudaStream_t stream) {
+                                   long long a_stride, const float* dt_bias, const float* a_log, float* qk, float* decay,
+                                   float* beta, int T, int H, int G, int D, int A, float unit_eps, cudaStream_t stream) {
   if (T <= 0) return 0;
+  if (A != 1 && A != D) return fail("delta_prepare: %d decays a head (one, or one per key channel)", A);
   if (G <= 0 || H % G) return fail("delta_prepare: %d heads do not divide into %d key heads", H, G);
-  launch_pdl(delta_prepare_kernel, dim3((unsigned)T), dim3(256), 0, stream, y, y_stride, b, b_stride, a, dt_bias, a_log, qk,
-             decay, beta, H, G, D, unit_eps);
+  launch_pdl(delta_prepare_kernel, dim3((unsigned)T), dim3(256), 0, stream, y, y_stride, b, b_stride, a, a_stride,
+             dt_bias, a_log, qk, decay, beta, H, G, D, A, unit_eps);
   return check_launch("delta_prepare");
 }
 
@@ -792,33 +817,35 @@ static cudaError_t launch_scan(bool early, void (*kernel)(KArgs...), dim3 grid, 
 }
 
 extern "C" int flint_recurrence_scan(const float* q, long long q_stride, const float* k, long long k_stride, const float* v,
-                                     long long v_stride, const float* decay, int delta, const float* w1, const float* skip,
+                                     long long v_stride, const float* decay, int rule, const float* w1, const float* skip,
                                      const int* slot, const int* seq_start, int n_seq, float* state,
                                      long long state_stride, float* o, int H, int G, int D, int V, cudaStream_t stream) {
   if (n_seq <= 0) return 0;
   if (D < 1 || D > 256 || V < 1) return fail("recurrence_scan: %d key dims per head are not supported (1 to 256)", D);
+  if (rule != STATE_SPACE && rule != DELTA_CHANNEL && rule != DELTA_HEAD) return fail("recurrence_scan: unknown rule %d", rule);
   if (G <= 0 || H % G) return fail("recurrence_scan: %d heads do not divide into %d key heads", H, G);
   if (n_seq > 65535 || H > 65535) return fail("recurrence_scan: too many requests or heads");
   const int tpc = D <= 32 ? 1 : D <= 64 ? 2 : D <= 128 ? 4 : 8;
   const int dp = tpc * SEG, cols = SCAN_THREADS / tpc;
   const int tb = tpc <= 2 ? 16 : tpc <= 4 ? 8 : 4;
-  const size_t smem = (size_t)2 * tb * ((delta ? 3 : 2) * dp + cols + 4) * sizeof(float);
+  const size_t smem = (size_t)2 * tb * ((rule == DELTA_CHANNEL ? 3 : 2) * dp + cols + 4) * sizeof(float);
   const dim3 grid((unsigned)((V + cols - 1) / cols), (unsigned)H, (unsigned)n_seq), block(SCAN_THREADS);
   // 16-byte copies need every staged row to start on such a boundary
   auto lined = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
   const bool vec = D % 4 == 0 && V % 4 == 0 && q_stride % 4 == 0 && k_stride % 4 == 0 && v_stride % 4 == 0 && lined(q) &&
-                   lined(k) && lined(v) && (!delta || lined(decay));
+                   lined(k) && lined(v) && (rule != DELTA_CHANNEL || lined(decay));
   // A walk over prompts starts as an ordinary dependent, on an empty chip, where its few blocks get an SM each: started
   // early they land beside the blocks of the kernel before, several to an SM (a prompt of 2,048 tokens then ran half
   // a millisecond longer a layer).  A batch of single tokens fills the chip anyway and starts early.
   const bool early = seq_start == nullptr;
-#define SCAN(TPC, DELTA, VEC)                                                                                          \
-  launch_scan(early, recurrence_scan_kernel<TPC, DELTA, VEC>, grid, block, smem, stream, q, q_stride, k, k_stride, v,   \
+#define SCAN(TPC, RULE, VEC)                                                                                           \
+  launch_scan(early, recurrence_scan_kernel<TPC, RULE, VEC>,  grid, block, smem, stream, q, q_stride, k, k_stride, v,   \
               v_stride, decay, w1, skip, slot, seq_start, state, state_stride, o, H, G, D, V, tb)
 #define SCAN_T(TPC)                                                                                       \
   do {                                                                                                    \
-    if (delta) { if (vec) SCAN(TPC, true, true); else SCAN(TPC, true, false); }                           \
-    else { if (vec) SCAN(TPC, false, true); else SCAN(TPC, false, false); }                               \
+    if (rule == DELTA_CHANNEL) { if (vec) SCAN(TPC, DELTA_CHANNEL, true); else SCAN(TPC, DELTA_CHANNEL, false); } \
+    else if (rule == DELTA_HEAD) { if (vec) SCAN(TPC, DELTA_HEAD, true); else SCAN(TPC, DELTA_HEAD, false); }     \
+    else { if (vec) SCAN(TPC, STATE_SPACE, true); else SCAN(TPC, STATE_SPACE, false); }                   \
   } while (0)
   if (tpc == 1) SCAN_T(1);
   else if (tpc == 2) SCAN_T(2);
@@ -964,8 +991,8 @@ extern "C" int flint_head_finish(const void* attn, int dtype, const int* pos, co
                                  int interleaved, const float* gate, long long gate_stride, int gate_each, void* out, int T,
                                  int nq, int vd, cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (vd % 2) return fail("head_finish: value heads of %d dims cannot rotate in pairs", vd);
-  const long long n = (long long)T * nq * (vd / 2);
+  if (vd % 2 && vcos) return fail("head_finish: value heads of %d dims cannot rotate in pairs", vd);
+  const long long n = (long long)T * nq * ((vd + 1) / 2);
   FLINT_DISPATCH_DTYPE(dtype, TA,
       launch_pdl(head_finish_kernel<TA>, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream, (const TA*)attn, pos, vcos,
                  vsin, interleaved, gate, gate_stride, gate_each, (TA*)out, T, nq, vd));

@@ -219,7 +219,7 @@ class Model:
         self.cache = CacheManager(kv_calls, state_calls, page_size=page_size, n_pages=n_pages, max_slots=max_slots,
                                   max_context=self.max_context, dtype=cache_dtype, device=self.device)
         # one mixer of each kind plans the step, and the step carries a tiling for every distinct declaration
-        self.planners = list({type(m): m for m in (layer.parts.get("mixer") for layer in self.layers)
+        self.planners = list({m.plan_key(): m for m in (layer.parts.get("mixer") for layer in self.layers)
                               if m is not None}.values())
         needs = [n for n in (m.step_needs() for layer in self.layers for m in [layer.parts.get("mixer")] if m is not None)
                  if n is not None]
@@ -355,6 +355,7 @@ class Model:
         elif history is not None:
             history[0].copy_(h)
         carry = None     # an addition to h that a layer left for the next norm to apply
+        finish = step.record is not None and "rows_after" in step.record      # asked for what every call leaves
         x0 = None        # the embedded rows in the type the pass inputs' product reads
         if self.pass_inputs:
             wdt = self.pass_w[0].dtype
@@ -374,11 +375,11 @@ class Model:
             owner = i if call.cache_of is None else call.cache_of
             carry = layer.block.forward(h, step, self.cache.view(owner), self.cache.state_of(i),
                                         writes_cache=call.cache_of is None, carry=carry)
-            if spec.streams and step.record is not None and "rows_after" in step.record:
-                ops.apply_pending(h, carry)       # asked for what every call leaves (the streams' sum): finished here
+            if carry is not None and finish:
+                ops.apply_pending(h, carry)       # of streams their sum is recorded
                 carry = None
-                step.record["rows_after"].append(h.sum(1))
-            if step.record is not None and carry is None and history is None and not spec.streams:
+                step.record["rows_after"].append(h.sum(1) if spec.streams else h.clone())
+            elif step.record is not None and carry is None and history is None and not spec.streams:
                 step.record.setdefault("rows_after", []).append(h.clone())      # the rows as this call leaves them
             if history is not None:
                 if carry is not None:

@@ -1,2 +1,2 @@
 """Architectures.  Importing this package registers the built-in ones."""
-from . import dumizen, gepadra, phimoe, puledra, sinilorn, tefovik  # noqa: F401
+from . import dumizen, gepadra, phimoe, puledra, sinilorn, sokipel, tefovik  # noqa: F401

@@ -15,10 +15,12 @@ Norm          ``forward(x, want, row_index=None, pending=None, router=None) -> {
               ``Pending`` addition to x first; one with ``supports_router`` can fill a
               ``RouterRequest``.  Both are optional abilities; the block works without them.
 Mixer         ``input_dtypes()``, ``cache_spec()``, ``state_spec()``, optionally ``step_needs()`` (rows cut into
-              tiles) and ``plan_step(step, captured)`` (how this step's work is cut),
+              tiles), ``plan_step(step, captured)`` (how this step's work is cut) and ``plan_key()`` (which mixers plan alike),
               ``forward(x, residual, step, cache, state, writes_cache=True)``:
               adds its output into ``residual`` (float32 [T, H]) in place and returns None,
-              or returns a ``Pending`` that the block hands to the next norm.
+              or returns a ``Pending`` that the block hands to the next norm.  One with
+              ``from_rows(residual, carry, step, cache, state, writes_cache)`` forms its input from the rows
+              themselves, with the addition ``carry`` (or None) applied to them on the way, and returns a ``Pending``.
 FeedForward   ``input_dtypes()``, ``forward(x, residual, step)``: adds into ``residual`` or
               returns a ``Pending``.  A feed-forward with ``router_request(n_rows)`` gets the
               filled request back as ``forward(..., routed=request)``.
@@ -49,7 +51,9 @@ class Pending:
     (``partials`` [S, T, H] float32, plus an optional ``bias`` [H]), or the selected experts'
     outputs (``y`` [kT, H] with ``row_of`` [T, k] and ``gates`` [T, k], k choices a token), or both.  For a residual of
     several streams ``mix`` [S, S] ([from, to]) and ``spread`` [S] say how it goes into them: with r the addition,
-    x_t <- sum_s mix[s, t] x_s + spread[t] r for all t at once."""
+    x_t <- sum_s mix[s, t] x_s + spread[t] r for all t at once.  ``branches``: several products' partial sums, each with a
+    bias (or None) and a constant weight.  With ``gamma`` [H] the sum of all of it is divided by its root mean square (``eps``
+    inside the root) and scaled before it is added."""
     partials: torch.Tensor | None = None
     bias: torch.Tensor | None = None
     y: torch.Tensor | None = None
@@ -57,6 +61,14 @@ class Pending:
     gates: torch.Tensor | None = None
     mix: torch.Tensor | None = None
     spread: torch.Tensor | None = None
+    branches: tuple = ()
+    gamma: torch.Tensor | None = None
+    eps: float = 0.0
+
+    @property
+    def alone(self) -> bool:
+        """Whether it is added by a kernel of its own (a norm's kernel cannot apply it on the way)."""
+        return self.gamma is not None or bool(self.branches)
 
 
 @dataclass
@@ -145,6 +157,10 @@ class Mixer(Part):
     def step_needs(self):
         """A ``StepNeeds`` if the mixer wants the step's rows cut into tiles (see ``engine/step.py``), else None."""
         return None
+
+    def plan_key(self):
+        """Mixers with the same key plan a step alike: one of them is asked."""
+        return type(self)
 
     def plan_step(self, step, captured: bool):
         """Called once per step (on one mixer of each kind) before the layers run, with the host-side view of

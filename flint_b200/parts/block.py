@@ -8,6 +8,8 @@
 the norms come after the sums (a and the scales s are the norms' ``residual_scale`` and ``branch_scale``).
 ``sandwich``: h += norm1b(mixer(norm1(h))); h += norm2b(ffn(norm2(h))): a norm before and one after each part, the
 second applied to what the part adds (RMS norms; the second half only with a feed-forward).
+``outnorm``: h += norm1(mixer(h)); h += norm2(ffn(h)): the parts read the rows themselves, and a norm is applied to what a
+part adds (RMS norms; the second half only with a feed-forward).
 ``streams``: the residual is S streams; a part reads norm(sum_s gather[s] x_s) and what it adds, r, goes into all of
 them: x_t <- sum_s mix[s, t] x_s + spread[t] r (the second half only with a feed-forward).
 An arrangement only orders parts; it does not know what they are.
@@ -25,7 +27,7 @@ from .base import Pending, StreamMix
 def run_norm(norm, residual, want, pending=None, router=None, row_index=None, gather=None):
     """Run a norm; a pending addition or a routing request that the norm cannot take is served
     by separate kernels instead.  Returns (outputs, router or None if it still has to be done)."""
-    if pending is not None and not norm.supports_pending:
+    if pending is not None and (pending.alone or not norm.supports_pending):
         norm.ops.apply_pending(residual, pending)
         pending = None
     if router is not None and not norm.supports_router:
@@ -238,6 +240,46 @@ class PostNormBlock(Block):
         fed = branch_of(ffn, residual, lambda rows: ffn.forward(y, rows, step))
         p["norm2"].post(residual, fed)
         return None
+
+
+@BLOCKS.register("outnorm")
+class OutNormBlock(Block):
+    """h += norm1(mixer(h)); h += norm2(ffn(h)), the second half only with a feed-forward.  What a part adds stays pending
+    together with its norm: one kernel sums it, norms it, adds it into the rows and prepares what the next part reads (the
+    feed-forward's routing and copy of the rows; for a mixer with ``from_rows`` its input)."""
+    roles = ("norm1", "mixer")
+
+    @staticmethod
+    def _normed(part, norm, residual, run):
+        if norm.mode != "rms":
+            raise ConfigError("block 'outnorm': the norms after the parts are RMS norms")
+        pend = branch_of(part, residual, run)
+        pend.gamma, pend.eps = norm.gamma, norm.eps
+        return pend
+
+    def forward(self, residual, step, cache, state, writes_cache=True, carry=None):
+        p = self.parts
+        mixer, ffn = p["mixer"], p.get("ffn")
+        if hasattr(mixer, "from_rows"):
+            run = lambda rows: mixer.from_rows(residual, carry, step, cache, state, writes_cache)
+        else:
+            settle(mixer, residual, carry)
+            x = rows_in(mixer.ops, residual, step, mixer.input_dtypes())
+            run = lambda rows: mixer.forward(x, rows, step, cache, state, writes_cache)
+        pend = self._normed(mixer, p["norm1"], residual, run)
+        if ffn is None:
+            return pend
+        if "norm2" not in p:
+            raise ConfigError("block 'outnorm': a feed-forward needs its norm (norm2)")
+        request = ffn.router_request(residual.shape[0]) if hasattr(ffn, "router_request") else None
+        if request is not None and step.record is not None and getattr(request, "logits", 0) is None:
+            request.logits = request.weight.new_empty((residual.shape[0], request.weight.shape[0]), dtype=torch.float32)
+        want = set(ffn.input_dtypes_when_routed() if request is not None else ffn.input_dtypes())
+        copies = [torch.empty(residual.shape, dtype=dt, device=residual.device) for dt in want if dt != residual.dtype]
+        ffn.ops.row_post(residual, pend, out=copies[0] if copies else None, router=request)
+        y = {residual.dtype: residual, **{c.dtype: c for c in copies}}
+        return self._normed(ffn, p["norm2"], residual, lambda rows: ffn.forward(y, rows, step, routed=request)
+                            if request is not None else ffn.forward(y, rows, step))
 
 
 @STREAM_MIXES.register("hyper_connection")

@@ -26,8 +26,8 @@ from .block import branch_of
 @MIXERS.register("branches")
 class Branches(Mixer):
     """params: hidden_size, eps, branches: ((name, PartSpec), ...), combine ("rms_mean", the default, or "weighted"
-    with ``scales``, one number a branch).  tensors: every branch's own under ``<name>.``, and for the mean
-    ``<name>.out`` [hidden]."""
+    with ``scales``, one number a branch), leave_branches (with "weighted": the sum is left to whoever adds it, as
+    ``Pending.branches``).  tensors: every branch's own under ``<name>.``, and for the mean ``<name>.out`` [hidden]."""
 
     returns_pending = True
 
@@ -45,6 +45,7 @@ class Branches(Mixer):
             raise ConfigError(f"branches: {len(self.branches)} branches are not supported (1 to 4)")
         if sum(m.cache_spec() is not None for _, m in self.branches) > 1:
             raise ConfigError("branches: at most one branch may own a paged cache")
+        self.leave_branches = bool(params.get("leave_branches", False)) and self.combine == "weighted"
         self.graph_safe = all(m.graph_safe for _, m in self.branches)
         self.out_w = []
 
@@ -90,6 +91,9 @@ class Branches(Mixer):
             raise ConfigError("branches: the branches ask for different tilings of the step's rows")
         return needs[0] if needs else None
 
+    def plan_key(self):
+        return (type(self), tuple(m.plan_key() for _, m in self.branches))
+
     def plan_step(self, step, captured):
         return tuple(m.plan_step(step, captured) for _, m in self.branches)
 
@@ -105,6 +109,8 @@ class Branches(Mixer):
             c = cache if m.cache_spec() is not None else None
             outs.append(branch_of(m, next(iter(x.values())),
                                   lambda rows, m=m, c=c, st=st: m.forward(x, rows, step, c, st, writes_cache)))
+        if self.leave_branches:
+            return Pending(branches=tuple((o.partials, o.bias, s) for o, s in zip(outs, self.scales)))
         T = outs[0].partials.shape[1]
         out = torch.empty((1, T, self.hidden), dtype=torch.float32, device=outs[0].partials.device)
         if self.combine == "weighted":

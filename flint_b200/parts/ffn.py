@@ -16,6 +16,18 @@ from ..registry import FEED_FORWARDS
 from .base import FeedForward, Pending, RouterRequest, mat, matmul_dtype, vec
 
 
+def gated_act_params(who, act, params):
+    """(slope, limit) of act ``swish_clamped`` from a part's parameters, None for the gated acts without constants."""
+    if act == "swish_clamped":
+        slope, limit = float(params["act_slope"]), float(params["act_limit"])
+        if limit <= 0:
+            raise ConfigError(f"{who}: act_limit must be positive, got {limit}")
+        return slope, limit
+    if act not in ("silu", "gelu_pytorch_tanh"):
+        raise ConfigError(f"{who}: unknown activation {act!r}")
+    return None
+
+
 @FEED_FORWARDS.register("gated_mlp")
 class GatedMLP(FeedForward):
     """params: hidden_size, intermediate_size, act; tensors gate_proj/up_proj [I,H], down_proj [H,I].
@@ -32,13 +44,7 @@ class GatedMLP(FeedForward):
         self.act = params.get("act", "silu")
         self.has_bias = bool(params.get("bias", False))
         self.returns_pending = bool(params.get("pending", False))
-        self.act_params = None
-        if self.act == "swish_clamped":
-            self.act_params = (float(params["act_slope"]), float(params["act_limit"]))
-            if self.act_params[1] <= 0:
-                raise ConfigError(f"gated_mlp: act_limit must be positive, got {self.act_params[1]}")
-        elif self.act not in ("silu", "gelu_pytorch_tanh"):
-            raise ConfigError(f"gated_mlp: unknown activation {self.act!r}")
+        self.act_params = gated_act_params("gated_mlp", self.act, params)
 
     def weights(self):
         w = {"gate_proj.weight": mat(self.inter, self.hidden), "up_proj.weight": mat(self.inter, self.hidden),
@@ -208,7 +214,7 @@ class GroupedTopKMoE(FeedForward):
         self.groups, self.keep = int(p.get("groups", 1)), int(p.get("keep_groups", 1))
         self.router_scale = float(p.get("router_scale", 1.0))
         self.act = p.get("act", "silu")
-        self.act_params = (float(p["act_slope"]), float(p["act_limit"])) if self.act == "swish_clamped" else None
+        self.act_params = gated_act_params("grouped_topk_moe", self.act, p)
         self.identity = int(p.get("identity", 0) or 0)
         self.correction = bool(p.get("correction", False))
         self.choices = self.E + self.identity          # what the router chooses from
@@ -220,10 +226,6 @@ class GroupedTopKMoE(FeedForward):
             raise ConfigError(f"{self.choices} experts do not form {self.groups} equal groups (up to 64)")
         if not 1 <= self.keep <= self.groups or self.keep * (self.choices // self.groups) < self.top:
             raise ConfigError(f"{self.keep} of {self.groups} groups cannot give {self.top} experts a token")
-        if self.act_params is not None and self.act_params[1] <= 0:
-            raise ConfigError(f"grouped_topk_moe: act_limit must be positive, got {self.act_params[1]}")
-        if self.act_params is None and self.act not in ("silu", "gelu_pytorch_tanh"):
-            raise ConfigError(f"grouped_topk_moe: unknown activation {self.act!r}")
 
     def weights(self):
         w = {"router": mat(self.choices, self.hidden)}
@@ -296,11 +298,13 @@ class GroupedTopKMoE(FeedForward):
 
 @FEED_FORWARDS.register("sigmoid_topk_moe")
 class SigmoidTopKMoE(FeedForward):
-    """A mixture of small ungated experts, expert(x) = W_down act(W_up x), with a sigmoid router: scores
+    """A mixture of small experts, ungated (expert(x) = W_down act(W_up x)) or gated, with a sigmoid router: scores
     s = sigmoid(W_router x) in float32; the ``top`` experts with the largest scores are chosen (the lower index
     among equals) and their scores are used as they are.  A score scales the expert's INPUT: the output is
     sum_e expert_e(s_e x).  Since W_up is linear, act(W_up (s x)) = act(s (W_up x)): the score is applied to the
-    up product's float32 sums, before the activation.  An optional shared expert of the same form runs on every
+    up product's float32 sums, before the activation.  With ``gated`` experts, W_down (unit of W_gate x and W_up x) with
+    the gated acts of ``gated_mlp`` (constants included), the rows are multiplied by their scores in float32 on their way to
+    the experts instead.  An optional shared expert of the same form runs on every
     token and is weighted by sigmoid(w_sg . x), one number a token; it rides along as one more row per token of
     the experts' pending rows.  (No counterpart in the reference, whose feed-forward is dense:
     crates/thuban_model/src/ops/mlp.rs:24-79.)
@@ -313,9 +317,10 @@ class SigmoidTopKMoE(FeedForward):
     shared expert is added as it is (no gate tensor).
 
     params: hidden_size, intermediate_size, num_experts, top, shared_intermediate_size (0: none), act ("gelu",
-    the erf form, or "gelu_pytorch_tanh", "silu", "relu2"); weighting ("input", the default, or "output"), groups,
+    the erf form, or "gelu_pytorch_tanh", "silu", "relu2"), gated (default false; weighting "input" and no shared expert);
+    weighting ("input", the default, or "output"), groups,
     keep_groups, correction, normalize, router_scale, shared_gate (default true).
-    tensors: router [E, H]; e{i}.up [I, H], e{i}.down [H, I]; shared.up [Is, H], shared.down [H, Is], shared.sg [1, H];
+    tensors: router [E, H]; e{i}.up [I, H], e{i}.down [H, I], gated also e{i}.gate [I, H]; shared.up [Is, H], shared.down [H, Is], shared.sg [1, H];
     correction [E]."""
 
     graph_safe = True
@@ -348,7 +353,12 @@ class SigmoidTopKMoE(FeedForward):
             raise ConfigError(f"{self.E} experts do not form {self.groups} equal groups (up to 64)")
         if not 1 <= self.keep <= self.groups or self.keep * (self.E // self.groups) < self.top:
             raise ConfigError(f"{self.keep} of {self.groups} groups cannot give {self.top} experts a token")
-        if self.act not in ("gelu", "gelu_pytorch_tanh", "silu", "relu2"):
+        self.gated, self.act_params = bool(p.get("gated", False)), None
+        if self.gated:
+            if self.weighting != "input" or self.shared:
+                raise ConfigError("sigmoid_topk_moe: gated experts go with weighting 'input' and without a shared expert")
+            self.act_params = gated_act_params("sigmoid_topk_moe", self.act, p)
+        elif self.act not in ("gelu", "gelu_pytorch_tanh", "silu", "relu2"):
             raise ConfigError(f"sigmoid_topk_moe: unknown activation {self.act!r}")
         if self.weighting == "input" and self.act == "relu2":
             raise ConfigError("sigmoid_topk_moe: act 'relu2' goes with weighting 'output'")
@@ -356,6 +366,8 @@ class SigmoidTopKMoE(FeedForward):
     def weights(self):
         w = {"router": mat(self.E, self.hidden)}
         for e in range(self.E):
+            if self.gated:
+                w[f"e{e}.gate"] = mat(self.inter, self.hidden)
             w[f"e{e}.up"] = mat(self.inter, self.hidden)
             w[f"e{e}.down"] = mat(self.hidden, self.inter)
         if self.shared:
@@ -372,7 +384,10 @@ class SigmoidTopKMoE(FeedForward):
             if self.shared and self.shared_gate else t["router"]
         self.w_correction = t.get("correction")
         dt = matmul_dtype(*(v for k, v in t.items() if k not in ("router", "shared.sg", "correction")))
-        self.w_up = torch.stack([t[f"e{e}.up"].to(dt) for e in range(self.E)], 0).contiguous()
+        up = lambda e: t[f"e{e}.up"].to(dt)
+        if self.gated:          # gate and up rows in the layout the kernels want: one product gives both
+            up = lambda e: self.ops.pair_gate_up(t[f"e{e}.gate"].to(dt), t[f"e{e}.up"].to(dt))
+        self.w_up = torch.stack([up(e) for e in range(self.E)], 0).contiguous()
         self.w_down = torch.stack([t[f"e{e}.down"].to(dt) for e in range(self.E)], 0).contiguous()
         if self.shared:
             self.w_sup, self.w_sdown = t["shared.up"].to(dt), t["shared.down"].to(dt)
@@ -394,11 +409,11 @@ class SigmoidTopKMoE(FeedForward):
                              weights=torch.empty((n_rows, k + extra), dtype=torch.float32, device=dev))
 
     def input_dtypes_when_routed(self):
-        return (self.w_up.dtype,)
+        return (torch.float32,) if self.gated else (self.w_up.dtype,)
 
     def forward(self, x, residual, step, routed=None):
         ops = self.ops
-        xa = x[self.w_up.dtype]
+        xa = x[torch.float32 if self.gated else self.w_up.dtype]
         T, dev, k, extra = xa.shape[0], xa.device, self.top, 1 if self.shared else 0
         if self.weighting == "output":
             return self._forward_output_weighted(x, xa, step, routed)
@@ -412,9 +427,15 @@ class SigmoidTopKMoE(FeedForward):
             weights = torch.empty((T, k + extra), dtype=torch.float32, device=dev)
             logits = torch.empty((T, self.E + extra), dtype=torch.float32, device=dev) if step.record is not None else None
             ops.router_sigmoid(x[torch.float32], self.w_router, self.E, k, ids, scores, weights, logits)
-        plan, xs = ops.moe_dispatch(ids, self.E, ops.moe_tile_rows(T, self.E, self.w_up.dtype, k, (self.hidden, self.inter)), xa)
+        tile = ops.moe_tile_rows(T, self.E, self.w_up.dtype, k, (self.hidden, self.inter))
         a = torch.empty((k * T, self.inter), dtype=self.w_up.dtype, device=dev)
-        ops.row_act(ops.gemm_partials(xs, self.w_up, plan=plan), a, self.act, row_of=plan.row_of, row_scale=scores)
+        if self.gated:
+            plan, xs = ops.moe_dispatch(ids, self.E, tile, xa, scale=scores, out_dtype=self.w_up.dtype)
+            kw = {} if self.act_params is None else {"act_params": self.act_params}
+            ops.gated_gemm(xs, self.w_up, a, self.act, plan, **kw)
+        else:
+            plan, xs = ops.moe_dispatch(ids, self.E, tile, xa)
+            ops.row_act(ops.gemm_partials(xs, self.w_up, plan=plan), a, self.act, row_of=plan.row_of, row_scale=scores)
         y = torch.empty(((k + extra) * T, self.hidden), dtype=torch.float32, device=dev)
         ops.grouped_gemm(a, self.w_down, y[:k * T], plan, plan_ready=True)
         row_of = plan.row_of

@@ -5,7 +5,8 @@ RMSNorm: y = x * rsqrt(mean(x^2) + eps) * gamma; with ``weight_offset`` c the st
 gamma = c + w (formed once, in float32, when the tensors are loaded).  Statistics are float32.  With
 ``branch_scale`` the norm also stores a scale s per channel for what a block adds before it, and ``post`` runs the
 norm after the sum: x <- norm(a x + s * branch) with a = ``residual_scale``, in place.  ``output_scale`` c multiplies the
-result (folded into gamma and beta when they are loaded).  The
+result (folded into gamma and beta when they are loaded).  ``one_number``: the stored scale is a single number for all
+coordinates.  The
 reference's norm shader has both as modes (crates/thuban_kernel/wgsl/norm.wgsl:66-83,
 112-121) and picks by config key (crates/thuban_architectures/src/phi.rs:55-63).
 """
@@ -14,6 +15,7 @@ from __future__ import annotations
 import torch
 
 from ..registry import NORMS
+from ..weights.sources import WeightSpec
 from .base import Norm, vec
 
 
@@ -32,10 +34,12 @@ class _RowNorm(Norm):
         self.residual_scale = float(params.get("residual_scale", 1.0))
         self.has_branch_scale = bool(params.get("branch_scale", False))
         self.output_scale = float(params.get("output_scale", 1.0))
+        self.one_number = bool(params.get("one_number", False))
         self.gamma = self.beta = self.branch_scale = None
 
     def weights(self):
-        w = {"weight": vec(self.width, init="normal" if self.weight_offset else "gamma")}
+        init = "normal" if self.weight_offset else "gamma"
+        w = {"weight": WeightSpec((), role="vector", init=init) if self.one_number else vec(self.width, init=init)}
         if self.has_bias:
             w["bias"] = vec(self.width)
         if self.has_branch_scale:
@@ -44,6 +48,8 @@ class _RowNorm(Norm):
 
     def load(self, tensors):
         self.gamma = tensors["weight"]
+        if self.one_number:
+            self.gamma = self.gamma.to(torch.float32).expand(self.width).contiguous()
         if self.weight_offset:
             self.gamma = (self.gamma.to(torch.float32) + self.weight_offset).contiguous()
         self.beta = tensors.get("bias")

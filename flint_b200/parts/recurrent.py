@@ -17,8 +17,9 @@ row v and S [dim, value_dim]:
     state space        S <- a S + B (dt x)^T;                                    y = S^T C + D x
 
 ``gated_delta``: q, k, v pass the convolution and SiLU; q and k become unit vectors per head (q also times
-dim^(-1/2)); beta = sigmoid(W_b x); g = exp(-exp(A_log) softplus(W_a2 W_a1 x + dt_bias)) per head and key channel; each
-head's o is divided by its root mean square, scaled by ``norm`` and by sigmoid(W_g2 W_g1 x), then projected.
+dim^(-1/2)); beta = sigmoid(W_b x); g = exp(-exp(A_log) softplus(W_a2 W_a1 x + dt_bias)) per head and key channel, or
+exp(-exp(A_log) softplus(W_a x + dt_bias)) per head; each head's o is divided by its root mean square, scaled by ``norm`` and by
+the gate, sigmoid(W_g2 W_g1 x) or act(W_g x), then projected.
 ``ssd``: W_in x = [z | x | B | C | dt]; x, B, C pass the convolution (with a bias) and SiLU; dt = softplus(dt + dt_bias),
 a = exp(-exp(A_log) dt); y times silu(z) is RMS-normed in ``norm_groups`` equal parts, scaled by ``norm`` and projected.
 Decays, step sizes, gates of the recurrence, unit norms and the state are float32 whatever the products run in.
@@ -68,9 +69,12 @@ class _Recurrent(Mixer):
 @MIXERS.register("gated_delta")
 class GatedDeltaRule(_Recurrent):
     """params: hidden_size, num_heads (value heads), num_kv_heads (query/key heads), dim, value_dim, conv_taps,
-    unit_eps, norm_eps.  tensors: q, k [G dim, hidden]; v [H value_dim, hidden]; q.conv, k.conv, v.conv [channels, taps];
-    b [H, hidden]; a1 [r, hidden], a2 [H dim, r], dt_bias [H dim], A_log [H]; g1 [r', hidden], g2 [H value_dim, r'];
-    norm [value_dim]; o [hidden, H value_dim].  The ranks r, r' are read from the tensors."""
+    unit_eps, norm_eps, head_decay (default false: a decay per key channel from a low-rank pair; true: one per head),
+    full_gate (default false: the gate through a low-rank pair; true: one matrix), gate_act ("sigmoid", the default, or
+    "silu").  tensors: q, k [G dim, hidden]; v [H value_dim, hidden]; q.conv, k.conv, v.conv [channels, taps];
+    b [H, hidden]; a1 [r, hidden], a2 [H dim, r], dt_bias [H dim], or a [H, hidden], dt_bias [H]; A_log [H]; g1 [r', hidden],
+    g2 [H value_dim, r'], or g [H value_dim, hidden]; norm [value_dim]; o [hidden, H value_dim].  The ranks r, r' are read
+    from the tensors."""
 
     def __init__(self, params, ctx):
         super().__init__(params, ctx)
@@ -85,28 +89,43 @@ class GatedDeltaRule(_Recurrent):
         self.unit_eps, self.eps = float(p["unit_eps"]), float(p["norm_eps"])
         self.rank_a = int(p.get("decay_rank", 0)) or None
         self.rank_g = int(p.get("gate_rank", 0)) or None
+        self.head_decay, self.full_gate = bool(p.get("head_decay", False)), bool(p.get("full_gate", False))
+        self.gate_act = p.get("gate_act", "sigmoid")
         self.conv_ch = 2 * self.G * self.D + self.H * self.V
 
     def weights(self):
         H, G, D, V, W, t = self.H, self.G, self.D, self.V, self.hidden, self.taps
         ra, rg = self.rank_a or max(W // 16, 1), self.rank_g or max(W // 16, 1)
         any_rank = lambda rows, cols: WeightSpec((rows, cols), role="matrix", free_dims=(0,))
-        return {"q": mat(G * D, W), "k": mat(G * D, W), "v": mat(H * V, W), "q.conv": conv_weight(G * D, t),
-                "k.conv": conv_weight(G * D, t), "v.conv": conv_weight(H * V, t), "b": mat(H, W), "a1": any_rank(ra, W),
-                "a2": WeightSpec((H * D, ra), std=0.2, free_dims=(1,)), "dt_bias": vec(H * D), "A_log": vec(H),
-                "g1": any_rank(rg, W), "g2": WeightSpec((H * V, rg), std=0.2, free_dims=(1,)), "norm": vec(V, init="gamma"), "o": mat(W, H * V)}
+        w = {"q": mat(G * D, W), "k": mat(G * D, W), "v": mat(H * V, W), "q.conv": conv_weight(G * D, t),
+             "k.conv": conv_weight(G * D, t), "v.conv": conv_weight(H * V, t), "b": mat(H, W)}
+        if self.head_decay:
+            w.update({"a": mat(H, W), "dt_bias": vec(H)})
+        else:
+            w.update({"a1": any_rank(ra, W), "a2": WeightSpec((H * D, ra), std=0.2, free_dims=(1,)), "dt_bias": vec(H * D)})
+        w["A_log"] = vec(H)
+        if self.full_gate:
+            w["g"] = mat(H * V, W)
+        else:
+            w.update({"g1": any_rank(rg, W), "g2": WeightSpec((H * V, rg), std=0.2, free_dims=(1,))})
+        w.update({"norm": vec(V, init="gamma"), "o": mat(W, H * V)})
+        return w
 
     def load(self, t):
-        names = ("q", "k", "v", "b", "a1", "g1")
-        dt = matmul_dtype(*(t[n] for n in names), t["o"], t["a2"], t["g2"])
-        self.ra, self.rg = t["a1"].shape[0], t["g1"].shape[0]
-        if t["a2"].shape[1] != self.ra or t["g2"].shape[1] != self.rg:
-            raise ConfigError(f"gated_delta: the low-rank pairs disagree (a1 {tuple(t['a1'].shape)} with a2 "
-                              f"{tuple(t['a2'].shape)}, g1 {tuple(t['g1'].shape)} with g2 {tuple(t['g2'].shape)})")
-        # one product gives q, k, v, the write strength's logit and the two low-rank inputs
+        low = () if self.head_decay else (("a1", "a2"),)
+        low += () if self.full_gate else (("g1", "g2"),)
+        for first, second in low:
+            if t[second].shape[1] != t[first].shape[0]:
+                raise ConfigError(f"gated_delta: the low-rank pairs disagree ({first} {tuple(t[first].shape)} with {second} "
+                                  f"{tuple(t[second].shape)})")
+        names = ("q", "k", "v", "b", "a" if self.head_decay else "a1", "g" if self.full_gate else "g1")
+        dt = matmul_dtype(*(t[n] for n in names), t["o"], *(t[second] for _, second in low))
+        # one product gives q, k, v, the write strength's logit and the decay's and the gate's columns (or low-rank inputs)
         self.w_in = torch.cat([t[n].to(dt) for n in names], 0).contiguous()
+        self.n_a, self.n_g = t[names[4]].shape[0], t[names[5]].shape[0]
         self.w_conv = torch.cat([t["q.conv"], t["k.conv"], t["v.conv"]], 0).contiguous()
-        self.w_a2, self.w_g2, self.w_o = t["a2"].to(dt), t["g2"].to(dt), t["o"].to(dt)
+        self.w_a2, self.w_g2 = (None if self.head_decay else t["a2"].to(dt)), (None if self.full_gate else t["g2"].to(dt))
+        self.w_o = t["o"].to(dt)
         self.dt_bias, self.a_log, self.w_norm = t["dt_bias"], t["A_log"], t["norm"]
 
     def input_dtypes(self):
@@ -126,14 +145,16 @@ class GatedDeltaRule(_Recurrent):
         C = self.conv_ch
         y = torch.empty((T, C), **f32)
         ops.short_conv(proj, 0, self.w_conv, None, "silu", step.pos, step.slot, conv_state, y)
-        # the low-rank second halves read float32 columns of the projection
-        c_b, c_a, c_g = C, C + H, C + H + self.ra
-        a = torch.empty((T, H * D), **f32)
-        ops.gemm(proj[:, c_a:c_a + self.ra], self.w_a2, a)
-        gate = torch.empty((T, H * V), **f32)
-        ops.gemm(proj[:, c_g:c_g + self.rg], self.w_g2, gate)
+        c_b, c_a, c_g = C, C + H, C + H + self.n_a
+        a, gate = proj[:, c_a:c_g], proj[:, c_g:c_g + self.n_g]
+        if not self.head_decay:       # the low-rank second halves read float32 columns of the projection
+            low, a = a, torch.empty((T, H * D), **f32)
+            ops.gemm(low, self.w_a2, a)
+        if not self.full_gate:
+            low, gate = gate, torch.empty((T, H * V), **f32)
+            ops.gemm(low, self.w_g2, gate)
         qk = torch.empty((T, 2 * G * D), **f32)
-        decay = torch.empty((T, H * D), **f32)
+        decay = torch.empty((T, H if self.head_decay else H * D), **f32)
         beta = torch.empty((T, H), **f32)
         ops.delta_prepare(y, proj[:, c_b:c_b + H], a, self.dt_bias, self.a_log, qk, decay, beta, H, G, D, self.unit_eps)
         o = torch.empty((T, H * V), **f32)
@@ -141,7 +162,7 @@ class GatedDeltaRule(_Recurrent):
                             request_starts(step), len(step.entries), S, o, H, G, D, V)
         act = self.ctx.act_dtype if self.w_o.dtype == torch.bfloat16 else torch.float32
         out = torch.empty((T, H * V), dtype=act, device=dev)
-        ops.gated_norm(o, gate, "sigmoid", False, self.w_norm, self.eps, H, out)
+        ops.gated_norm(o, gate, self.gate_act, False, self.w_norm, self.eps, H, out)
         return Pending(partials=ops.gemm_partials(out, self.w_o))
 
 

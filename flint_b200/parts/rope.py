@@ -1,4 +1,4 @@
-"""Rotary position encoding with optional LongRoPE or YaRN scaling.
+"""Rotary position encoding with optional linear, banded, LongRoPE or YaRN scaling.
 
 The cos/sin tables are built on the host in float64 and stored as float32
 [positions, rotary_dim/2]: inv_i = theta^(-2i/rot), divided by the short factor for
@@ -27,7 +27,10 @@ class RotaryEncoding(PositionEncoding):
     short_factor, long_factor, original_max_positions, short_mscale, long_mscale.  For YaRN: ``yarn`` = {factor,
     original, fast, slow}: with dim(t) = rot ln(original / (2 pi t)) / (2 ln theta), lo = max(floor(dim(fast)), 0),
     hi = min(ceil(dim(slow)), rot - 1) and ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), frequency i is
-    inv_i / factor * ramp_i + inv_i (1 - ramp_i), and cos and sin are multiplied by 0.1 ln(factor) + 1.  The tables
+    inv_i / factor * ramp_i + inv_i (1 - ramp_i), and cos and sin are multiplied by 0.1 ln(factor) + 1.  ``linear`` =
+    factor: every frequency is divided by it.  ``banded`` = {factor, low, high, original} (as in Llama 3.1): with the
+    wavelength l = 2 pi / inv_i, frequency i stays for l < original / high, is divided by the factor for l > original / low,
+    and between the two is (1 - s) inv_i / factor + s inv_i with s = (original / l - low) / (high - low).  The tables
     cover the positions the model is built to serve (``BuildContext.max_context``) when that is fewer than
     ``max_positions``."""
 
@@ -72,7 +75,20 @@ class RotaryEncoding(PositionEncoding):
                 ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0, 1)
                 ang = pos[:, None] * (inv / factor * ramp + inv * (1 - ramp))[None, :]
                 scale = torch.full((1, 1), 0.1 * math.log(factor) + 1, dtype=torch.float64)
+            elif p.get("banded") is not None:
+                b = {k: float(p["banded"][k]) for k in ("factor", "low", "high", "original")}
+                if min(b.values()) <= 0 or b["high"] < b["low"]:
+                    raise ConfigError("banded frequencies: factor, low, high and original must be positive, high at least low")
+                turns = b["original"] * inv / (2 * math.pi)           # original / wavelength
+                share = ((turns - b["low"]) / max(b["high"] - b["low"], 1e-30)).clamp(0, 1)
+                ang = pos[:, None] * torch.where(turns > b["high"], inv, torch.where(
+                    turns < b["low"], inv / b["factor"], (1 - share) * inv / b["factor"] + share * inv))[None, :]
+                scale = torch.ones((1, 1), dtype=torch.float64)
             else:
+                if p.get("linear") is not None:
+                    if float(p["linear"]) <= 0:
+                        raise ConfigError(f"the frequencies' divisor must be positive, got {p['linear']}")
+                    inv = inv / float(p["linear"])
                 ang = pos[:, None] * inv[None, :]
                 scale = torch.ones((1, 1), dtype=torch.float64)
             cos = (torch.cos(ang) * scale).to(torch.float32).contiguous().to(self.ctx.device)

@@ -97,7 +97,25 @@ class RefOps:
                 self.router_sparsemixer(tmp, router.weight, router.jitter_eps, router.expert_ids, router.gates,
                                         getattr(router, "logits", None))
 
+    def row_post(self, x, pending=None, out=None, router=None, conv=None):
+        if pending is not None:
+            branches = ([(pending.partials, pending.bias, 1.0)] if pending.partials is not None else []) + list(pending.branches)
+            rows = (pending.y, pending.row_of, pending.gates) if pending.y is not None else None
+            self.sum_norm_add(x, [b[:2] for b in branches], [b[2] for b in branches], expert_rows=rows, gamma=pending.gamma,
+                              eps=pending.eps)
+        if conv is not None:
+            w, ring, pos, slot = conv
+            self.short_conv(x, 0, w, None, "plus_input", pos, slot, ring, out)
+        elif out is not None:
+            out.copy_(x.to(torch.float32).to(out.dtype))
+        if router is not None:
+            assert router.rule == "sigmoid"
+            self.router_sigmoid(x, router.weight, router.weight.shape[0] - router.extra, router.top, router.expert_ids,
+                                router.gates, router.weights, getattr(router, "logits", None))
+
     def apply_pending(self, x, pending):
+        if pending.alone:
+            return self.row_post(x, pending)
         if x.dim() == 3:
             r = torch.zeros((x.shape[0], x.shape[2]), dtype=self.cd)
             if pending.partials is not None:
@@ -392,7 +410,7 @@ class RefOps:
                 state[sl, r * C:(r + 1) * C] = x[t].to(state.dtype)
         if bias is not None:
             res = res + bias.to(self.cd)
-        y.copy_(_act(res, act).to(y.dtype))
+        y.copy_((x + res if act == "plus_input" else _act(res, act)).to(y.dtype))
 
     def delta_prepare(self, y, b, a, dt_bias, a_log, qk, decay, beta, H, G, D, unit_eps):
         T = y.shape[0]
@@ -401,8 +419,8 @@ class RefOps:
         x[:, :G] = x[:, :G] * D ** -0.5
         qk.copy_(x.reshape(T, 2 * G * D).to(qk.dtype))
         beta.copy_(torch.sigmoid(b.to(self.cd)).to(beta.dtype))
-        sp = torch.nn.functional.softplus(a.to(self.cd) + dt_bias.to(self.cd), threshold=30.0).view(T, H, D)
-        decay.copy_(torch.exp(-torch.exp(a_log.to(self.cd)).view(1, H, 1) * sp).reshape(T, H * D).to(decay.dtype))
+        sp = torch.nn.functional.softplus(a.to(self.cd) + dt_bias.to(self.cd), threshold=30.0).view(T, H, -1)
+        decay.copy_(torch.exp(-torch.exp(a_log.to(self.cd)).view(1, H, 1) * sp).reshape(decay.shape).to(decay.dtype))
 
     def ssd_prepare(self, raw, dt_bias, a_log, dt, decay):
         d = torch.nn.functional.softplus(raw.to(self.cd) + dt_bias.to(self.cd), threshold=30.0)
@@ -412,7 +430,7 @@ class RefOps:
     def recurrence_scan(self, q, k, v, decay, delta, beta, dt, skip, slot, seq_start, n_seq, state, out, H, G, D, V):
         T = q.shape[0]
         qq, kk, vv = q.to(self.cd).view(T, G, D), k.to(self.cd).view(T, G, D), v.to(self.cd).view(T, H, V)
-        dec = decay.to(self.cd).view(T, H, D) if delta else decay.to(self.cd)
+        dec = decay.to(self.cd).view(T, H, -1).expand(T, H, D) if delta else decay.to(self.cd)      # per channel or per head
         starts = list(range(n_seq + 1)) if seq_start is None else seq_start.tolist()
         res = torch.zeros(T, H, V, dtype=self.cd)
         for e in range(n_seq):
@@ -833,10 +851,15 @@ class RefOps:
         return MoePlan(n_experts, tile_rows, max_tiles, i32(counts), i32(offsets), i32(row_of).view(-1, top),
                        i32(token_of), pad(tiles_e), pad(tiles_r), i32([len(tiles_e)]), top)
 
-    def moe_dispatch(self, expert_ids, n_experts, tile_rows, x):
+    def moe_dispatch(self, expert_ids, n_experts, tile_rows, x, scale=None, out_dtype=None):
         plan = self.moe_plan(expert_ids, n_experts, tile_rows)
         xs = torch.empty((plan.token_of.numel(), x.shape[1]), dtype=x.dtype)
         self.gather_rows(x, plan.token_of, xs)
+        if scale is not None:
+            row = plan.row_of.reshape(-1).long()
+            mine = row < xs.shape[0]
+            xs[row[mine]] *= scale.reshape(-1)[mine].to(xs.dtype)[:, None]
+            xs = xs.to(out_dtype or xs.dtype)
         return plan, xs
 
     # ------------------------------------------------------------------ sampling
