@@ -836,6 +836,121 @@ def run_sinilorn_pair(args, pk, rng):
     return out
 
 
+def sokipel_config(width, heads, kv_heads, dim, vdim, chunk, rot, d_heads, d_kv_heads, d_dim, d_vdim, ff, experts, top, layers,
+                   vocab, taps=4, canon=3):
+    """A Sokipel configuration of ``layers`` layers in the order delta rule, parallel mixer (gated attention over the whole
+    sequence beside a delta rule), attention in chunks, delta rule, ...; every layer with a mixture of clamped experts."""
+    head = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5}
+    delta = {"heads": d_heads, "kv_heads": d_kv_heads, "dim": d_dim, "vdim": d_vdim, "conv": taps}
+    mlp = {"kind": "moe", "expert": {"ff": ff, "limit": 7.0}, "router": {"experts": experts, "top": top}}
+    out = []
+    for i in range(layers):
+        if i % 4 == 1:
+            kind = "parallel"
+            m = {"left": {**head, "rot": {"dims": rot, "base": 5e5, "scaling": {"factor": 2.0}}}, "right": delta,
+                 "left_scale": 1.0, "right_scale": 1.0}
+        elif i % 4 == 2:
+            kind = "attention"
+            m = {**head, "mask": {"size": chunk}, "rot": {"dims": dim, "base": 5e5, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0,
+                                                                                              "original": 8192}}}
+        else:
+            kind, m = "delta", delta
+        out.append({"type": kind, "mixer": m, "mlp": mlp})
+    return {"architecture": "Sokipel", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": float(width) ** 0.5},
+            "residual_mult": 0.5, "canon": {"taps": canon}, "logit_softcap": 30.0, "layers": out}
+
+
+# layer sizes that resemble real models of this kind, beside a Tefovik of equal width, attention heads and delta-rule heads
+# whose attention sees as far (its runs are longer than the prompt) and whose feed-forward has the parameters that a token's
+# experts have
+SOKIPEL_SIZES = {
+    "2048x16": dict(width=2048, heads=16, kv_heads=4, dim=128, vdim=128, chunk=4096, rot=64, d_heads=16, d_kv_heads=8, d_dim=128,
+                    d_vdim=128, ff=1408, experts=16, top=2,
+                    tefovik=dict(width=2048, heads=16, kv_heads=4, dim=128, vdim=128, chunk=4096, rot=64, d_heads=16, d_kv_heads=8,
+                                 d_dim=128, d_vdim=128, s_heads=64, s_vdim=64, s_state=128, s_groups=8, ff=4224)),
+    "4096x32": dict(width=4096, heads=32, kv_heads=8, dim=128, vdim=128, chunk=4096, rot=64, d_heads=32, d_kv_heads=16, d_dim=128,
+                    d_vdim=128, ff=1408, experts=32, top=4,
+                    tefovik=dict(width=4096, heads=32, kv_heads=8, dim=128, vdim=128, chunk=4096, rot=64, d_heads=32, d_kv_heads=16,
+                                 d_dim=128, d_vdim=128, s_heads=128, s_vdim=64, s_state=128, s_groups=8, ff=8448)),
+}
+
+
+def run_sokipel_pair(args, pk, rng):
+    """Prefill and decode of Sokipel at layer sizes that resemble real models, beside Tefovik at equal width, heads and state
+    shape: tokens/s, and for the kernels of both the time a launch and, for attention, recurrences and expert products, the
+    distance from the roofline (decode: cache, state or weight bytes over the measured copy bandwidth; prefill: flops over
+    the sustained library product rate, for the recurrences over the chip's float32 multiply-add rate)."""
+    import torch
+    layers = args.layers or 8
+    vocab = args.vocab or 32064
+    batch, ctx = args.batch, args.prompt_tokens
+    fp32_rate = FP32_FMA_LANES * 2 * 1.965e9
+    out = {"design": "Sokipel", "beside": "Tefovik", "layers": layers, "batch": batch, "prompt_tokens": ctx, "dtype": "bf16",
+           "data": "synthetic: seeded random weights, uniform-random token ids",
+           "peaks": {**{k: pk[k] for k in ("hbm_gbs", "bf16_tflops_sustained", "source")},
+                     "fp32_tflops_nominal": round(fp32_rate / 1e12, 1)}, "sizes": {}}
+    for name, sz in SOKIPEL_SIZES.items():
+        if args.design_sizes and name not in args.design_sizes:
+            continue
+        cfgs = {"sokipel": sokipel_config(**{k: v for k, v in sz.items() if k != "tefovik"}, layers=layers, vocab=vocab),
+                "tefovik": tefovik_config(**sz["tefovik"], layers=layers, vocab=vocab)}
+        row = {}
+        for which, cfg in cfgs.items():
+            cfg.setdefault("vocab_size", cfg.get("vocab"))
+            model = build_model(cfg, max(batch, 1), ctx + 256)
+            pre_ms = run_prefill(model, cfg, ctx, reps=3, warmup=3, rng=rng)
+            dec = run_decode(model, cfg, batch, ctx, args.steps, max(args.warmup, 3), rng, count_experts=False)
+            pre_t, dec_t, distinct = profile_tables(model, cfg, batch, ctx, rng)
+            graph = graph_step_table(model, cfg, batch, ctx, rng)
+            kv = ctx + 2
+            tokens = {"prefill": ctx, "decode": batch}
+            h, d = (sz[k] for k in ("heads", "d_heads"))
+            att_bytes = batch * min(kv, sz["chunk"]) * sz["kv_heads"] * (sz["dim"] + sz["vdim"]) * 2
+            att_flops = sum(2 * h * (sz["dim"] + sz["vdim"]) * k for k in range(1, ctx + 1))
+            state = {"delta": (d * sz["d_dim"] * sz["d_vdim"], 9)}       # elements of a layer's state, flops an element costs a token
+            if which == "tefovik":
+                t = sz["tefovik"]
+                state["ssd"] = (t["s_heads"] * t["s_state"] * t["s_vdim"], 5)
+            tables = [("prefill", pre_t), ("decode", dec_t)] + ([("decode, captured", graph[0])] if graph else [])
+            kern = {}
+            for kind, table in tables:
+                decoding = kind != "prefill"
+                for kname, (n, ms) in sorted(table.items()):
+                    secs = ms / n * 1e-3
+                    e = {"launches": n, "us": round(secs * 1e6, 2)}
+                    scan = next((s for s in state if kname.startswith(("flint_recurrence_scan " + s, "flint_delta_token"))), None)
+                    if scan is not None:
+                        elems, flops = state[scan]
+                        if decoding:                # the state is read and written once a token
+                            e["frac_of_copy_bandwidth"] = round(batch * elems * 4 * 2 / secs / 1e9 / pk["hbm_gbs"], 4)
+                        else:
+                            e["frac_of_fp32_rate"] = round(ctx * elems * flops / secs / fp32_rate, 4)
+                            e["ns_per_token"] = round(secs * 1e9 / ctx, 1)
+                    elif kname.startswith("flint_sink_attention"):
+                        if decoding:
+                            e["frac_of_copy_bandwidth"] = round(att_bytes / secs / 1e9 / pk["hbm_gbs"], 4)
+                        else:
+                            e["frac_of_sustained_product_rate"] = round(att_flops / secs / (pk["bf16_tflops_sustained"] * 1e12), 4)
+                    elif kname.startswith("flint_gemm_tc "):
+                        shape = kname.split()[1]
+                        N, K = (int(v) for v in shape.split("x"))
+                        gated = 2 if kname.split()[2:3] == ["gated"] else 1
+                        if decoding:
+                            mats = sum(distinct) / len(distinct) if kname.endswith("experts") and distinct else 1
+                            e["frac_of_copy_bandwidth"] = round(mats * gated * N * K * 2 / secs / 1e9 / pk["hbm_gbs"], 4)
+                        else:
+                            rows = tokens[kind] * (sz["top"] if kname.endswith("experts") else 1)
+                            e["frac_of_sustained_product_rate"] = round(2 * rows * gated * N * K / secs / (pk["bf16_tflops_sustained"] * 1e12), 4)
+                    kern[f"{kind}: {kname}"] = e
+            row[which] = {"prefill_tok_s": round(ctx * 1000.0 / pre_ms, 1), "prefill_ms": round(pre_ms, 3),
+                          "decode_tok_s": round(dec["tok_s"], 1), "decode_ms_per_step": round(dec["ms"], 4),
+                          "decode_launches": dec["launches"], "weight_gb": round(model.weight_bytes() / 1e9, 2), "kernels": kern}
+            del model
+            torch.cuda.empty_cache()
+        out["sizes"][name] = row
+    return out
+
+
 def run_design_pair(args, pk, rng):
     """Prefill and decode of Puledra or Gepadra at layer sizes that resemble real models, beside Phi-MoE at equal width, heads
     and active expert parameters: tokens/s, and for the attention kernels of both the time a layer and the
@@ -1005,7 +1120,7 @@ def graph_step_table(model, cfg, batch, prompt_len, rng):
                          if e.device_type == torch.autograd.DeviceType.CUDA and "Memcpy" not in e.name and "Memset" not in e.name))
         except Exception:            # no CUPTI here: the caller falls back to the eager table
             ev = []
-        followers = ("splitk_reduce", "attention_combine")      # second kernels of a launcher call
+        followers = ("splitk_reduce", "attention_combine", "sink_combine", "short_conv_keep")      # second kernels of a launcher call
         paired, i = [], 0
         for start, end, name in ev:
             if any(f in name for f in followers) and paired:
@@ -1156,9 +1271,10 @@ def main():
     ap.add_argument("--sweep", action="store_true",
                     help="instead of the default run: decode at batch 1 and 8 with contexts of 16,384 and 65,536 tokens, "
                          "batch 1 with 131,008, and batch 128 and 256 with 2,048, each with its roofline fraction")
-    ap.add_argument("--design", choices=["puledra", "gepadra", "tefovik", "dumizen", "sinilorn"], default=None,
+    ap.add_argument("--design", choices=["puledra", "gepadra", "tefovik", "dumizen", "sinilorn", "sokipel"], default=None,
                     help="prefill and decode of this design at layer sizes that resemble real models, beside the closest "
-                         "earlier model at equal sizes (Phi-MoE; for tefovik and dumizen Gepadra, for sinilorn Puledra), with its kernels' shares of the peaks")
+                         "earlier model at equal sizes (Phi-MoE; for tefovik and dumizen Gepadra, for sinilorn Puledra, for sokipel Tefovik), with its "
+                         "kernels' shares of the peaks")
     ap.add_argument("--design-sizes", nargs="+", default=None, help="which of the design's size points to run")
     ap.add_argument("--profile", action="store_true",
                     help="print per-kernel device times of one prefill and one decode step to stderr and exit")
@@ -1190,7 +1306,8 @@ def main():
         print(json.dumps(run_tiny(args.tiny)))
         return 0
     if args.design:
-        run = {"tefovik": run_tefovik_pair, "dumizen": run_dumizen_pair, "sinilorn": run_sinilorn_pair}.get(args.design, run_design_pair)
+        run = {"tefovik": run_tefovik_pair, "dumizen": run_dumizen_pair, "sinilorn": run_sinilorn_pair,
+               "sokipel": run_sokipel_pair}.get(args.design, run_design_pair)
         print(json.dumps(run(args, pk, rng)))
         return 0
     if args.sweep:

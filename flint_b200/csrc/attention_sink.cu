@@ -19,6 +19,8 @@
 // a lane owns a key in the score phase and value dims lane, lane + 32, ... in the value phase.  With several
 // splits a second kernel merges (max, sum, unnormalised output) records in a fixed order and adds the sink.
 // Head sizes up to 256; rows of whole 16-byte units are read in such units, others element by element.
+// In bfloat16, with head sizes in multiples of 16 up to 128 and a softmax, the rows run on the tensor cores instead
+// (flint_sink_attention_rows): a block per row, key head, chunk of up to 16 query heads and split.
 //
 // The reference's attention has the causal and window mask only (crates/thuban_kernel/wgsl/attn.wgsl:78-90).
 #include <math.h>
@@ -645,6 +647,212 @@ sink_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat
   }
 }
 
+// ------------------------------------------------------------------------------------------- single rows on the tensor cores
+// A row (bfloat16, head sizes in multiples of 16 up to 128), a key head and a run of its seen keys: one block of four warps.
+// Up to 16 query heads of the group are the 16 rows of the mma's A operand.  The keys are numbered as above and walked in tiles
+// of 64 in two alternating stages (asynchronous 16-byte copies, two threads a key); each warp takes 16 keys of every tile with
+// a maximum, sum and output of its own, so the warps meet only at the end, through shared memory.  A seen key needs no mask:
+// only the last tile of the run is cut.
+template <int HDS, int VDT>
+__global__ void __launch_bounds__(128)
+sink_attention_rows_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_cache,
+                           const __nv_bfloat16* __restrict__ v_cache, const int* __restrict__ block_table, int max_pages,
+                           int page_size, const int* __restrict__ pos, const int* __restrict__ slot,
+                           __nv_bfloat16* __restrict__ out, float* __restrict__ scratch, int nq, int nkv, int hd, int vd,
+                           int window, int keep_first, int run, const float* __restrict__ sinks, float scale, int split_keys,
+                           int n_splits, int g_chunks, const int* __restrict__ row_list, const __nv_bfloat16* __restrict__ pool_k,
+                           const __nv_bfloat16* __restrict__ pool_v, int pool, int pool_slots) {
+  extern __shared__ __align__(16) unsigned char sm_raw[];
+  __shared__ float m_s[4][16], l_s[4][16];
+  const int ldk = hd + 8, ldv = vd + 8, stage_bytes = MK * (ldk + ldv) * 2;
+  pdl_launch();
+  pdl_wait();
+  int item = blockIdx.x;
+  const int split = item % n_splits;
+  item /= n_splits;
+  const int gchunk = item % g_chunks;
+  item /= g_chunks;
+  const int kvh = item % nkv, ti = item / nkv;
+  const int t = row_list ? row_list[ti] : ti;
+  const int G = nq / nkv, ng = min(16, G - gchunk * 16), h0 = kvh * G + gchunk * 16;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
+  const int hd16 = hd / 16, vdt = vd / 8, chunks_k = hd / 8, chunks_v = vd / 8;
+  const int lm = lane >> 3, lr = lane & 7;
+  const int p = pos[t];
+  const int lo = run > 0 ? (p / run) * run : (window > 0 ? max(0, p + 1 - window) : 0);
+  const int n_first = pool > 0 ? max(0, (p - window + 1) / pool) : min(keep_first, lo);
+  const int total = n_first + (p + 1 - lo);
+  const int u_lo = split * split_keys, u_hi = min(total, u_lo + split_keys);
+  const int* bt = block_table + (size_t)slot[t] * max_pages;
+
+  auto fetch = [&](int u0, int stage) {
+    __nv_bfloat16* k_d = reinterpret_cast<__nv_bfloat16*>(sm_raw + (size_t)stage * stage_bytes);
+    __nv_bfloat16* v_d = k_d + MK * ldk;
+    const int r = tid >> 1, half = tid & 1, u = u0 + r;
+    long long at = -1;
+    const __nv_bfloat16 *ks = k_cache, *vs = v_cache;
+    if (u < u_hi) {
+      if (pool > 0 && u < n_first) {
+        const int page = bt[u / pool_slots];
+        if (page >= 0) at = ((long long)page * nkv + kvh) * pool_slots + u % pool_slots;
+        ks = pool_k;
+        vs = pool_v;
+      } else {
+        const int j = u < n_first ? u : lo + (u - n_first);
+        const int page = bt[j / page_size];
+        if (page >= 0) at = ((long long)page * nkv + kvh) * page_size + j % page_size;
+      }
+    }
+    __nv_bfloat16* kd = k_d + r * ldk;
+    __nv_bfloat16* vd_ = v_d + r * ldv;
+    if (at >= 0) {
+      for (int c = half; c < chunks_k; c += 2) copy16(kd + c * 8, ks + at * hd + c * 8);
+      for (int c = half; c < chunks_v; c += 2) copy16(vd_ + c * 8, vs + at * vd + c * 8);
+    } else {
+      for (int c = half; c < chunks_k; c += 2) *reinterpret_cast<uint4*>(kd + c * 8) = make_uint4(0u, 0u, 0u, 0u);
+      for (int c = half; c < chunks_v; c += 2) *reinterpret_cast<uint4*>(vd_ + c * 8) = make_uint4(0u, 0u, 0u, 0u);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  if (u_lo < u_hi) fetch(u_lo, 0);
+
+  // the heads' queries as A fragments, straight from memory: heads g and g + 8, dims 2 tq and 2 tq + 8 of every step
+  uint32_t qf[HDS][4];
+#pragma unroll
+  for (int ks = 0; ks < HDS; ++ks)
+    if (ks < hd16) {
+      const __nv_bfloat16* q0 = q + ((size_t)t * nq + h0 + g) * hd + ks * 16 + 2 * tq;
+      const __nv_bfloat16* q1 = q0 + (size_t)8 * hd;
+      qf[ks][0] = g < ng ? *reinterpret_cast<const uint32_t*>(q0) : 0u;
+      qf[ks][1] = g + 8 < ng ? *reinterpret_cast<const uint32_t*>(q1) : 0u;
+      qf[ks][2] = g < ng ? *reinterpret_cast<const uint32_t*>(q0 + 8) : 0u;
+      qf[ks][3] = g + 8 < ng ? *reinterpret_cast<const uint32_t*>(q1 + 8) : 0u;
+    }
+  float m_r[2] = {-INFINITY, -INFINITY}, l_r[2] = {0.f, 0.f};
+  float o[VDT][4];
+#pragma unroll
+  for (int nt = 0; nt < VDT; ++nt)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) o[nt][e] = 0.f;
+
+  int stage = 0;
+  for (int u0 = u_lo; u0 < u_hi; u0 += MK, stage ^= 1) {
+    if (u0 + MK < u_hi) {
+      fetch(u0 + MK, stage ^ 1);
+      asm volatile("cp.async.wait_group 1;" ::: "memory");
+    } else {
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
+    }
+    __syncthreads();
+    const __nv_bfloat16* k_s = reinterpret_cast<const __nv_bfloat16*>(sm_raw + (size_t)stage * stage_bytes) + warp * 16 * ldk;
+    const __nv_bfloat16* v_s = reinterpret_cast<const __nv_bfloat16*>(sm_raw + (size_t)stage * stage_bytes) + MK * ldk + warp * 16 * ldv;
+    const int left = u_hi - u0 - warp * 16;                  // keys of this warp's 16 that are seen
+    if (left > 0) {
+      float s[2][4];
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) s[nt][e] = 0.f;
+#pragma unroll
+      for (int ks = 0; ks < HDS; ++ks)
+        if (ks < hd16) {
+          uint32_t b0, b1, b2, b3;
+          const __nv_bfloat16* src = k_s + ((lm >> 1) * 8 + lr) * ldk + ks * 16 + (lm & 1) * 8;
+          ldsm4((uint32_t)__cvta_generic_to_shared(src), b0, b1, b2, b3);
+          mma16816(s[0], qf[ks], b0, b1);
+          mma16816(s[1], qf[ks], b2, b3);
+        }
+      float mx[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          s[nt][e] = nt * 8 + 2 * tq + (e & 1) < left ? s[nt][e] * scale : -INFINITY;
+          mx[e >> 1] = fmaxf(mx[e >> 1], s[nt][e]);
+        }
+      float alpha[2], sum[2] = {0.f, 0.f};
+#pragma unroll
+      for (int rs = 0; rs < 2; ++rs) {
+        mx[rs] = fmaxf(mx[rs], __shfl_xor_sync(0xffffffffu, mx[rs], 1));
+        mx[rs] = fmaxf(mx[rs], __shfl_xor_sync(0xffffffffu, mx[rs], 2));
+        const float m_new = fmaxf(m_r[rs], mx[rs]);            // finite: the warp's first key is seen
+        alpha[rs] = __expf(m_r[rs] - m_new);
+        m_r[rs] = m_new;
+      }
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          s[nt][e] = __expf(s[nt][e] - m_r[e >> 1]);
+          sum[e >> 1] += s[nt][e];
+        }
+#pragma unroll
+      for (int rs = 0; rs < 2; ++rs) l_r[rs] = l_r[rs] * alpha[rs] + sum[rs];      // a lane's own columns; summed at the end
+#pragma unroll
+      for (int nt = 0; nt < VDT; ++nt) {
+        o[nt][0] *= alpha[0]; o[nt][1] *= alpha[0];
+        o[nt][2] *= alpha[1]; o[nt][3] *= alpha[1];
+      }
+      const uint32_t a[4] = {pack_bf16(s[0][0], s[0][1]), pack_bf16(s[0][2], s[0][3]), pack_bf16(s[1][0], s[1][1]),
+                             pack_bf16(s[1][2], s[1][3])};
+#pragma unroll
+      for (int vp = 0; vp < VDT / 2; ++vp)
+        if (2 * vp < vdt) {
+          uint32_t b0, b1, b2, b3;
+          const __nv_bfloat16* src = v_s + ((lm & 1) * 8 + lr) * ldv + vp * 16 + (lm >> 1) * 8;
+          ldsm4t((uint32_t)__cvta_generic_to_shared(src), b0, b1, b2, b3);
+          mma16816(o[2 * vp], a, b0, b1);
+          mma16816(o[2 * vp + 1], a, b2, b3);
+        }
+    }
+    __syncthreads();        // this stage is refilled in the next round
+  }
+
+  // the four warps' records meet in shared memory: outputs [4][16][vd + 4], maxima and sums [4][16]
+  float* o_s = reinterpret_cast<float*>(sm_raw);
+  const int ldo = vd + 4;
+#pragma unroll
+  for (int rs = 0; rs < 2; ++rs) {
+    l_r[rs] += __shfl_xor_sync(0xffffffffu, l_r[rs], 1);
+    l_r[rs] += __shfl_xor_sync(0xffffffffu, l_r[rs], 2);
+    if (tq == 0) {
+      m_s[warp][g + 8 * rs] = m_r[rs];
+      l_s[warp][g + 8 * rs] = l_r[rs];
+    }
+#pragma unroll
+    for (int nt = 0; nt < VDT; ++nt)
+      if (nt < vdt && g + 8 * rs < ng)
+        *reinterpret_cast<float2*>(o_s + (size_t)(warp * 16 + g + 8 * rs) * ldo + nt * 8 + 2 * tq) = make_float2(o[nt][2 * rs], o[nt][2 * rs + 1]);
+  }
+  __syncthreads();
+  for (int i = tid; i < ng * vd; i += 128) {
+    const int hh = i / vd, d = i % vd;
+    float M = -INFINITY;
+#pragma unroll
+    for (int w = 0; w < 4; ++w) M = fmaxf(M, m_s[w][hh]);
+    const bool last = n_splits == 1;
+    const float sk = last && sinks ? sinks[h0 + hh] : -INFINITY;
+    M = fmaxf(M, sk);
+    float L = sk > -INFINITY ? expf(sk - M) : 0.f, acc = 0.f;
+#pragma unroll
+    for (int w = 0; w < 4; ++w) {
+      const float f = m_s[w][hh] > -INFINITY ? expf(m_s[w][hh] - M) : 0.f;
+      L += f * l_s[w][hh];
+      acc += f * o_s[(size_t)(w * 16 + hh) * ldo + d];
+    }
+    if (last) {
+      out[((size_t)t * nq + h0 + hh) * vd + d] = __float2bfloat16_rn(L > 0.f ? acc / L : 0.f);
+    } else {
+      float* dst = scratch + (((size_t)ti * nq + h0 + hh) * n_splits + split) * (vd + 2);
+      dst[d] = acc;
+      if (d == 0) {
+        dst[vd] = M;
+        dst[vd + 1] = L;
+      }
+    }
+  }
+}
+
 }  // namespace
 
 extern "C" int flint_qkv_write(const float* qkv, int n_partials, long long partial_stride, const float* bias,
@@ -770,6 +978,46 @@ extern "C" int flint_sink_attention_tiles(const void* q, const void* k_cache, co
     launch_pdl(sink_attention_mma_kernel<8, 16>, grid, block, smem, stream, qq, kk, vv, block_table, max_pages, page_size, tiles,
                (__nv_bfloat16*)out, nq, nkv, hd, vd, window, keep_first, run, sinks, scale, pk, pv, pool, pool_slots, sw);
   return check_launch("sink_attention_tiles");
+}
+
+// The rows of flint_sink_attention on the tensor cores: bfloat16 q, cache and out; head sizes in multiples of 16 up to 128.
+extern "C" int flint_sink_attention_rows(const void* q, const void* k_cache, const void* v_cache, const int* block_table,
+                                         int max_pages, int page_size, const int* pos, const int* slot, void* out, int T, int nq,
+                                         int nkv, int hd, int vd, int window, int keep_first, int run, const float* sinks,
+                                         float scale, int split_keys, int n_splits, float* scratch, const int* row_list,
+                                         const void* pool_k, const void* pool_v, int pool, int pool_slots, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (hd < 16 || vd < 16 || hd % 16 || vd % 16 || hd > 128 || vd > 128)
+    return fail("sink_attention_rows: head sizes %d and %d (multiples of 16 up to 128)", hd, vd);
+  if (nkv <= 0 || nq % nkv) return fail("sink_attention_rows: %d query heads do not divide into %d kv heads", nq, nkv);
+  if (n_splits < 1 || split_keys < 1 || (n_splits > 1 && !scratch)) return fail("sink_attention_rows: bad splits, or no scratch memory");
+  if (window < 0 || keep_first < 0 || page_size <= 0 || run < 0 || (run > 0 && (window > 0 || keep_first > 0)))
+    return fail("sink_attention_rows: bad window or page size");
+  if (pool < 0 || (pool > 0 && (window < 1 || keep_first > 0 || run > 0 || !pool_k || !pool_v || pool_slots < 1)))
+    return fail("sink_attention_rows: block means need a window, their storage, and no kept first tokens or runs");
+  if (((uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)pool_k | (uintptr_t)pool_v) & 15)
+    return fail("sink_attention_rows: the cache must start on 16 bytes");
+  const int g_chunks = (nq / nkv + 15) / 16;
+  const long long blocks = (long long)T * nkv * g_chunks * n_splits;
+  if (blocks > 0x7fffffffLL) return fail("sink_attention_rows: too many work items");
+  const size_t stages = 2 * (size_t)MK * ((hd + 8) + (vd + 8)) * 2, merge = (size_t)4 * 16 * (vd + 4) * sizeof(float);
+  const size_t smem = stages > merge ? stages : merge;
+  static bool sized = false;
+  if (!sized) {
+    cudaFuncSetAttribute(sink_attention_rows_kernel<4, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024);
+    cudaFuncSetAttribute(sink_attention_rows_kernel<8, 16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024);
+    sized = true;
+  }
+  typedef const __nv_bfloat16* B;
+  auto* kernel = hd <= 64 && vd <= 64 ? sink_attention_rows_kernel<4, 8> : sink_attention_rows_kernel<8, 16>;
+  launch_pdl(kernel, dim3((unsigned)blocks), dim3(128), smem, stream, (B)q, (B)k_cache, (B)v_cache, block_table, max_pages, page_size,
+             pos, slot, (__nv_bfloat16*)out, scratch, nq, nkv, hd, vd, window, keep_first, run, sinks, scale, split_keys, n_splits,
+             g_chunks, row_list, (B)pool_k, (B)pool_v, pool, pool_slots);
+  int rc = check_launch("sink_attention_rows");
+  if (rc || n_splits == 1) return rc;
+  launch_pdl(sink_combine_kernel<__nv_bfloat16>, dim3((unsigned)((long long)T * nq)), dim3(vd >= 128 ? 128 : 64), 0, stream,
+             (const float*)scratch, (__nv_bfloat16*)out, vd, n_splits, nq, sinks, row_list, 0);
+  return check_launch("sink_combine");
 }
 
 extern "C" const char* flint_attention_sink_last_error() { return g_error; }

@@ -926,8 +926,14 @@ class CudaOps:
                   c_int(T), c_int(nq), c_int(nkv), c_int(hd), c_int(vd), _ptr(v_keep), _ptr(v_from), c_float(blend),
                   _ptr(status))
 
-    def sink_attention_plan(self, T, nq, nkv, span):
-        """(keys per split, splits): enough warps to fill the device, at least 64 keys each."""
+    def sink_attention_plan(self, T, nq, nkv, span, tensor_cores=False):
+        """(keys per split, splits): enough warps to fill the device, at least 64 keys each; on the tensor cores a block a
+        split and up to 16 query heads, three blocks a multiprocessor."""
+        if tensor_cores:
+            base = T * nkv * -(-(nq // nkv) // 16)
+            n = max(1, min(-(-max(span, 1) // 64), 3 * self.sm_count // base))
+            keys = -(-(-(-max(span, 1) // n)) // 64) * 64
+            return keys, -(-max(span, 1) // keys)
         base = T * nkv * -(-(nq // nkv) // 4)
         span = max(span, 1)
         n = max(1, min(-(-span // 64), -(-8 * self.sm_count // base)))
@@ -935,7 +941,7 @@ class CudaOps:
         return keys, -(-span // keys)
 
     def sink_attention(self, q, cache, step, out, nq, nkv, hd, vd, window, keep_first, sinks, scale, splits=None,
-                       tiling=None, rows=None, chunk=0, pool=0, sigmoid=None):
+                       tiling=None, rows=None, chunk=0, pool=0, sigmoid=None, kernel=None):
         """Every row over its request's cached keys [.., hd] and values [.., vd]: row at position p sees key j if
         j <= p and (p - j < window or j < keep_first) (window 0: all); ``sinks`` [nq] float32 (or None): a logit
         per query head that joins the softmax's denominator.  q [T, nq hd] -> out [T, nq vd].  ``tiling``: the step's
@@ -946,7 +952,8 @@ class CudaOps:
         one mean key and value per block of P positions that lies wholly before it, from ``cache.pool_k`` /
         ``cache.pool_v`` (written by ``pool_write``), in the same softmax.  ``sigmoid`` = (cap, r1, r2, bias) instead
         of a softmax: key j weighs sigmoid(cap tanh(score / cap) - r1_h ln(1 + r2_h (p - j)) + bias_h), not normalised
-        (cap 0: no cap; r1, r2, bias float32 [nq] or None)."""
+        (cap 0: no cap; r1, r2, bias float32 [nq] or None).  ``kernel``: the rows in no tile on the tensor cores ("mma":
+        bfloat16, head sizes as for the tiles, a softmax; the default where it can) or the float32 pipes ("simt")."""
         _check(q, "q", dims=2)
         _check(out, "out", q.dtype, 2)
         cap, r1, r2, w_bias = sigmoid if sigmoid is not None else (0.0, None, None, None)
@@ -989,11 +996,22 @@ class CudaOps:
             span = min(step.max_kv_len, window + step.max_kv_len // pool)
         if chunk:
             span = min(span, chunk)
-        keys, n = splits if splits is not None else self.sink_attention_plan(T, nq, nkv, span)
+        mma_ok = sigmoid is None and self.sink_attention_tiles_ok(q.dtype, cache.k.dtype, hd, vd)
+        if kernel == "mma" and not mma_ok:
+            raise KernelError("sink_attention: the tensor-core rows take bfloat16, head sizes in multiples of 16 up to 128, a softmax")
+        mma = mma_ok and kernel != "simt"
+        keys, n = splits if splits is not None else self.sink_attention_plan(T, nq, nkv, span, mma)
         if keys * n < span:
             raise KernelError(f"sink_attention: {n} splits of {keys} keys do not cover {span} keys")
         scratch = torch.empty(T * nq * n * (vd + 2), dtype=torch.float32, device=q.device) if n > 1 else None
         self._label = kind
+        if mma:
+            return self._run("attention_sink", "flint_sink_attention_rows", _ptr(q), _ptr(cache.k), _ptr(cache.v),
+                             _ptr(cache.block_table), c_int(cache.block_table.shape[1]), c_int(P), _ptr(step.pos), _ptr(step.slot),
+                             _ptr(out), c_int(T), c_int(nq), c_int(nkv), c_int(hd), c_int(vd), c_int(window), c_int(keep_first),
+                             c_int(chunk), _ptr(sinks), c_float(scale), c_int(keys), c_int(n), _ptr(scratch), _ptr(rows),
+                             _ptr(cache.pool_k if pool else None), _ptr(cache.pool_v if pool else None), c_int(pool),
+                             c_int(cache.pool_slots if pool else 0))
         self._run("attention_sink", "flint_sink_attention", _ptr(q), c_int(_code(q.dtype)), _ptr(cache.k), _ptr(cache.v),
                   c_int(_code(cache.k.dtype)), _ptr(cache.block_table), c_int(cache.block_table.shape[1]), c_int(P),
                   _ptr(step.pos), _ptr(step.slot), _ptr(out), c_int(T), c_int(nq), c_int(nkv), c_int(hd), c_int(vd),
@@ -1120,6 +1138,28 @@ class CudaOps:
         self._run("recurrent", "flint_delta_prepare", _ptr(y), c_longlong(y.stride(0)), _ptr(b), c_longlong(b.stride(0)),
                   _ptr(a), c_longlong(a.stride(0)), _ptr(dt_bias), _ptr(a_log), _ptr(qk), _ptr(decay), _ptr(beta), c_int(T),
                   c_int(H), c_int(G), c_int(D), c_int(A), c_float(unit_eps))
+
+    def delta_token(self, proj, conv_w, dt_bias, a_log, norm_w, gate_act, pos, slot, state, unit_eps, eps, out, H, G, D, V):
+        """The gated delta rule with one decay a head and a full gate for a batch of single tokens (row e is request e), from
+        its projection to the normed and gated heads: proj [S, T, N] float32 partial sums, columns q | k | v | b | a | gate;
+        conv_w [2 G D + H V, taps]; state's rows [S (H D V) | taps rows of the convolution's inputs (the input at p in row p
+        mod taps; none for one tap)] are brought up to date; out [T, H V].  The kernel reads the state before the kernel
+        before it in the stream has ended: that must not be one that writes it."""
+        _check(proj, "proj", torch.float32, 3)
+        _check(conv_w, "conv_w", torch.float32, 2)
+        _check(state, "state", torch.float32, 2, contiguous=False)
+        _check(out, "out", dims=2)
+        S, T, N = proj.shape
+        C, taps = conv_w.shape
+        if N != 2 * G * D + 2 * H * V + 2 * H or C != 2 * G * D + H * V or tuple(out.shape) != (T, H * V) or state.stride(1) != 1 \
+                or state.shape[1] < H * D * V + (taps * C if taps > 1 else 0) or norm_w.numel() != V or gate_act not in ("sigmoid", "silu") \
+                or pos.numel() != T or slot.numel() != T or any(t.dtype != torch.float32 or t.numel() != H for t in (dt_bias, a_log)):
+            raise KernelError("delta_token: shapes do not match")
+        self._label = f"H{H} D{D} V{V}"
+        self._run("delta_token", "flint_delta_token", _ptr(proj), c_int(S), c_longlong(proj.stride(0)), c_int(N), _ptr(conv_w),
+                  c_int(taps), _ptr(dt_bias), _ptr(a_log), _ptr(norm_w), _ptr(pos), _ptr(slot), _ptr(state),
+                  c_longlong(state.stride(0)), c_float(unit_eps), c_float(eps), c_int(1 if gate_act == "silu" else 0), _ptr(out),
+                  c_int(_code(out.dtype)), c_int(T), c_int(H), c_int(G), c_int(D), c_int(V))
 
     def ssd_prepare(self, raw, dt_bias, a_log, dt, decay):
         """dt = softplus(raw + dt_bias), decay = exp(-exp(a_log) dt): raw a [T, H] float32 view, dt and decay [T, H]."""
@@ -1258,18 +1298,23 @@ class CudaOps:
         self._run("recurrent", "flint_cast_rows", _ptr(x), _ptr(out), c_int(_code(out.dtype)), c_longlong(x.numel()))
 
     def qk_norm_write(self, y, q_norm, k_norm, eps, pos, slot, cos, sin, rot, style, v_cos, v_sin, v_style, q_out, cache,
-                      nq, nkv, hd, vd, status, whole=False, v_from_k=False, q_temp=None):
-        """y [T, (nq + nkv) hd + nkv vd] float32 (q | k | v): every q and k head is divided by its root mean square
+                      nq, nkv, hd, vd, status, whole=False, v_from_k=False, q_temp=None, bias=None):
+        """y [T, (nq + nkv) hd + nkv vd] float32 (q | k | v), or [S, T, ...] partial sums that are added here, with ``bias``
+        (float32, one a column of q | k | v, or None): every q and k head is divided by its root mean square
         and scaled by q_norm / k_norm [hd] (both None: no norm), its leading ``rot`` dims rotate by the row's
         position; every value head rotates over all vd dims with tables of its own (None: not at all).  q goes to
         q_out [T, nq hd], keys and values into the row's cache page.  ``whole``: q is divided by one root mean square
         over all its heads and scaled by q_norm [nq hd], k likewise with k_norm [nkv hd].  ``v_from_k``: the values are
         the keys as projected, before norm and rotation (vd = hd; y has no value columns).  ``q_temp`` = (coef, every):
         q at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1)."""
-        _check(y, "y", torch.float32, 2, contiguous=False)
-        T = y.shape[0]
-        if y.stride(1) != 1 or y.shape[1] < (nq + nkv) * hd + (0 if v_from_k else nkv * vd):
+        if y.dim() == 2:
+            y = y.unsqueeze(0)
+        _check(y, "y", torch.float32, 3, contiguous=False)
+        T, W = y.shape[1], (nq + nkv) * hd + (0 if v_from_k else nkv * vd)
+        if y.stride(2) != 1 or y.shape[2] < W:
             raise KernelError("qk_norm_write: the rows' width does not match the head counts")
+        if bias is not None and (bias.dtype != torch.float32 or bias.numel() != W):
+            raise KernelError("qk_norm_write: bias must be float32 of the projection's width")
         if v_from_k and vd != hd:
             raise KernelError("qk_norm_write: values that are the keys need vd = hd")
         qt_coef, qt_every = (float(q_temp[0]), int(q_temp[1])) if q_temp is not None else (0.0, 1)
@@ -1287,7 +1332,8 @@ class CudaOps:
         if tuple(k.shape[1:]) != (nkv, P, hd) or tuple(v.shape[1:]) != (nkv, P, vd) or v.dtype != k.dtype:
             raise KernelError(f"qk_norm_write: cache pages are {tuple(k.shape[1:])} and {tuple(v.shape[1:])}, expected "
                               f"{(nkv, P, hd)} and {(nkv, P, vd)}")
-        self._run("recurrent", "flint_qk_norm_write", _ptr(y), c_longlong(y.stride(0)), _ptr(q_norm), _ptr(k_norm), c_float(eps),
+        self._run("recurrent", "flint_qk_norm_write", _ptr(y), c_longlong(y.stride(1)), c_int(y.shape[0]),
+                  c_longlong(y.stride(0)), _ptr(bias), _ptr(q_norm), _ptr(k_norm), c_float(eps),
                   _ptr(pos), _ptr(slot), _ptr(cos), _ptr(sin), c_int(rot), c_int(1 if style == "interleaved" else 0),
                   _ptr(v_cos), _ptr(v_sin), c_int(1 if v_style == "interleaved" else 0), _ptr(q_out),
                   c_int(_code(q_out.dtype)), _ptr(k), _ptr(v), c_int(_code(k.dtype)), _ptr(bt), c_int(bt.shape[1]), c_int(P),
@@ -1297,20 +1343,23 @@ class CudaOps:
     def head_finish(self, attn, pos, v_cos, v_sin, v_style, gate, out, nq, vd):
         """attn [T, nq vd]: every head's sum is turned back by the row's position (tables None: not at all) and
         multiplied by sigmoid(gate[t, head]) (gate a [T, nq] float32 view, or None), or, with a gate [T, nq vd], number
-        by number by sigmoid(gate[t, head, d])."""
+        by number by sigmoid(gate[t, head, d]).  A gate [S, T, ...] is partial sums that are added here."""
         _check(attn, "attn", dims=2)
         _check(out, "out", attn.dtype, 2)
         T = attn.shape[0]
         if tuple(attn.shape) != (T, nq * vd) or out.shape != attn.shape:
             raise KernelError("head_finish: shapes do not match")
         if gate is not None:
-            _check(gate, "gate", torch.float32, 2, contiguous=False)
-            if tuple(gate.shape) not in ((T, nq), (T, nq * vd)) or gate.stride(1) != 1:
+            if gate.dim() == 2:
+                gate = gate.unsqueeze(0)
+            _check(gate, "gate", torch.float32, 3, contiguous=False)
+            if tuple(gate.shape[1:]) not in ((T, nq), (T, nq * vd)) or gate.stride(2) != 1:
                 raise KernelError("head_finish: the gates must be [rows, heads] or [rows, heads x value dims]")
         self._run("recurrent", "flint_head_finish", _ptr(attn), c_int(_code(attn.dtype)), _ptr(pos), _ptr(v_cos), _ptr(v_sin),
                   c_int(1 if v_style == "interleaved" else 0), _ptr(gate),
+                  c_longlong(gate.stride(1) if gate is not None else 0), c_int(gate.shape[0] if gate is not None else 0),
                   c_longlong(gate.stride(0) if gate is not None else 0),
-                  c_int(1 if gate is not None and gate.shape[1] == nq * vd and vd > 1 else 0), _ptr(out), c_int(T), c_int(nq),
+                  c_int(1 if gate is not None and gate.shape[2] == nq * vd and vd > 1 else 0), _ptr(out), c_int(T), c_int(nq),
                   c_int(vd))
 
     def sum_norm_add(self, dst, branches=(), scales=(), expert_rows=None, gamma=None, eps=0.0, accumulate=True):

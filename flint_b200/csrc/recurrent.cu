@@ -644,9 +644,11 @@ __global__ void cast_rows_kernel(const float* __restrict__ x, TC* __restrict__ o
 // y [T, (nq + nkv) hd + nkv vd] float32: q | k | v.  Every q and k head is divided by its root mean square (eps) and
 // scaled by qw / kw [hd] (null: no norm), then its leading `rot` dims rotate by the row's position; every v head's
 // vd dims rotate by the row's position with tables of their own (null: as they are).  q goes to q_out, k and v into
-// the row's cache page.  One block per row, a warp per head.
+// the row's cache page.  y is the sum of n_partials partial sums (stride y_partial) and y_bias (or null).  A warp per head; a
+// few rows (decoded tokens) are shared by several blocks each.
 template <typename TQ, typename TC>
-__global__ void qk_norm_write_kernel(const float* __restrict__ y, long long y_stride, const float* __restrict__ qw,
+__global__ void qk_norm_write_kernel(const float* __restrict__ y, long long y_stride, int n_partials, long long y_partial,
+                                     const float* __restrict__ y_bias, const float* __restrict__ qw,
                                      const float* __restrict__ kw, float eps, const int* __restrict__ pos,
                                      const int* __restrict__ slot, const float* __restrict__ cos_t,
                                      const float* __restrict__ sin_t, int rot, int interleaved,
@@ -663,13 +665,30 @@ __global__ void qk_norm_write_kernel(const float* __restrict__ y, long long y_st
   const int page = lp < max_pages ? block_table[(size_t)slot[t] * max_pages + lp] : -1;
   if (page < 0 && threadIdx.x == 0) atomicExch(status, 1);
   const float* row = y + (size_t)t * y_stride;
+  auto at = [&](int c) {                 // column c of the row
+    float x = row[c];
+    for (int z0 = 1; z0 < n_partials; z0 += 4) {          // four loads in flight, added in a fixed order
+      float v[4];
+#pragma unroll
+      for (int u = 0; u < 4; ++u) v[u] = z0 + u < n_partials ? row[(size_t)(z0 + u) * y_partial + c] : 0.f;
+#pragma unroll
+      for (int u = 0; u < 4; ++u) x += v[u];
+    }
+    return y_bias ? x + y_bias[c] : x;
+  };
   // a temperature on the queries that grows with the position: 1 + coef ln(floor((p + 1) / every) + 1)
   const float q_temp = qt_coef != 0.f ? 1.0f + qt_coef * logf(floorf((float)(p + 1) / (float)qt_every) + 1.0f) : 1.0f;
   float inv_whole[2] = {1.f, 1.f};
   if (whole && qw) {          // one root mean square over all query heads, one over all key heads
     float sq = 0.f, sk = 0.f;
-    for (int e = threadIdx.x; e < nq * hd; e += blockDim.x) sq = fmaf(row[e], row[e], sq);
-    for (int e = threadIdx.x; e < nkv * hd; e += blockDim.x) sk = fmaf(row[(size_t)nq * hd + e], row[(size_t)nq * hd + e], sk);
+    for (int e = threadIdx.x; e < nq * hd; e += blockDim.x) {
+      const float x = at(e);
+      sq = fmaf(x, x, sq);
+    }
+    for (int e = threadIdx.x; e < nkv * hd; e += blockDim.x) {
+      const float x = at(nq * hd + e);
+      sk = fmaf(x, x, sk);
+    }
     sq = warp_sum(sq);
     sk = warp_sum(sk);
     if (lane == 0) { part[0][warp] = sq; part[1][warp] = sk; }
@@ -679,13 +698,11 @@ __global__ void qk_norm_write_kernel(const float* __restrict__ y, long long y_st
     inv_whole[0] = 1.0f / sqrtf(sq / (float)(nq * hd) + eps);
     inv_whole[1] = 1.0f / sqrtf(sk / (float)(nkv * hd) + eps);
   }
-  for (int head = warp; head < nq + 2 * nkv; head += nw) {
+  for (int head = blockIdx.y * nw + warp; head < nq + 2 * nkv; head += nw * gridDim.y) {
     const bool is_v = head >= nq + nkv;
     const int n = is_v ? vd : hd;
     // values that are the keys as projected come from the key's columns (vd = hd), before norm and rotation
-    const float* src = is_v ? (v_from_k ? row + (size_t)(head - nkv) * hd
-                                        : row + (size_t)(nq + nkv) * hd + (size_t)(head - nq - nkv) * vd)
-                            : row + (size_t)head * hd;
+    const int src = is_v ? (v_from_k ? (head - nkv) * hd : (nq + nkv) * hd + (head - nq - nkv) * vd) : head * hd;
     const float* w = is_v ? nullptr : (head < nq ? qw : kw);
     float inv = 1.f;
     if (w && whole) {
@@ -693,7 +710,10 @@ __global__ void qk_norm_write_kernel(const float* __restrict__ y, long long y_st
       w += (size_t)(head < nq ? head : head - nq) * hd;       // a scale per column of the projection
     } else if (w) {
       float ss = 0.f;
-      for (int d = lane; d < n; d += 32) ss = fmaf(src[d], src[d], ss);
+      for (int d = lane; d < n; d += 32) {
+        const float x = at(src + d);
+        ss = fmaf(x, x, ss);
+      }
       inv = 1.0f / sqrtf(warp_sum(ss) / (float)n + eps);
     }
     if (head < nq) inv *= q_temp;
@@ -701,13 +721,13 @@ __global__ void qk_norm_write_kernel(const float* __restrict__ y, long long y_st
     const float* st = is_v ? vsin : sin_t;
     const int r = is_v ? (vcos ? vd : 0) : rot, half = r / 2, il = is_v ? v_interleaved : interleaved;
     for (int d = lane; d < n; d += 32) {
-      float x = src[d] * inv * (w ? w[d] : 1.f);
+      float x = at(src + d) * inv * (w ? w[d] : 1.f);
       if (d < r) {
         int i, partner;
         bool first;
         if (il) { i = d >> 1; first = !(d & 1); partner = first ? d + 1 : d - 1; }
         else { i = d < half ? d : d - half; first = d < half; partner = first ? d + half : d - half; }
-        const float z = src[partner] * inv * (w ? w[partner] : 1.f);
+        const float z = at(src + partner) * inv * (w ? w[partner] : 1.f);
         const float c = ct[(size_t)p * half + i], s = st[(size_t)p * half + i];
         x = first ? x * c - z * s : x * c + z * s;
       }
@@ -722,11 +742,13 @@ __global__ void qk_norm_write_kernel(const float* __restrict__ y, long long y_st
 }
 
 // attn [T, nq vd]: every head's sum is rotated back by the row's position (tables null: not at all) and multiplied by
-// sigmoid(gate[t, head]) (gate null: by 1).  One thread per pair of dims.
+// sigmoid(gate[t, head]) (gate null: by 1; the gates' logits are the sum of gate_partials partial sums).  One thread per
+// pair of dims.
 template <typename TA>
 __global__ void head_finish_kernel(const TA* __restrict__ attn, const int* __restrict__ pos, const float* __restrict__ vcos,
                                    const float* __restrict__ vsin, int interleaved, const float* __restrict__ gate,
-                                   long long gate_stride, int gate_each, TA* __restrict__ out, int T, int nq, int vd) {
+                                   long long gate_stride, int gate_partials, long long gate_partial, int gate_each,
+                                   TA* __restrict__ out, int T, int nq, int vd) {
   pdl_launch();
   pdl_wait();
   const int half = (vd + 1) / 2;          // an odd size (never with a rotation) leaves one dim without a partner
@@ -745,8 +767,13 @@ __global__ void head_finish_kernel(const TA* __restrict__ attn, const int* __res
   }
   // a gate per head, or one per number of every head
   const float* gr = gate + (size_t)t * gate_stride;
-  const float ga = !gate ? 1.f : sigmoidf_(gate_each ? gr[(size_t)head * vd + a] : gr[head]);
-  const float gb = !gate ? 1.f : (gate_each ? sigmoidf_(gr[(size_t)head * vd + (pair ? b : a)]) : ga);
+  auto gate_of = [&](int c) {
+    float x = 0.f;
+    for (int z = 0; z < gate_partials; ++z) x += gr[(size_t)z * gate_partial + c];
+    return sigmoidf_(x);
+  };
+  const float ga = !gate ? 1.f : gate_of(gate_each ? head * vd + a : head);
+  const float gb = !gate ? 1.f : (gate_each ? gate_of(head * vd + (pair ? b : a)) : ga);
   out[base + a] = from_f32<TA>(u * ga);
   if (pair) out[base + b] = from_f32<TA>(v * gb);
 }
@@ -969,33 +996,37 @@ extern "C" int flint_cast_rows(const float* x, void* out, int out_dtype, long lo
   return check_launch("cast_rows");
 }
 
-extern "C" int flint_qk_norm_write(const float* y, long long y_stride, const float* qw, const float* kw, float eps,
+extern "C" int flint_qk_norm_write(const float* y, long long y_stride, int n_partials, long long y_partial,
+                                   const float* y_bias, const float* qw, const float* kw, float eps,
                                    const int* pos, const int* slot, const float* cos_t, const float* sin_t, int rot,
                                    int interleaved, const float* vcos, const float* vsin, int v_interleaved, void* q_out,
                                    int q_dtype, void* k_cache, void* v_cache, int cache_dtype, const int* block_table,
                                    int max_pages, int page_size, int T, int nq, int nkv, int hd, int vd, int whole, int v_from_k,
                                    float qt_coef, int qt_every, int* status, cudaStream_t stream) {
   if (T <= 0) return 0;
+  if (n_partials < 1) return fail("qk_norm_write: needs at least one partial sum");
+  // few rows: sixteen warps a block, and as many blocks as the heads fill
+  const unsigned threads = T <= 64 ? 512u : 256u, shares = T <= 64 ? (unsigned)((nq + 2 * nkv + 15) / 16) : 1u;
   if (rot < 0 || rot > hd || rot % 2 || (vcos && vd % 2)) return fail("qk_norm_write: bad rotation sizes");
   if (v_from_k && vd != hd) return fail("qk_norm_write: values that are the keys need vd = hd");
   if (qt_coef != 0.f && qt_every < 1) return fail("qk_norm_write: the query temperature's period must be positive");
   if ((qw == nullptr) != (kw == nullptr)) return fail("qk_norm_write: q and k are normed together or not at all");
   FLINT_DISPATCH_DTYPE(q_dtype, TQ, FLINT_DISPATCH_DTYPE(cache_dtype, TC,
-      launch_pdl(qk_norm_write_kernel<TQ, TC>, dim3((unsigned)T), dim3(256), 0, stream, y, y_stride, qw, kw, eps, pos, slot,
-                 cos_t, sin_t, rot, interleaved, vcos, vsin, v_interleaved, (TQ*)q_out, (TC*)k_cache, (TC*)v_cache,
+      launch_pdl(qk_norm_write_kernel<TQ, TC>, dim3((unsigned)T, shares), dim3(threads), 0, stream, y, y_stride, n_partials,
+                 y_partial, y_bias, qw, kw, eps, pos, slot, cos_t, sin_t, rot, interleaved, vcos, vsin, v_interleaved, (TQ*)q_out, (TC*)k_cache, (TC*)v_cache,
                  block_table, max_pages, page_size, nq, nkv, hd, vd, whole, v_from_k, qt_coef, qt_every, status)));
   return check_launch("qk_norm_write");
 }
 
 extern "C" int flint_head_finish(const void* attn, int dtype, const int* pos, const float* vcos, const float* vsin,
-                                 int interleaved, const float* gate, long long gate_stride, int gate_each, void* out, int T,
-                                 int nq, int vd, cudaStream_t stream) {
+                                 int interleaved, const float* gate, long long gate_stride, int gate_partials,
+                                 long long gate_partial, int gate_each, void* out, int T, int nq, int vd, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (vd % 2 && vcos) return fail("head_finish: value heads of %d dims cannot rotate in pairs", vd);
   const long long n = (long long)T * nq * ((vd + 1) / 2);
   FLINT_DISPATCH_DTYPE(dtype, TA,
       launch_pdl(head_finish_kernel<TA>, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream, (const TA*)attn, pos, vcos,
-                 vsin, interleaved, gate, gate_stride, gate_each, (TA*)out, T, nq, vd));
+                 vsin, interleaved, gate, gate_stride, gate_partials, gate_partial, gate_each, (TA*)out, T, nq, vd));
   return check_launch("head_finish");
 }
 

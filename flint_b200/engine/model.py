@@ -254,8 +254,11 @@ class Model:
     def _parts_with_tensors(self):
         for part, _ in self.embed_additions:
             yield part
-        for layer in self.layers:
-            yield from layer.parts.values()
+        parts = [p for layer in self.layers for p in layer.parts.values()]
+        while parts:
+            part = parts.pop()
+            yield part
+            parts += part.subparts()
 
     def weight_bytes(self):
         seen, total = set(), 0

@@ -269,18 +269,22 @@ class Attention(Mixer):
         T, dev = xin.shape[0], xin.device
         act = self.ctx.act_dtype if self.w_qkv.dtype == torch.bfloat16 else torch.float32
         W = (nq + nkv) * hd + (0 if self.values_from_keys else nkv * vd)
-        proj = torch.empty((T, self.w_qkv.shape[0]), dtype=torch.float32, device=dev)
-        ops.gemm(xin, self.w_qkv, proj, bias=self.b_qkv_all)
+        bias = None
         if self.taps:
             if self.taps > 1 and state is None:
                 raise ModelError("attention: the convolution needs a state slab")
+            proj = torch.empty((1, T, self.w_qkv.shape[0]), dtype=torch.float32, device=dev)
+            ops.gemm(xin, self.w_qkv, proj[0], bias=self.b_qkv_all)
             y = torch.empty((T, W), dtype=torch.float32, device=dev)
-            ops.short_conv(proj, 0, self.w_conv, None, "none", step.pos, step.slot, state, y)
-        else:
-            y = proj[:, :W]
+            ops.short_conv(proj[0], 0, self.w_conv, None, "none", step.pos, step.slot, state, y)
+        else:                 # left as partial sums, which the next kernels add up with the bias
+            proj = ops.gemm_partials(xin, self.w_qkv)
+            y, bias = proj[:, :, :W], self.b_qkv
         q = torch.empty((T, nq * hd), dtype=act, device=dev)
         extra = {k: v for k, v in (("whole", self.qk_whole), ("v_from_k", self.values_from_keys), ("q_temp", self.q_temp))
                  if v}
+        if bias is not None:
+            extra["bias"] = bias
         ops.qk_norm_write(y, self.q_norm, self.k_norm, self.qk_eps, step.pos, step.slot, self.cos, self.sin, self.rot,
                           self.rot_style, self.v_cos, self.v_sin,
                           self.value_position.style if self.value_position is not None else "half", q, cache, nq, nkv, hd,
@@ -297,7 +301,7 @@ class Attention(Mixer):
             out = torch.empty_like(attn)
             ops.head_finish(attn, step.pos, self.v_cos, self.v_sin,
                             self.value_position.style if self.value_position is not None else "half",
-                            proj[:, W:] if self.head_gate or self.out_gate else None, out, nq, vd)
+                            proj[:, :, W:] if self.head_gate or self.out_gate else None, out, nq, vd)
             attn = out
         return Pending(partials=ops.gemm_partials(attn, self.w_o), bias=self.b_o)
 

@@ -139,6 +139,10 @@ class Part:
         stands for, stacked by rows in that order (all under this part's prefix)."""
         return {}
 
+    def subparts(self) -> list:
+        """The parts this one is made of (their tensors are its own)."""
+        return []
+
     def load(self, tensors: dict):
         """Receives the tensors named by ``weights()`` (already on the device and typed
         by the loader's policy)."""

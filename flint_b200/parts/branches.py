@@ -58,6 +58,9 @@ class Branches(Mixer):
                 w[f"{name}.out"] = vec(self.hidden, init="gamma")
         return w
 
+    def subparts(self):
+        return [m for _, m in self.branches]
+
     def fused(self):
         return {f"{name}.{k}": [f"{name}.{p}" for p in pieces] for name, m in self.branches for k, pieces in m.fused().items()}
 

@@ -43,6 +43,9 @@ class InputConv(Mixer):
     def weights(self):
         return {self.CONV: conv_weight(self.hidden, self.taps), **self.inner.weights()}
 
+    def subparts(self):
+        return [self.inner]
+
     def fused(self):
         return self.inner.fused()
 

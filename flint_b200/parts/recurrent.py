@@ -92,6 +92,10 @@ class GatedDeltaRule(_Recurrent):
         self.head_decay, self.full_gate = bool(p.get("head_decay", False)), bool(p.get("full_gate", False))
         self.gate_act = p.get("gate_act", "sigmoid")
         self.conv_ch = 2 * self.G * self.D + self.H * self.V
+        # single tokens of the form without low-rank pairs take one launch, in which several blocks read an input that one of
+        # them stores: the convolution's inputs then have one row more than are ever read (position p in row p mod taps)
+        self.one_launch = self.head_decay and self.full_gate
+        self.ring = self.taps if self.one_launch and self.taps > 1 else self.taps - 1
 
     def weights(self):
         H, G, D, V, W, t = self.H, self.G, self.D, self.V, self.hidden, self.taps
@@ -132,19 +136,25 @@ class GatedDeltaRule(_Recurrent):
         return (self.w_in.dtype,)
 
     def state_spec(self):
-        return StateSpec((self.H * self.D * self.V + (self.taps - 1) * self.conv_ch,), torch.float32)
+        return StateSpec((self.H * self.D * self.V + self.ring * self.conv_ch,), torch.float32)
 
     def forward(self, x, residual, step, cache, state, writes_cache=True):
         ops, H, G, D, V = self.ops, self.H, self.G, self.D, self.V
         S, conv_state = self._split_state(state, H * D * V)
         xin = x[self.w_in.dtype]
         T, dev = xin.shape[0], xin.device
+        act = self.ctx.act_dtype if self.w_o.dtype == torch.bfloat16 else torch.float32
+        out = torch.empty((T, H * V), dtype=act, device=dev)
+        if self.one_launch and T == len(step.entries):          # single tokens: one launch from the projection to the gated heads
+            ops.delta_token(ops.gemm_partials(xin, self.w_in), self.w_conv, self.dt_bias, self.a_log, self.w_norm, self.gate_act,
+                            step.pos, step.slot, state, self.unit_eps, self.eps, out, H, G, D, V)
+            return Pending(partials=ops.gemm_partials(out, self.w_o))
         f32 = dict(dtype=torch.float32, device=dev)
         proj = torch.empty((T, self.w_in.shape[0]), **f32)
         ops.gemm(xin, self.w_in, proj)
         C = self.conv_ch
         y = torch.empty((T, C), **f32)
-        ops.short_conv(proj, 0, self.w_conv, None, "silu", step.pos, step.slot, conv_state, y)
+        ops.short_conv(proj, 0, self.w_conv, None, "silu", step.pos, step.slot, conv_state, y, ring_rows=self.ring or None)
         c_b, c_a, c_g = C, C + H, C + H + self.n_a
         a, gate = proj[:, c_a:c_g], proj[:, c_g:c_g + self.n_g]
         if not self.head_decay:       # the low-rank second halves read float32 columns of the projection
@@ -160,8 +170,6 @@ class GatedDeltaRule(_Recurrent):
         o = torch.empty((T, H * V), **f32)
         ops.recurrence_scan(qk[:, :G * D], qk[:, G * D:], y[:, 2 * G * D:], decay, True, beta, None, None, step.slot,
                             request_starts(step), len(step.entries), S, o, H, G, D, V)
-        act = self.ctx.act_dtype if self.w_o.dtype == torch.bfloat16 else torch.float32
-        out = torch.empty((T, H * V), dtype=act, device=dev)
         ops.gated_norm(o, gate, self.gate_act, False, self.w_norm, self.eps, H, out)
         return Pending(partials=ops.gemm_partials(out, self.w_o))
 

@@ -296,7 +296,7 @@ class RefOps:
         cache.v[pages, :, p % P, :] = v.to(cache.v.dtype)
 
     def sink_attention(self, q, cache, step, out, nq, nkv, hd, vd, window, keep_first, sinks, scale, splits=None,
-                       tiling=None, rows=None, chunk=0, pool=0, sigmoid=None):
+                       tiling=None, rows=None, chunk=0, pool=0, sigmoid=None, kernel=None):
         T, P, G = q.shape[0], cache.page_size, nq // nkv
         qq = q.to(self.cd).view(T, nq, hd)
         res = torch.zeros(T, nq, vd, dtype=self.cd)
@@ -422,6 +422,17 @@ class RefOps:
         sp = torch.nn.functional.softplus(a.to(self.cd) + dt_bias.to(self.cd), threshold=30.0).view(T, H, -1)
         decay.copy_(torch.exp(-torch.exp(a_log.to(self.cd)).view(1, H, 1) * sp).reshape(decay.shape).to(decay.dtype))
 
+    def delta_token(self, proj, conv_w, dt_bias, a_log, norm_w, gate_act, pos, slot, state, unit_eps, eps, out, H, G, D, V):
+        x = proj.to(self.cd).sum(0)
+        T, C, taps = x.shape[0], conv_w.shape[0], conv_w.shape[1]
+        y, qk = torch.zeros(T, C, dtype=self.cd), torch.zeros(T, 2 * G * D, dtype=self.cd)
+        decay, beta, o = torch.zeros(T, H, dtype=self.cd), torch.zeros(T, H, dtype=self.cd), torch.zeros(T, H * V, dtype=self.cd)
+        self.short_conv(x, 0, conv_w, None, "silu", pos, slot, state[:, H * D * V:], y, ring_rows=taps if taps > 1 else None)
+        self.delta_prepare(y, x[:, C:C + H], x[:, C + H:C + 2 * H], dt_bias, a_log, qk, decay, beta, H, G, D, unit_eps)
+        self.recurrence_scan(qk[:, :G * D], qk[:, G * D:], y[:, 2 * G * D:], decay, True, beta, None, None, slot, None, T,
+                             state, o, H, G, D, V)
+        self.gated_norm(o, x[:, C + 2 * H:], gate_act, False, norm_w, eps, H, out)
+
     def ssd_prepare(self, raw, dt_bias, a_log, dt, decay):
         d = torch.nn.functional.softplus(raw.to(self.cd) + dt_bias.to(self.cd), threshold=30.0)
         dt.copy_(d.to(dt.dtype))
@@ -522,9 +533,11 @@ class RefOps:
         return torch.cat([both, h[..., rot:]], -1)
 
     def qk_norm_write(self, y, q_norm, k_norm, eps, pos, slot, cos, sin, rot, style, v_cos, v_sin, v_style, q_out, cache,
-                      nq, nkv, hd, vd, status, whole=False, v_from_k=False, q_temp=None):
-        T = y.shape[0]
-        x = y.to(self.cd)
+                      nq, nkv, hd, vd, status, whole=False, v_from_k=False, q_temp=None, bias=None):
+        x = y.to(self.cd).sum(0) if y.dim() == 3 else y.to(self.cd)
+        T = x.shape[0]
+        if bias is not None:
+            x = x[:, :bias.numel()] + bias.to(self.cd)
         p = pos.long()
         q = x[:, :nq * hd].reshape(T, nq, hd)
         k = x[:, nq * hd:(nq + nkv) * hd].reshape(T, nkv, hd)
@@ -552,6 +565,8 @@ class RefOps:
 
     def head_finish(self, attn, pos, v_cos, v_sin, v_style, gate, out, nq, vd):
         T = attn.shape[0]
+        if gate is not None and gate.dim() == 3:
+            gate = gate.to(self.cd).sum(0)
         x = attn.to(self.cd).view(T, nq, vd)
         if v_cos is not None:
             p = pos.long()

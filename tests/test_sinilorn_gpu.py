@@ -331,7 +331,7 @@ def pending_case(rn, T, W, S, which):
 
 
 def pend_on(p, device):
-    return Pending(**{k: (v.to(device) if v is not None else None) for k, v in vars(p).items()})
+    return Pending(**{k: (v.to(device) if isinstance(v, torch.Tensor) else v) for k, v in vars(p).items()})
 
 
 @pytest.mark.parametrize("S", [1, 2, 3, 4, 6])
