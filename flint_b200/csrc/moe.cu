@@ -396,8 +396,8 @@ extern "C" int flint_router_topk(const float* x, const void* wr, int w_dtype, in
 
 // Upper bound of row tiles for n_assign rows over E experts.
 // --------------------------------------------------------------------------- sigmoid router
-// Scores s_e = sigmoid(<x, Wr[e]>) in float32 over the first E rows of Wr; the `top` largest are chosen (the lower
-// index among equals) with their scores as they are.  Rows E .. E + X - 1 of Wr are not experts but gates of
+// Scores s_e = sigmoid(<x, Wr[e]>) in float32 over the first E rows of Wr; the `top` largest are chosen (by their logits; the
+// lower index among equals) with their scores as they are.  Rows E .. E + X - 1 of Wr are not experts but gates of
 // always-on parts: their sigmoids go to weights[:, top:], and weights[:, :top] is 1 (the chosen experts' scores
 // scale their inputs, so their outputs are added as they are).  A warp takes RT tokens and reads every weight
 // row once for all of them.

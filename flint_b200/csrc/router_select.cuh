@@ -100,15 +100,15 @@ __device__ __forceinline__ void select_topk_by_warp(float* s, int lane, int E, i
 }
 
 // The choice of a sigmoid router, by one warp, from float32 logits in shared memory: scores sigmoid(logit) over the
-// first E entries, the `top` largest chosen (the lower index among equals), their scores given as they are.  The
+// first E entries, the `top` largest chosen (the lower index among equals), their scores given as they are.  The logits
+// decide, which have the order of the scores: float32 scores near 1 lie too close to tell experts apart.  The
 // `extra` entries after them are gates of always-on parts: weights [top + extra] gets 1 for every chosen expert
 // and the sigmoids of those entries.  `s` holds the logits on entry and is overwritten.
 __device__ __forceinline__ void select_sigmoid_by_warp(float* s, int lane, int E, int extra, int top, int* ids,
                                                        float* scores, float* weights) {
-  for (int e = lane; e < E + extra; e += 32) s[e] = 1.0f / (1.0f + expf(-s[e]));
-  __syncwarp();
+  for (int e = lane; e < extra; e += 32) weights[top + e] = 1.0f / (1.0f + expf(-s[E + e]));
   for (int c = 0; c < top; ++c) {
-    float val = -1.f;
+    float val = -INFINITY;
     int idx = 0x7fffffff;
     for (int e = lane; e < E; e += 32)
       if (s[e] > val) { val = s[e]; idx = e; }
@@ -119,14 +119,14 @@ __device__ __forceinline__ void select_sigmoid_by_warp(float* s, int lane, int E
       if (ov > val || (ov == val && oi < idx)) { val = ov; idx = oi; }
     }
     if (lane == 0) {
+      if (idx >= E) idx = c;                  // logits that are no numbers: any expert, within bounds
       ids[c] = idx;
-      scores[c] = val;
+      scores[c] = 1.0f / (1.0f + expf(-val));
       weights[c] = 1.0f;
-      s[idx] = -2.f;                          // taken
+      s[idx] = -INFINITY;                     // taken
     }
     __syncwarp();
   }
-  for (int e = lane; e < extra; e += 32) weights[top + e] = s[E + e];
 }
 
 // The choice of a router with corrected choice scores, limited to groups, by one warp, from float32 logits in shared

@@ -642,9 +642,9 @@ class RefOps:
     def router_sigmoid(self, x, wr, E, top, expert_ids, scores, weights, logits_out=None):
         z = x.to(self.cd) @ wr.to(self.cd).T
         s = torch.sigmoid(z)
-        val, idx = torch.sort(s[:, :E], dim=-1, descending=True, stable=True)
-        expert_ids.copy_(idx[:, :top].to(torch.int32))
-        scores.copy_(val[:, :top].to(scores.dtype))
+        idx = torch.sort(z[:, :E], dim=-1, descending=True, stable=True).indices[:, :top]       # the order of the scores
+        expert_ids.copy_(idx.to(torch.int32))
+        scores.copy_(s.gather(1, idx).to(scores.dtype))
         weights[:, :top] = 1.0
         if wr.shape[0] > E:
             weights[:, top:] = s[:, E:].to(weights.dtype)

@@ -224,23 +224,24 @@ def test_rows_get_what_is_added_normed(ops, T, W):
 
 
 @pytest.mark.parametrize("T,W", [(1, 208), (8, 2048), (300, 200), (2048, 256), (9, 38), (16, 1028)])
-@pytest.mark.parametrize("E,top", [(13, 3), (70, 6), (5, 1)])
-def test_the_sigmoid_router_rides_on_the_sum(ops, T, W, E, top):
-    """The choice is exactly the rule applied to the logits the kernel reports, and those agree with the plain product."""
+@pytest.mark.parametrize("E,top,gain", [(13, 3, 2.5), (70, 6, 2.5), (5, 1, 2.5), (40, 2, 12.0)])
+def test_the_sigmoid_router_rides_on_the_sum(ops, T, W, E, top, gain):
+    """The choice is exactly the rule applied to the logits the kernel reports, also where many scores round to 1 in float32,
+    and those agree with the plain product."""
     rn = gen(T + E)
-    x, p, wr = rn(T, W), pending_case(rn, T, W, "partials norm"), (2.5 * rn(E, W) / math.sqrt(W)).to(torch.bfloat16)
+    x, p, wr = rn(T, W), pending_case(rn, T, W, "partials norm"), (gain * rn(E, W) / math.sqrt(W)).to(torch.bfloat16)
     req = RouterRequest(wr.to(DEV), 0.0, torch.zeros(T, top, dtype=torch.int32, device=DEV), torch.zeros(T, top, device=DEV),
                         logits=torch.zeros(T, E, device=DEV), top=top, rule="sigmoid", weights=torch.zeros(T, top, device=DEV))
     a, b = x.double(), x.to(DEV)
     RefOps(F64).row_post(a, p)
     ops.row_post(b, pend_on(p, DEV), router=req)
     assert (b.cpu().double() - a).abs().max() < 1e-4
-    assert (req.logits.cpu().double() - a @ wr.double().T).abs().max() < 5e-4
+    assert (req.logits.cpu().double() - a @ wr.double().T).abs().max() < 2e-4 * gain
     s = torch.sigmoid(req.logits.cpu().double())
-    ids = torch.sort(s, dim=-1, descending=True, stable=True).indices[:, :top]
+    ids = torch.sort(req.logits.cpu(), dim=-1, descending=True, stable=True).indices[:, :top]
     same = (ids == req.expert_ids.cpu().long()).all(-1)
-    assert int((~same).sum()) <= max(1, T // 200)                # float32 scores against float64 ones: a tie at most
-    assert (req.gates.cpu().double() - s.gather(1, ids))[same].abs().max() < 1e-5 and bool((req.weights == 1).all())
+    assert bool(same.all())
+    assert (req.gates.cpu().double() - s.gather(1, ids)).abs().max() < 1e-5 and bool((req.weights == 1).all())
 
 
 @pytest.mark.parametrize("W,taps", [(64, 3), (37, 4), (1024, 2), (2048, 5), (40, 1), (72, 6)])
