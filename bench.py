@@ -916,6 +916,8 @@ def run_sokipel_pair(args, pk, rng):
             for kind, table in tables:
                 decoding = kind != "prefill"
                 for kname, (n, ms) in sorted(table.items()):
+                    if kind.endswith("captured"):
+                        n = dec_t[kname][0]          # a launcher's second kernels counted with its first
                     secs = ms / n * 1e-3
                     e = {"launches": n, "us": round(secs * 1e6, 2)}
                     scan = next((s for s in state if kname.startswith(("flint_recurrence_scan " + s, "flint_delta_token"))), None)

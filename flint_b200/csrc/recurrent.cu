@@ -380,6 +380,48 @@ __global__ void gated_norm_kernel(const float* __restrict__ o, const float* __re
   }
 }
 
+// The same with parts of whole 16-byte units, every row on 16 bytes: a warp per (row, group), the part in registers (U units
+// a lane) between the sum of squares and the store.
+template <int U, typename TO>
+__global__ void __launch_bounds__(256)
+gated_norm_vec_kernel(const float* __restrict__ o, const float* __restrict__ gate, long long gate_stride, int gate_act,
+                      int gate_first, const float* __restrict__ w, int w_len, float eps, int groups, int N, TO* __restrict__ out,
+                      long long parts) {
+  pdl_launch();
+  pdl_wait();
+  const long long part = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (part >= parts) return;
+  const int lane = threadIdx.x & 31, gs = N / groups, c0 = (int)(part % groups) * gs;
+  const long long t = part / groups;
+  const float* orow = o + t * N + c0;
+  const float* grow = gate + t * gate_stride + c0;
+  auto act = [&](float z) { return gate_act ? siluf_(z) : sigmoidf_(z); };
+  float4 x[U], g[U];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < U; ++i) {
+    const int c = 4 * (lane + 32 * i);
+    x[i] = g[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c < gs) {
+      x[i] = *reinterpret_cast<const float4*>(orow + c);
+      const float4 z = *reinterpret_cast<const float4*>(grow + c);
+      g[i] = make_float4(act(z.x), act(z.y), act(z.z), act(z.w));
+      if (gate_first) { x[i].x *= g[i].x; x[i].y *= g[i].y; x[i].z *= g[i].z; x[i].w *= g[i].w; }
+    }
+    ss = fmaf(x[i].x, x[i].x, fmaf(x[i].y, x[i].y, fmaf(x[i].z, x[i].z, fmaf(x[i].w, x[i].w, ss))));
+  }
+  const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)gs + eps);
+#pragma unroll
+  for (int i = 0; i < U; ++i) {
+    const int c = 4 * (lane + 32 * i);
+    if (c >= gs) continue;
+    const float4 s = *reinterpret_cast<const float4*>(w + (c0 + c) % w_len);
+    float4 y = make_float4(x[i].x * inv * s.x, x[i].y * inv * s.y, x[i].z * inv * s.z, x[i].w * inv * s.w);
+    if (!gate_first) { y.x *= g[i].x; y.y *= g[i].y; y.z *= g[i].z; y.w *= g[i].w; }
+    store4(out + t * N + c0 + c, y);
+  }
+}
+
 // ------------------------------------------------------------------------------------------- weighted sums of branches, normed, added
 struct SumList {
   const float* partials[4];
@@ -646,7 +688,8 @@ __global__ void cast_rows_kernel(const float* __restrict__ x, TC* __restrict__ o
 // vd dims rotate by the row's position with tables of their own (null: as they are).  q goes to q_out, k and v into
 // the row's cache page.  y is the sum of n_partials partial sums (stride y_partial) and y_bias (or null).  A warp per head; a
 // few rows (decoded tokens) are shared by several blocks each.
-template <typename TQ, typename TC>
+// SUM: more than one partial sum.
+template <typename TQ, typename TC, bool SUM>
 __global__ void qk_norm_write_kernel(const float* __restrict__ y, long long y_stride, int n_partials, long long y_partial,
                                      const float* __restrict__ y_bias, const float* __restrict__ qw,
                                      const float* __restrict__ kw, float eps, const int* __restrict__ pos,
@@ -667,7 +710,7 @@ __global__ void qk_norm_write_kernel(const float* __restrict__ y, long long y_st
   const float* row = y + (size_t)t * y_stride;
   auto at = [&](int c) {                 // column c of the row
     float x = row[c];
-    for (int z0 = 1; z0 < n_partials; z0 += 4) {          // four loads in flight, added in a fixed order
+    for (int z0 = 1; SUM && z0 < n_partials; z0 += 4) {   // four loads in flight, added in a fixed order
       float v[4];
 #pragma unroll
       for (int u = 0; u < 4; ++u) v[u] = z0 + u < n_partials ? row[(size_t)(z0 + u) * y_partial + c] : 0.f;
@@ -744,7 +787,7 @@ __global__ void qk_norm_write_kernel(const float* __restrict__ y, long long y_st
 // attn [T, nq vd]: every head's sum is rotated back by the row's position (tables null: not at all) and multiplied by
 // sigmoid(gate[t, head]) (gate null: by 1; the gates' logits are the sum of gate_partials partial sums).  One thread per
 // pair of dims.
-template <typename TA>
+template <typename TA, bool SUM>
 __global__ void head_finish_kernel(const TA* __restrict__ attn, const int* __restrict__ pos, const float* __restrict__ vcos,
                                    const float* __restrict__ vsin, int interleaved, const float* __restrict__ gate,
                                    long long gate_stride, int gate_partials, long long gate_partial, int gate_each,
@@ -768,8 +811,8 @@ __global__ void head_finish_kernel(const TA* __restrict__ attn, const int* __res
   // a gate per head, or one per number of every head
   const float* gr = gate + (size_t)t * gate_stride;
   auto gate_of = [&](int c) {
-    float x = 0.f;
-    for (int z = 0; z < gate_partials; ++z) x += gr[(size_t)z * gate_partial + c];
+    float x = gr[c];
+    for (int z = 1; SUM && z < gate_partials; ++z) x += gr[(size_t)z * gate_partial + c];
     return sigmoidf_(x);
   };
   const float ga = !gate ? 1.f : gate_of(gate_each ? head * vd + a : head);
@@ -890,6 +933,18 @@ extern "C" int flint_gated_norm(const float* o, const float* gate, long long gat
   if (groups < 1 || N % groups || w_len < 1) return fail("gated_norm: %d numbers do not divide into %d parts", N, groups);
   if ((long long)T * groups > 0x7fffffffLL) return fail("gated_norm: too many rows");
   const int gs = N / groups, threads = gs >= 1024 ? 256 : gs > 64 ? 128 : gs > 32 ? 64 : 32;
+  if (gs % 4 == 0 && gs <= 512 && w_len % 4 == 0 && gate_stride % 4 == 0 &&
+      !(((uintptr_t)o | (uintptr_t)gate | (uintptr_t)w | (uintptr_t)out) & 15)) {
+    const long long parts = (long long)T * groups;
+#define GO(U) FLINT_DISPATCH_DTYPE(out_dtype, TO,                                                                             \
+      launch_pdl(gated_norm_vec_kernel<U, TO>, dim3((unsigned)((parts + 7) / 8)), dim3(256), 0, stream, o, gate, gate_stride, \
+                 gate_act, gate_first, w, w_len, eps, groups, N, (TO*)out, parts))
+    if (gs <= 128) GO(1);
+    else if (gs <= 256) GO(2);
+    else GO(4);
+#undef GO
+    return check_launch("gated_norm");
+  }
   FLINT_DISPATCH_DTYPE(out_dtype, TO,
       launch_pdl(gated_norm_kernel<TO>, dim3((unsigned)(T * groups)), dim3(threads), 0, stream, o, gate, gate_stride, gate_act,
                  gate_first, w, w_len, eps, groups, N, (TO*)out));
@@ -1012,7 +1067,7 @@ extern "C" int flint_qk_norm_write(const float* y, long long y_stride, int n_par
   if (qt_coef != 0.f && qt_every < 1) return fail("qk_norm_write: the query temperature's period must be positive");
   if ((qw == nullptr) != (kw == nullptr)) return fail("qk_norm_write: q and k are normed together or not at all");
   FLINT_DISPATCH_DTYPE(q_dtype, TQ, FLINT_DISPATCH_DTYPE(cache_dtype, TC,
-      launch_pdl(qk_norm_write_kernel<TQ, TC>, dim3((unsigned)T, shares), dim3(threads), 0, stream, y, y_stride, n_partials,
+      launch_pdl(n_partials > 1 ? qk_norm_write_kernel<TQ, TC, true> : qk_norm_write_kernel<TQ, TC, false>, dim3((unsigned)T, shares), dim3(threads), 0, stream, y, y_stride, n_partials,
                  y_partial, y_bias, qw, kw, eps, pos, slot, cos_t, sin_t, rot, interleaved, vcos, vsin, v_interleaved, (TQ*)q_out, (TC*)k_cache, (TC*)v_cache,
                  block_table, max_pages, page_size, nq, nkv, hd, vd, whole, v_from_k, qt_coef, qt_every, status)));
   return check_launch("qk_norm_write");
@@ -1025,7 +1080,7 @@ extern "C" int flint_head_finish(const void* attn, int dtype, const int* pos, co
   if (vd % 2 && vcos) return fail("head_finish: value heads of %d dims cannot rotate in pairs", vd);
   const long long n = (long long)T * nq * ((vd + 1) / 2);
   FLINT_DISPATCH_DTYPE(dtype, TA,
-      launch_pdl(head_finish_kernel<TA>, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream, (const TA*)attn, pos, vcos,
+      launch_pdl(gate_partials > 1 ? head_finish_kernel<TA, true> : head_finish_kernel<TA, false>, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream, (const TA*)attn, pos, vcos,
                  vsin, interleaved, gate, gate_stride, gate_partials, gate_partial, gate_each, (TA*)out, T, nq, vd));
   return check_launch("head_finish");
 }
