@@ -61,9 +61,10 @@ template <> struct Cols<4> {
   }
 };
 
-// RW: rows of S a warp holds (D <= 16 RW); CPL: columns a lane holds (32 CPL columns at a time)
-template <int RW, int CPL, typename TO>
-__global__ void __launch_bounds__(NW * 32)
+// RW: rows of S a warp holds (D <= 16 RW); CPL: columns a lane holds (32 CPL columns at a time); BLOCKS: blocks a multiprocessor
+// (one with all the registers it wants, or, where there are more blocks than multiprocessors, two)
+template <int RW, int CPL, int BLOCKS, typename TO>
+__global__ void __launch_bounds__(NW * 32, BLOCKS)
 delta_token_kernel(const __grid_constant__ TokenArgs a, TO* __restrict__ out) {
   extern __shared__ __align__(16) float sm[];          // sums of the warps [NW][32 CPL], then q [D], k [D], v [V], gate [V], o [V]
   __shared__ float scalars[2], red[32];
@@ -121,13 +122,8 @@ delta_token_kernel(const __grid_constant__ TokenArgs a, TO* __restrict__ out) {
   }
   __syncthreads();
   const float beta = scalars[0], decay = scalars[1];
-  float kr[RW], qr[RW];
-#pragma unroll
-  for (int i = 0; i < RW; ++i) {
-    const int d = warp + NW * i;
-    kr[i] = d < D ? k_s[d] : 0.f;
-    qr[i] = d < D ? q_s[d] : 0.f;
-  }
+  auto key = [&](int i) { return warp + NW * i < D ? k_s[warp + NW * i] : 0.f; };        // of the warp's i-th row
+  auto query = [&](int i) { return warp + NW * i < D ? q_s[warp + NW * i] : 0.f; };
   // ---- the recurrence, a run of columns at a time
   float sq = 0.f;
   for (int c0 = 0; c0 < V; c0 += COLS) {
@@ -137,12 +133,14 @@ delta_token_kernel(const __grid_constant__ TokenArgs a, TO* __restrict__ out) {
 #pragma unroll
     for (int j = 0; j < CPL; ++j) acc[j] = 0.f;
 #pragma unroll
-    for (int i = 0; i < RW; ++i)
+    for (int i = 0; i < RW; ++i) {
+      const float kd = key(i);
 #pragma unroll
       for (int j = 0; j < CPL; ++j) {
         S[i][j] *= decay;
-        acc[j] = fmaf(S[i][j], kr[i], acc[j]);
+        acc[j] = fmaf(S[i][j], kd, acc[j]);
       }
+    }
     Cols<CPL>::store(part + warp * COLS + lane * CPL, acc);
     __syncthreads();
     float u[CPL];
@@ -161,10 +159,11 @@ delta_token_kernel(const __grid_constant__ TokenArgs a, TO* __restrict__ out) {
     }
 #pragma unroll
     for (int i = 0; i < RW; ++i) {
+      const float kd = key(i), qd = query(i);
 #pragma unroll
       for (int j = 0; j < CPL; ++j) {
-        S[i][j] = fmaf(kr[i], u[j], S[i][j]);
-        acc[j] = fmaf(S[i][j], qr[i], acc[j]);
+        S[i][j] = fmaf(kd, u[j], S[i][j]);
+        acc[j] = fmaf(S[i][j], qd, acc[j]);
       }
       const int d = warp + NW * i;
       if (d < D && c < V) Cols<CPL>::store(S_g + (size_t)d * V + c, S[i]);
@@ -188,17 +187,29 @@ delta_token_kernel(const __grid_constant__ TokenArgs a, TO* __restrict__ out) {
   }
 }
 
+template <int RW, int CPL, int BLOCKS, typename TO>
+void launch_form(const TokenArgs& a, int n, TO* out, size_t smem, cudaStream_t stream) {
+  static bool sized = false;             // per instantiation
+  if (smem > 48 * 1024 && !sized) {
+    cudaFuncSetAttribute(delta_token_kernel<RW, CPL, BLOCKS, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    sized = true;
+  }
+  launch_pdl(delta_token_kernel<RW, CPL, BLOCKS, TO>, dim3((unsigned)a.H, (unsigned)n), dim3(NW * 32), smem, stream, a, out);
+}
+
 template <int RW, int CPL>
 int launch_token(const TokenArgs& a, int n, void* out, int out_dtype, size_t smem, cudaStream_t stream) {
+  constexpr int MORE = RW * CPL <= 32 ? 2 : 1;
+  static int sms = 0;
+  if (!sms) {
+    int dev = 0;
+    cudaGetDevice(&dev);
+    cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
+  }
+  const bool many = (long long)a.H * n > sms;
   FLINT_DISPATCH_DTYPE(out_dtype, TO, {
-    if (smem > 48 * 1024) {
-      static bool sized = false;         // per instantiation
-      if (!sized) {
-        cudaFuncSetAttribute(delta_token_kernel<RW, CPL, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
-        sized = true;
-      }
-    }
-    launch_pdl(delta_token_kernel<RW, CPL, TO>, dim3((unsigned)a.H, (unsigned)n), dim3(NW * 32), smem, stream, a, (TO*)out);
+    if (many) launch_form<RW, CPL, MORE, TO>(a, n, (TO*)out, smem, stream);
+    else launch_form<RW, CPL, 1, TO>(a, n, (TO*)out, smem, stream);
   });
   return check_launch("delta_token");
 }
